@@ -72,11 +72,14 @@ class ScheduleEntry:
     its own), and ``cache_from`` lets an entry read the cache that an EARLIER entry
     of the schedule wrote instead of owning one.  ``inject`` is added to the stream
     before the entry runs (a model that repeats a span of its layers marks the start
-    of each pass this way)."""
+    of each pass this way).  ``average``: with X_0 the embedding output and X_(j+1) the
+    result of entry j, what entry i hands on is sum_j w[j] X_j over j = 0 .. i + 1, w being
+    the tensor of ``ModelSpec.extra_tensors`` ([i + 2]) that ``average`` names."""
 
     layer: int
     cache_from: Optional[int] = None
     inject: Optional[StreamInject] = None
+    average: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -126,6 +129,11 @@ class ModelSpec:
                     raise ValueError(
                         f"schedule entry {i} reads the cache of entry {e.cache_from}, "
                         "which owns no cache itself")
+            if e.average is not None and i and self.schedule[i - 1].average is None:
+                raise ValueError(f"schedule entry {i} averages over depth and the entry before it does not: not built")
+            if e.average is not None and tuple(self.extra_tensors.get(e.average, ((),))[0]) != (i + 2,):
+                raise ValueError(f"schedule entry {i} averages over depth by {e.average!r}, which is not a [{i + 2}] tensor of "
+                                 "the model")
             if e.inject is not None and e.inject.mix is not None:
                 if e.inject.embedding or e.inject.vector is not None:
                     raise ValueError(f"schedule entry {i}: the stream is either replaced by a mix or added to, not both")

@@ -6,7 +6,9 @@
 //   * rotation of the first `rot` channels of queries and keys (pairs (i, i + rot/2)), and of ALL channels of the values
 //     (pairs (m, m + dv/2), their own frequencies); a head's output at position i is turned back by -i;
 //   * score = (q . k) * scale * temp[head], then cap * tanh(score / cap);
+//   * minus r1[head] * ln(1 + r2[head] * (i - j)) (a bias by distance, after the cap; not together with blocks);
 //   * one more term exp(sink[head]) in the softmax's denominator, without key or value;
+//   * values divided by their root mean square over the head's channels before they are cached;
 //   * the output multiplied by sigmoid(gate[t, head * dv + c]).
 //
 // Kernels:
@@ -40,13 +42,14 @@ template <typename TT>
 __global__ void pooled_prepare_kernel(const float* __restrict__ proj, long ld, const int* __restrict__ positions,
                                       const float* __restrict__ freq_k, int rot, const float* __restrict__ freq_v,
                                       TT* __restrict__ q_out, long ldq, const int* __restrict__ slots, TT* __restrict__ k_cache,
-                                      TT* __restrict__ v_cache, int H, int G, int dk, int dv, int page_size) {
+                                      TT* __restrict__ v_cache, int H, int G, int dk, int dv, int page_size, float v_eps) {
   extern __shared__ __align__(16) float sm[];
   co_pdl_launch_dependents();
   const size_t t = blockIdx.x;
   const int hk = rot / 2, hv = freq_v ? dv / 2 : 0;
   float* cs_k = sm;               // [hk][2]
   float* cs_v = sm + 2 * hk;      // [hv][2]
+  float* v_mult = cs_v + 2 * hv;  // [G] with v_eps >= 0: 1 / rms of every value head
   co_pdl_wait();
   const float p = (float)positions[t];
   for (int i = threadIdx.x; i < hk + hv; i += blockDim.x) {
@@ -54,8 +57,18 @@ __global__ void pooled_prepare_kernel(const float* __restrict__ proj, long ld, c
     if (i < hk) { pa_sincos(p, freq_k, i, c, s); cs_k[2 * i] = c; cs_k[2 * i + 1] = s; }
     else { pa_sincos(p, freq_v, i - hk, c, s); cs_v[2 * (i - hk)] = c; cs_v[2 * (i - hk) + 1] = s; }
   }
-  __syncthreads();
   const float* row = proj + t * ld;
+  if (v_eps >= 0.f && slots) {
+    const int lane = threadIdx.x & 31;
+    for (int g = threadIdx.x >> 5; g < G; g += blockDim.x >> 5) {
+      const float* src = row + (size_t)(H + G) * dk + (size_t)g * dv;
+      float ss = 0.f;
+      for (int c = lane; c < dv; c += 32) ss = fmaf(src[c], src[c], ss);
+      ss = co_warp_sum(ss);
+      if (lane == 0) v_mult[g] = 1.0f / sqrtf(ss / (float)dv + v_eps);
+    }
+  }
+  __syncthreads();
   size_t k_at = 0, v_at = 0;
   if (slots) {
     const int slot = slots[t];
@@ -85,13 +98,14 @@ __global__ void pooled_prepare_kernel(const float* __restrict__ proj, long ld, c
     const int u = e / per_v, i = e - u * per_v;
     const float* src = vrow + (size_t)u * dv;
     TT* dst = v_cache + v_at + (size_t)u * page_size * dv;
+    const float m = v_eps >= 0.f ? v_mult[u] : 1.f;
     if (i < hv) {
       const float c = cs_v[2 * i], s = cs_v[2 * i + 1];
-      const float a = src[i], b = src[i + hv];
+      const float a = src[i] * m, b = src[i + hv] * m;
       dst[i] = co_from_float<TT>(a * c - b * s);
       dst[i + hv] = co_from_float<TT>(b * c + a * s);
     } else {
-      dst[i + hv] = co_from_float<TT>(src[i + hv]);
+      dst[i + hv] = co_from_float<TT>(src[i + hv] * m);
     }
   }
 }
@@ -139,6 +153,7 @@ struct AttnArgs {
   const int* token_req; const int* positions;
   const float* temps; const float* sinks; const float* gates; long ldgate;
   const float* freq_v;
+  const float* r1; const float* r2;      // [H] each or null: score -= r1 ln(1 + r2 (i - j))
   int H, G, dk, dv, page_size, window, pool, pool_rows;
   float scale, cap;
   int table_room;       // block-table entries that the kernel may keep in shared memory (the pages of a window)
@@ -228,6 +243,7 @@ __global__ void __launch_bounds__(PA_WARPS * 32) pooled_attention_kernel(AttnArg
     for (int b = 0; b < PA_KEYS; ++b) {
       float x = co_warp_sum(s[b]) * mult;
       if (A.cap > 0.f) x = A.cap * tanhf(x / A.cap);
+      if (A.r1) x -= A.r1[h] * log1pf(A.r2[h] * (float)max(i - lo - (n0 + b), 0));
       s[b] = n0 + b < total ? x : -INFINITY;
       m_new = fmaxf(m_new, s[b]);
     }
@@ -423,6 +439,7 @@ __global__ void __launch_bounds__(PG_WARPS * 32) pooled_attention_group_kernel(A
   const float my_mult = A.scale * (A.temps ? A.temps[h0 + my_h] : 1.f);
   float my_m = -INFINITY, my_l = 0.f;          // of head my_h (the lanes of a head agree)
   const float inv_cap = A.cap > 0.f ? 1.0f / A.cap : 0.f;
+  const float my_r1 = A.r1 ? A.r1[h0 + my_h] : 0.f, my_r2 = A.r1 ? A.r2[h0 + my_h] : 0.f;
   auto source = [](int idx) {
     int src = 0;
 #pragma unroll
@@ -457,6 +474,7 @@ __global__ void __launch_bounds__(PG_WARPS * 32) pooled_attention_group_kernel(A
     for (int o2 = 16 >> LOGN; o2 > 0; o2 >>= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], o2);
     float x = v[0] * my_mult;
     if (A.cap > 0.f) x = A.cap * tanhf(x * inv_cap);
+    if (A.r1) x -= my_r1 * log1pf(my_r2 * (float)max(i - lo - (n0 + my_b), 0));
     if (n0 + my_b >= total) x = -INFINITY;
     // the head's keys of this iteration sit in the lanes that differ in bits 4 and 3
     float top = fmaxf(x, __shfl_xor_sync(0xffffffffu, x, 16));
@@ -667,20 +685,21 @@ static bool launch_grouped(const AttnArgs& A, int T, cudaStream_t stream) {
 
 CO_EXPORT int coheryn_pooled_prepare(const float* proj, long ld, const int* positions, const float* freq_k, int rot,
                                      const float* freq_v, void* q_out, long ldq, int dtype, const int* slots, void* k_cache,
-                                     void* v_cache, int T, int H, int G, int dk, int dv, int page_size, cudaStream_t stream) {
+                                     void* v_cache, int T, int H, int G, int dk, int dv, int page_size, float v_eps,
+                                     cudaStream_t stream) {
   if (T <= 0) return 0;
   if (rot < 0 || rot > dk || (rot & 1)) CO_FAIL("pooled_prepare: %d rotated channels of %d", rot, dk);
   if (rot && !freq_k) CO_FAIL("pooled_prepare: a rotation needs frequencies");
   if (freq_v && (dv & 1)) CO_FAIL("pooled_prepare: rotated values need an even number of channels, not %d", dv);
   dim3 grid(T);
   const int threads = 256;
-  const size_t smem = (size_t)(rot + (freq_v ? dv : 0)) * sizeof(float);
+  const size_t smem = (size_t)(rot + (freq_v ? dv : 0) + (v_eps >= 0.f ? G : 0)) * sizeof(float);
   if (dtype == CO_F32)
     co_launch(pooled_prepare_kernel<float>, grid, dim3(threads), smem, stream, proj, ld, positions, freq_k, rot, freq_v, (float*)q_out, ldq,
-              slots, (float*)k_cache, (float*)v_cache, H, G, dk, dv, page_size);
+              slots, (float*)k_cache, (float*)v_cache, H, G, dk, dv, page_size, v_eps);
   else if (dtype == CO_BF16)
     co_launch(pooled_prepare_kernel<__nv_bfloat16>, grid, dim3(threads), smem, stream, proj, ld, positions, freq_k, rot, freq_v,
-              (__nv_bfloat16*)q_out, ldq, slots, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, H, G, dk, dv, page_size);
+              (__nv_bfloat16*)q_out, ldq, slots, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, H, G, dk, dv, page_size, v_eps);
   else CO_FAIL("pooled_prepare: unknown dtype %d", dtype);
   CO_CHECK_LAUNCH("pooled_prepare");
   return 0;
@@ -721,16 +740,17 @@ CO_EXPORT int coheryn_pooled_attention_splits(int T, int H, int G, int dv, long 
 CO_EXPORT int coheryn_pooled_attention(const void* q, long ldq, void* out, long ldo, const void* k, const void* v, const void* pk,
                                        const void* pv, int dtype, const int* tables, int table_width, const int* pool_tables,
                                        int pool_table_width, const int* token_req, const int* positions, const float* temps,
-                                       const float* sinks, const float* gates, long ldgate, const float* freq_v, int T, int H, int G,
-                                       int dk, int dv, int page_size, int window, int pool, int pool_rows, float scale, float cap,
+                                       const float* sinks, const float* gates, long ldgate, const float* freq_v, const float* r1,
+                                       const float* r2, int T, int H, int G, int dk, int dv, int page_size, int window, int pool, int pool_rows, float scale, float cap,
                                        float* scratch, long scratch_floats, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H < 1 || G < 1 || H % G) CO_FAIL("pooled_attention: %d heads over %d key heads", H, G);
   if (dk < 1 || dk > 32 * PA_MAX_PER_LANE || dv < 1 || dv > 32 * PA_MAX_PER_LANE)
     CO_FAIL("pooled_attention: head sizes %d / %d (1..%d)", dk, dv, 32 * PA_MAX_PER_LANE);
   if (pool > 0 && (!pk || !pv || !pool_tables)) CO_FAIL("pooled_attention: blocks need their cache");
+  if ((r1 == nullptr) != (r2 == nullptr) || (r1 && pool > 0)) CO_FAIL("pooled_attention: a bias by distance has two factors and no blocks");
   AttnArgs A{q, ldq, out, ldo, k, v, pk, pv, tables, table_width, pool_tables, pool_table_width, token_req, positions, temps, sinks,
-             gates, ldgate, freq_v, H, G, dk, dv, page_size, window, pool, pool_rows, scale, cap,
+             gates, ldgate, freq_v, r1, r2, H, G, dk, dv, page_size, window, pool, pool_rows, scale, cap,
              window > 0 && window / page_size + 2 <= 2048 ? window / page_size + 2 : 0, 1, scratch};
   A.splits = coheryn_pooled_attention_splits(T, H, G, dv, scratch_floats);
   if (dtype != CO_F32 && dtype != CO_BF16) CO_FAIL("pooled_attention: unknown dtype %d", dtype);

@@ -7,7 +7,7 @@
 //     rest), then the positions from the first one its FIRST row sees, counted in absolute multiples of BN so that a row's
 //     sums do not depend on where its portion was cut; rows and channels of a tile arrive by cp.async through the two
 //     block tables, two stages deep;
-//   * scores S = Q K^T in float32, times scale * temp[head], capped by cap * tanh(S / cap) (computed as
+//   * scores S = Q K^T in float32, times scale * temp[head] (less r1 ln(1 + r2 distance), where the heads have such a bias), capped by cap * tanh(S / cap) (computed as
 //     cap - 2 cap / (exp(2 S / cap) + 1), in units of log 2), masked; online softmax in float32; a weight enters the product with the values as the sum of two bfloat16 numbers (high + low part), so that it
 //     carries sixteen bits of mantissa; the sink joins the denominator at the end;
 //   * epilogue: the row divided by its denominator, turned back by minus its position over all value channels (the pair
@@ -45,6 +45,7 @@ struct TcArgs {
   const int* cu_q; const int* kv_lens;
   const float* temps; const float* sinks; const float* gates; long ldgate;
   const float* freq_v;
+  const float* r1; const float* r2;      // [H] each or null: score -= r1 ln(1 + r2 (i - j))
   int H, G, page_size, window, pool, pool_rows;
   float scale, cap;
 };
@@ -87,6 +88,11 @@ __device__ __forceinline__ void split_pack(float x, float y, unsigned& hi, unsig
 __device__ __forceinline__ float tc_ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float tc_lg2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
 __device__ __forceinline__ float tc_rcp(float x) {
@@ -153,7 +159,7 @@ __global__ void __launch_bounds__(WARPS * 32) pooled_attention_tc_kernel(TcArgs 
       const int prow = b - (int)(((long)lp * A.page_size) / A.pool);
       at = ((size_t)ptable[lp] * A.G + g) * A.pool_rows + prow;
     } else {
-      valid = idx <= p_last;
+      valid = idx <= p_last && idx >= lo_first;       // pages before the window may have been given back
       const int pos = valid ? idx : p_last;
       at = ((size_t)table[pos / A.page_size] * A.G + g) * A.page_size + (size_t)(pos % A.page_size);
     }
@@ -184,6 +190,7 @@ __global__ void __launch_bounds__(WARPS * 32) pooled_attention_tc_kernel(TcArgs 
 
   const float mult = A.scale * (A.temps ? A.temps[h] : 1.f);
   const float inv_cap = A.cap > 0.f ? 1.0f / A.cap : 0.f;
+  const float r1 = A.r1 ? A.r1[h] : 0.f, r2 = A.r1 ? A.r2[h] : 0.f;
   // this thread's two rows
   const int ia = p_first + warp * 16 + gi, ib = ia + 8;
   const int nba = (A.pool > 0 && ia - A.window + 1 > 0) ? (ia - A.window + 1) / A.pool : 0;
@@ -248,6 +255,16 @@ __global__ void __launch_bounds__(WARPS * 32) pooled_attention_tc_kernel(TcArgs 
 #pragma unroll
         for (int e = 0; e < 4; ++e)
           s[n][e] = A.cap > 0.f ? fmaf(-2.0f * cap2, tc_rcp(tc_ex2(s[n][e] * to_exp) + 1.0f), cap2) : s[n][e] * to_log2;
+      }
+      if (A.r1) {       // r1 ln(1 + r2 d) in units of log 2 is r1 log2(1 + r2 d); keys behind the row are masked below
+#pragma unroll
+        for (int n = 0; n < BN / 8; ++n) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int dist = (e >= 2 ? ib : ia) - (first + n * 8 + 2 * ti + (e & 1));
+            s[n][e] = fmaf(-r1, tc_lg2(fmaf(r2, (float)max(dist, 0), 1.0f)), s[n][e]);
+          }
+        }
       }
       if (!inner) {
 #pragma unroll
@@ -374,16 +391,18 @@ CO_EXPORT void coheryn_pooled_tc_shape(int* dk, int* dv) { *dk = DK; *dv = DV; }
 CO_EXPORT int coheryn_pooled_attention_tc(const void* q, long ldq, void* out, long ldo, const void* k, const void* v, const void* pk,
                                           const void* pv, const int* tables, int table_width, const int* pool_tables,
                                           int pool_table_width, const int* cu_q, const int* kv_lens, const float* temps,
-                                          const float* sinks, const float* gates, long ldgate, const float* freq_v, int B,
+                                          const float* sinks, const float* gates, long ldgate, const float* freq_v,
+                                          const float* r1, const float* r2, int B,
                                           int max_q_len, int H, int G, int page_size, int window, int pool, int pool_rows,
                                           float scale, float cap, cudaStream_t stream) {
   if (B <= 0 || max_q_len <= 0) return 0;
   if (H < 1 || G < 1 || H % G) CO_FAIL("pooled_attention_tc: %d heads over %d key heads", H, G);
   if (pool > 0 && (!pk || !pv || !pool_tables || window <= 0)) CO_FAIL("pooled_attention_tc: blocks need their cache and a window");
+  if ((r1 == nullptr) != (r2 == nullptr) || (r1 && pool > 0)) CO_FAIL("pooled_attention_tc: a bias by distance has two factors and no blocks");
   if ((ldq % 8) || ((uintptr_t)q & 15)) CO_FAIL("pooled_attention_tc: query rows must start on 16-byte boundaries");
   TcArgs A{(const __nv_bfloat16*)q, ldq, (__nv_bfloat16*)out, ldo, (const __nv_bfloat16*)k, (const __nv_bfloat16*)v,
            (const __nv_bfloat16*)pk, (const __nv_bfloat16*)pv, tables, table_width, pool_tables, pool_table_width, cu_q, kv_lens,
-           temps, sinks, gates, ldgate, freq_v, H, G, page_size, window, pool, pool_rows, scale, cap};
+           temps, sinks, gates, ldgate, freq_v, r1, r2, H, G, page_size, window, pool, pool_rows, scale, cap};
   const size_t smem = (size_t)(BM * LDK + 2 * BN * LDK + 2 * BN * LDV) * sizeof(__nv_bfloat16);
   static bool configured = false;
   if (!configured) {

@@ -5,36 +5,57 @@
 #include "common.cuh"
 
 // ---------------------------------------------------------------------------------
-// Embedding: out[t, :] = table[ids[t], :]  (float32 residual stream)
+// Embedding: out[t, :] = table[ids[t], :]  (float32 residual stream), optionally plus pos_table[positions[t], :];
+// `out2` (or null) receives the same rows once more (a model that keeps the embedding output beside the stream).
 // ---------------------------------------------------------------------------------
 template <typename TW>
 __global__ void embed_gather_kernel(const TW* __restrict__ table, const int* __restrict__ ids,
-                                    float* __restrict__ out, int H, int V, int* __restrict__ status, float scale) {
+                                    float* __restrict__ out, int H, int V, int* __restrict__ status, float scale,
+                                    const TW* __restrict__ pos_table, const int* __restrict__ positions, int P,
+                                    float* __restrict__ out2) {
   co_pdl_launch_dependents();
   co_pdl_wait();
   const int t = blockIdx.x;
   const int id = ids[t];
-  if (id < 0 || id >= V) {
+  const int p = pos_table ? positions[t] : 0;
+  if (id < 0 || id >= V || (pos_table && (p < 0 || p >= P))) {
     if (threadIdx.x == 0) atomicExch(status, 1);
-    for (int j = threadIdx.x; j < H; j += blockDim.x) out[(size_t)t * H + j] = 0.f;
+    for (int j = threadIdx.x; j < H; j += blockDim.x) {
+      out[(size_t)t * H + j] = 0.f;
+      if (out2) out2[(size_t)t * H + j] = 0.f;
+    }
     return;
   }
   const TW* row = table + (size_t)id * H;
-  if (scale == 1.0f) {
+  if (pos_table || out2) {
+    const TW* prow = pos_table ? pos_table + (size_t)p * H : nullptr;
+    for (int j = threadIdx.x; j < H; j += blockDim.x) {
+      float x = co_to_float(row[j]);
+      if (scale != 1.0f) x *= scale;
+      if (prow) x += co_to_float(prow[j]);
+      out[(size_t)t * H + j] = x;
+      if (out2) out2[(size_t)t * H + j] = x;
+    }
+  } else if (scale == 1.0f) {
     for (int j = threadIdx.x; j < H; j += blockDim.x) out[(size_t)t * H + j] = co_to_float(row[j]);
   } else {   // an architecture that multiplies its embedding rows by a constant
     for (int j = threadIdx.x; j < H; j += blockDim.x) out[(size_t)t * H + j] = co_to_float(row[j]) * scale;
   }
 }
 
+// pos_table: [P][H] of the table's dtype, or null.
 CO_EXPORT int coheryn_embed_gather(const void* table, int table_dtype, const int* ids, float* out,
-                                   int T, int H, int V, int* status, float scale, cudaStream_t stream) {
+                                   int T, int H, int V, int* status, float scale, const void* pos_table,
+                                   const int* positions, int P, float* out2, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (pos_table && !positions) CO_FAIL("embed_gather: a row per position needs the positions");
   const int threads = H >= 1024 ? 256 : 128;
   if (table_dtype == CO_F32)
-    co_launch(embed_gather_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float*)table, ids, out, H, V, status, scale);
+    co_launch(embed_gather_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float*)table, ids, out, H, V, status, scale,
+              (const float*)pos_table, positions, P, out2);
   else if (table_dtype == CO_BF16)
-    co_launch(embed_gather_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, (const __nv_bfloat16*)table, ids, out, H, V, status, scale);
+    co_launch(embed_gather_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, (const __nv_bfloat16*)table, ids, out, H, V, status, scale,
+              (const __nv_bfloat16*)pos_table, positions, P, out2);
   else
     CO_FAIL("embed_gather: unknown table dtype %d", table_dtype);
   CO_CHECK_LAUNCH("embed_gather");
@@ -836,6 +857,184 @@ CO_EXPORT int coheryn_add_normed_rmsnorm(float* resid, const float* parts, int n
     CO_FAIL("add_normed_rmsnorm: unknown output dtype %d", out_dtype);
   }
   CO_CHECK_LAUNCH("add_normed_rmsnorm");
+  return 0;
+}
+
+// ---------------------------------------------------------------------------------
+// A residual add followed by an average over depth, fused with the norm that reads the average:
+//   y = sum_p parts[p];  x = resid + y / rms(y) * post_w   (post_w given), or x = resid + y   (no parts: x = resid)
+//   s = sum_{j < n} avg_w[j] * hist[j] + avg_w[n] * x       (hist[j]: what the stream was after j earlier layers)
+//   hist[n] = x (when keep);  resid = s (when update);  out = s / rms(s) * w  (when w is given)
+// rms(z) = sqrt(mean(z^2) + eps).  One CTA per row.  With `rows` the CTA r reads row rows[r] of the stream, the parts and
+// the history and nothing is written but `out`; `hist_rows` names the history's rows when they are not the stream's.
+// ---------------------------------------------------------------------------------
+struct DepthArgs {
+  float* resid;
+  const float* parts; int n_parts; size_t part_stride; long ldp;
+  const void* post_w; int post_dtype;
+  float* hist; size_t hist_stride; const float* avg_w; int n;
+  const int* rows; const int* hist_rows;
+  const void* w; int w_dtype; float eps;
+  int H, update, keep;
+};
+
+template <typename TO>
+__global__ void __launch_bounds__(256) depth_average_norm_kernel(DepthArgs A, TO* __restrict__ out) {
+  extern __shared__ __align__(16) float row_s[];
+  __shared__ float scratch[33];
+  co_pdl_launch_dependents();
+  co_pdl_wait();
+  const int r = blockIdx.x, H = A.H;
+  const size_t src = A.rows ? (size_t)A.rows[r] : (size_t)r;
+  const size_t hrow = A.hist_rows ? (size_t)A.hist_rows[src] : src;
+  const float invH = 1.0f / (float)H;
+  float ss = 0.f;
+  for (int j = threadIdx.x; j < H; j += blockDim.x) {       // a thread touches its own elements of the row only
+    float y = 0.f;
+    for (int p = 0; p < A.n_parts; ++p) y += A.parts[p * A.part_stride + src * A.ldp + j];
+    row_s[j] = y;
+    ss = fmaf(y, y, ss);
+  }
+  float ps = 1.f;
+  if (A.post_w) {
+    ss = co_block_sum(ss, scratch);
+    ps = 1.0f / sqrtf(ss * invH + A.eps);
+  }
+  float* x = A.resid + src * H;
+  const float wn = A.avg_w[A.n];
+  float sx = 0.f;
+  for (int j = threadIdx.x; j < H; j += blockDim.x) {
+    const float y = row_s[j];
+    const float v = x[j] + (A.post_w ? (y * ps) * co_load_any(A.post_w, A.post_dtype, j) : y);
+    float s = 0.f;
+    for (int k = 0; k < A.n; ++k) s = fmaf(A.avg_w[k], A.hist[k * A.hist_stride + hrow * H + j], s);
+    s = fmaf(wn, v, s);
+    if (A.keep) A.hist[A.n * A.hist_stride + hrow * H + j] = v;
+    if (A.update) x[j] = s;
+    row_s[j] = s;
+    sx = fmaf(s, s, sx);
+  }
+  if (!A.w) return;
+  sx = co_block_sum(sx, scratch);
+  const float xs = 1.0f / sqrtf(sx * invH + A.eps);
+  TO* o = out + (size_t)r * H;
+  for (int j = threadIdx.x; j < H; j += blockDim.x) o[j] = co_from_float<TO>((row_s[j] * xs) * co_load_any(A.w, A.w_dtype, j));
+}
+
+// The same with the row in registers (H a multiple of 4 up to 1024 * VEC, everything on 16-byte boundaries): the history
+// is requested and summed before the reduction over the summand that the rest waits for.
+template <typename TO, int VEC>
+__global__ void __launch_bounds__(256) depth_average_norm_vec_kernel(DepthArgs A, TO* __restrict__ out) {
+  __shared__ float scratch[2][32];
+  co_pdl_launch_dependents();
+  co_pdl_wait();
+  const int r = blockIdx.x, H = A.H, H4 = H >> 2;
+  const size_t src = A.rows ? (size_t)A.rows[r] : (size_t)r;
+  const size_t hrow = A.hist_rows ? (size_t)A.hist_rows[src] : src;
+  const float invH = 1.0f / (float)H;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 y[VEC], s[VEC];
+  float* x = A.resid + src * H;
+  float sy[1] = {0.f};
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int j = threadIdx.x + i * 256;
+    y[i] = zero;
+    if (j < H4)
+      for (int p = 0; p < A.n_parts; ++p) {
+        const float4 d = reinterpret_cast<const float4*>(A.parts + p * A.part_stride + src * A.ldp)[j];
+        y[i].x += d.x; y[i].y += d.y; y[i].z += d.z; y[i].w += d.w;
+      }
+    sy[0] += y[i].x * y[i].x + y[i].y * y[i].y + y[i].z * y[i].z + y[i].w * y[i].w;
+  }
+  float4 xe[VEC];
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int j = threadIdx.x + i * 256;
+    xe[i] = j < H4 ? reinterpret_cast<const float4*>(x)[j] : zero;
+    s[i] = zero;
+    if (j < H4) {
+#pragma unroll 8
+      for (int k = 0; k < A.n; ++k) {
+        const float wk = A.avg_w[k];
+        const float4 h = reinterpret_cast<const float4*>(A.hist + k * A.hist_stride + hrow * H)[j];
+        s[i].x = fmaf(wk, h.x, s[i].x); s[i].y = fmaf(wk, h.y, s[i].y); s[i].z = fmaf(wk, h.z, s[i].z); s[i].w = fmaf(wk, h.w, s[i].w);
+      }
+    }
+  }
+  float ps = 1.f;
+  if (A.post_w) {
+    block_sum_n<1>(sy, scratch[0]);
+    ps = 1.0f / sqrtf(sy[0] * invH + A.eps);
+  }
+  const float wn = A.avg_w[A.n];
+  float sx[1] = {0.f};
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int j = threadIdx.x + i * 256;
+    if (j < H4) {
+      float4 v = y[i];
+      if (A.post_w) {
+        const float4 pw = load4_any(A.post_w, A.post_dtype, j);
+        v = make_float4((v.x * ps) * pw.x, (v.y * ps) * pw.y, (v.z * ps) * pw.z, (v.w * ps) * pw.w);
+      }
+      v = make_float4(xe[i].x + v.x, xe[i].y + v.y, xe[i].z + v.z, xe[i].w + v.w);
+      if (A.keep) reinterpret_cast<float4*>(A.hist + A.n * A.hist_stride + hrow * H)[j] = v;
+      s[i] = make_float4(fmaf(wn, v.x, s[i].x), fmaf(wn, v.y, s[i].y), fmaf(wn, v.z, s[i].z), fmaf(wn, v.w, s[i].w));
+      if (A.update) reinterpret_cast<float4*>(x)[j] = s[i];
+      sx[0] += s[i].x * s[i].x + s[i].y * s[i].y + s[i].z * s[i].z + s[i].w * s[i].w;
+    }
+  }
+  if (!A.w) return;
+  block_sum_n<1>(sx, scratch[1]);
+  const float xs = 1.0f / sqrtf(sx[0] * invH + A.eps);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int j = threadIdx.x + i * 256;
+    if (j < H4) {
+      const float4 wv = load4_any(A.w, A.w_dtype, j);
+      store4(out + (size_t)r * H, (size_t)j, make_float4((s[i].x * xs) * wv.x, (s[i].y * xs) * wv.y, (s[i].z * xs) * wv.z, (s[i].w * xs) * wv.w));
+    }
+  }
+}
+
+// hist: float32 [> n][history rows][H] (`hist_stride` elements between results); avg_w: float32 [n + 1].  parts, post_w, w
+// and out may be null.
+CO_EXPORT int coheryn_depth_average_norm(float* resid, const float* parts, int n_parts, long part_stride, long ldp,
+                                         const void* post_w, int post_dtype, float* hist, long hist_stride, const float* avg_w,
+                                         int n, const int* rows, const int* hist_rows, const void* w, int w_dtype, float eps,
+                                         void* out, int out_dtype, int n_rows, int H, int update, int keep, cudaStream_t stream) {
+  if (n_rows <= 0) return 0;
+  if (n < 1 || !hist || !avg_w) CO_FAIL("depth_average_norm: an average needs its history");
+  if ((parts == nullptr) != (n_parts == 0) || (post_w && !parts)) CO_FAIL("depth_average_norm: %d parts", n_parts);
+  if ((rows && update) || ((rows || hist_rows) && keep)) CO_FAIL("depth_average_norm: cannot write through a row gather");
+  if ((w == nullptr) != (out == nullptr)) CO_FAIL("depth_average_norm: a weight and an output go together");
+  if (out && out_dtype != CO_F32 && out_dtype != CO_BF16) CO_FAIL("depth_average_norm: unknown output dtype %d", out_dtype);
+  const DepthArgs A{resid, parts, n_parts, (size_t)part_stride, ldp, post_w, post_dtype, hist, (size_t)hist_stride, avg_w, n,
+                    rows, hist_rows, w, w_dtype, eps, H, update, keep};
+  const bool bf = out && out_dtype == CO_BF16;
+  const auto aligned = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  if (H % 4 == 0 && H <= 8192 && (part_stride & 3) == 0 && (ldp & 3) == 0 && (hist_stride & 3) == 0 && aligned(resid) &&
+      aligned(parts) && aligned(post_w) && aligned(hist) && aligned(w) && aligned(out)) {
+    const int steps = (H / 4 + 255) / 256;
+#define GO2(TO, V) co_launch(depth_average_norm_vec_kernel<TO, V>, dim3(n_rows), dim3(256), 0, stream, A, (TO*)out)
+#define GO(TO) do { if (steps <= 1) GO2(TO, 1); else if (steps <= 2) GO2(TO, 2); else if (steps <= 4) GO2(TO, 4); else GO2(TO, 8); } while (0)
+    if (bf) GO(__nv_bfloat16); else GO(float);
+#undef GO
+#undef GO2
+  } else {
+    const size_t smem = (size_t)H * sizeof(float);
+    const int threads = H >= 1024 ? 256 : 128;
+#define GO(TO)                                                                                                              \
+  do {                                                                                                                      \
+    auto kern = depth_average_norm_kernel<TO>;                                                                              \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);               \
+    co_launch(kern, dim3(n_rows), dim3(threads), smem, stream, A, (TO*)out);                                                \
+  } while (0)
+    if (bf) GO(__nv_bfloat16); else GO(float);
+#undef GO
+  }
+  CO_CHECK_LAUNCH("depth_average_norm");
   return 0;
 }
 

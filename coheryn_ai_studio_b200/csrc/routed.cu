@@ -3,7 +3,10 @@
 //   * route_select:   per token, from the router's float32 logits: softmax over all outputs, choice score = probability +
 //                     correction, experts in `n_groups` equal groups of neighbours of which only the `keep` groups with the
 //                     largest choice score may be chosen (the others count as minus infinity), the `top` largest choice
-//                     scores, weights = the chosen probabilities / (their sum + 1e-20) * scale;
+//                     scores, weights = the chosen probabilities / (their sum + 1e-20) * scale.  Other routers by mode: the
+//                     scores are the logits and the weights a softmax over the chosen ones, or the scores are sigmoids of
+//                     the logits; a group's score may be the sum of its two largest choice scores, and the weights may
+//                     stay as they are (times scale);
 //   * route_sort:     the (token, choice) pairs that name a real expert (id < n_real) ordered by expert: row ranges per
 //                     expert, each pair's row, each row's token, and the list of (expert, first row) row tiles;
 //   * grouped_linear: C[rows of group g] = A[rows of group g] . W_g^T; the groups are the experts' row ranges (rows
@@ -27,7 +30,8 @@ constexpr int RS_WARPS = 4;
 // smem per warp: choice[N], prob[N], gbest[n_groups]
 __global__ void __launch_bounds__(RS_WARPS * 32)
 route_select_kernel(const float* __restrict__ logits, long ld, const void* __restrict__ correction, int c_dtype, int T, int N,
-                    int n_groups, int keep, int top, float scale, int mode, int* __restrict__ ids, float* __restrict__ weights) {
+                    int n_groups, int keep, int top, float scale, int mode, int group_two, int renormalize,
+                    int* __restrict__ ids, float* __restrict__ weights) {
   extern __shared__ __align__(16) float sm[];
   co_pdl_launch_dependents();
   co_pdl_wait();
@@ -41,6 +45,12 @@ route_select_kernel(const float* __restrict__ logits, long ld, const void* __res
   if (mode == 1) {
     // the choice scores are the logits themselves (plus a bias); the weights come from the chosen ones alone
     for (int i = lane; i < N; i += 32) choice[i] = z[i] + (correction ? co_load_any(correction, c_dtype, i) : 0.f);
+  } else if (mode == 2) {
+    for (int i = lane; i < N; i += 32) {
+      const float p = 1.0f / (1.0f + expf(-z[i]));
+      prob[i] = p;
+      choice[i] = p + (correction ? co_load_any(correction, c_dtype, i) : 0.f);
+    }
   } else {
     float m = -INFINITY;
     for (int i = lane; i < N; i += 32) m = fmaxf(m, z[i]);
@@ -62,9 +72,13 @@ route_select_kernel(const float* __restrict__ logits, long ld, const void* __res
   if (n_groups > 1 && keep < n_groups) {
     const int per = N / n_groups;
     for (int g = lane; g < n_groups; g += 32) {
-      float b = -INFINITY;
-      for (int i = 0; i < per; ++i) b = fmaxf(b, choice[g * per + i]);
-      gbest[g] = b;
+      float b = -INFINITY, second = -INFINITY;
+      for (int i = 0; i < per; ++i) {
+        const float c = choice[g * per + i];
+        second = fmaxf(second, fminf(b, c));
+        b = fmaxf(b, c);
+      }
+      gbest[g] = group_two && per > 1 ? b + second : b;
     }
     __syncwarp();
     // the `keep` best groups, ties to the lower index; a kept group's best becomes NaN-free marker +inf
@@ -114,7 +128,7 @@ route_select_kernel(const float* __restrict__ logits, long ld, const void* __res
     }
     __syncwarp();
   }
-  const float f = scale / (wsum + 1e-20f);
+  const float f = renormalize ? scale / (wsum + 1e-20f) : scale;
   if (lane < top) weights[(size_t)t * top + lane] *= f;
   for (int r = 32 + lane; r < top; r += 32) weights[(size_t)t * top + r] *= f;
 }
@@ -447,10 +461,11 @@ route_combine_kernel(const float* __restrict__ y, long ldy, const TH* __restrict
 }  // namespace
 
 CO_EXPORT int coheryn_route_select(const float* logits, long ld, const void* correction, int c_dtype, int T, int N, int n_groups,
-                                   int keep, int top, float scale, int mode, int* ids, float* weights, cudaStream_t stream) {
+                                   int keep, int top, float scale, int mode, int group_two, int renormalize, int* ids,
+                                   float* weights, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (N < 1 || top < 1 || top > N) CO_FAIL("route_select: %d choices among %d outputs", top, N);
-  if (mode != 0 && mode != 1) CO_FAIL("route_select: unknown mode %d", mode);
+  if (mode < 0 || mode > 2) CO_FAIL("route_select: unknown mode %d", mode);
   if (n_groups < 1) n_groups = 1;
   if (N % n_groups) CO_FAIL("route_select: %d outputs do not form %d equal groups", N, n_groups);
   if (keep < 1 || keep > n_groups) keep = n_groups;
@@ -459,7 +474,7 @@ CO_EXPORT int coheryn_route_select(const float* logits, long ld, const void* cor
   if (smem > 200 * 1024) CO_FAIL("route_select: %d outputs do not fit in shared memory", N);
   if (smem > 48 * 1024) cudaFuncSetAttribute(route_select_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   co_launch(route_select_kernel, dim3((T + RS_WARPS - 1) / RS_WARPS), dim3(RS_WARPS * 32), smem, stream, logits, ld, correction,
-            c_dtype, T, N, n_groups, keep, top, scale, mode, ids, weights);
+            c_dtype, T, N, n_groups, keep, top, scale, mode, group_two, renormalize, ids, weights);
   CO_CHECK_LAUNCH("route_select");
   return 0;
 }

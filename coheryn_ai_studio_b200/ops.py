@@ -56,7 +56,8 @@ def launch_count() -> int:
 def total_launch_count() -> int:
     """Kernel launches made through every library of this package that is loaded."""
     n = launch_count()
-    for lib in list(_attn_libs.values()) + list(_maps_libs.values()) + [l for l in (_recurrent, _variants, _routed) if l is not None]:
+    for lib in list(_attn_libs.values()) + list(_maps_libs.values()) + list(_pooled_tc_libs.values()) + [
+            l for l in (_recurrent, _variants, _routed, _linear_recurrence, _pooled, _linear_attention) if l is not None]:
         n += int(lib.coheryn_launch_count())
     return n
 
@@ -104,18 +105,26 @@ def _i32(t: torch.Tensor, name: str) -> None:
 
 # ------------------------------------------------------------------------------------
 def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, status: torch.Tensor,
-                 scale: Optional[float] = None) -> None:
-    """out[t] = table[ids[t]] (* scale) as float32.  An id outside the table sets status to 1."""
-    _dev(table, ids, out, status)
+                 scale: Optional[float] = None, pos_table: Optional[torch.Tensor] = None,
+                 positions: Optional[torch.Tensor] = None, copy: Optional[torch.Tensor] = None) -> None:
+    """out[t] = table[ids[t]] (* scale) (+ pos_table[positions[t]]) as float32, written to ``copy`` as well when that is
+    given.  An id (or a position) outside its table sets status to 1."""
+    _dev(table, ids, out, status, pos_table, positions, copy)
     _i32(ids, "ids")
     V, H = table.shape
     T = ids.numel()
     assert out.dtype == torch.float32 and out.shape == (T, H) and out.is_contiguous()
     assert table.is_contiguous()
+    if pos_table is not None:
+        _i32(positions, "positions")
+        assert pos_table.dtype == table.dtype and pos_table.is_contiguous() and pos_table.shape[1] == H
+    if copy is not None:
+        assert copy.dtype == torch.float32 and copy.shape == (T, H) and copy.is_contiguous()
     lib = core()
     _check(lib, lib.coheryn_embed_gather(_ptr(table), _code(table), _ptr(ids), _ptr(out), c_int(T),
                                          c_int(H), c_int(V), _ptr(status), c_float(1.0 if scale is None else scale),
-                                         _stream()))
+                                         _ptr(pos_table), _ptr(positions if pos_table is not None else None),
+                                         c_int(pos_table.shape[0] if pos_table is not None else 0), _ptr(copy), _stream()))
 
 
 def gather_rows(src: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
@@ -285,6 +294,51 @@ def add_normed_rmsnorm(resid: torch.Tensor, parts: torch.Tensor, inner_weights: 
         c_int(_code(post_weight)), _ptr(rows), _ptr(weight if out is not None else None),
         c_int(_code(weight) if weight is not None else F32), c_float(eps), _ptr(out),
         c_int(_code(out) if out is not None else F32), c_int(n), c_int(H), c_int(0 if rows is not None else 1), _stream()))
+
+
+def depth_average_norm(resid: torch.Tensor, parts: Optional[torch.Tensor], post_weight: Optional[torch.Tensor],
+                       history: torch.Tensor, avg_weights: torch.Tensor, index: int, weight: Optional[torch.Tensor], eps: float,
+                       out: Optional[torch.Tensor], rows: Optional[torch.Tensor] = None,
+                       history_rows: Optional[torch.Tensor] = None, keep: bool = True) -> None:
+    """A residual add, an average over depth and the norm that reads it, in one kernel.  ``parts`` float32 [P, n, H] (or
+    [n, H], or None): y = their sum; x = resid + y / rms(y) * post_weight (``post_weight`` None: resid + y); with
+    ``history`` float32 [> index, m, H] and ``avg_weights`` float32 [index + 1],
+    s = sum_{j < index} avg_weights[j] history[j] + avg_weights[index] x;  history[index] = x (``keep``), resid = s,
+    out = s / rms(s) * weight (when both are given).  With ``rows`` only those rows are read and nothing but ``out`` is
+    written; ``history_rows`` int32 [n]: the history's row of every row of the stream when they are not the same."""
+    _dev(resid, parts, post_weight, history, avg_weights, weight, out, rows, history_rows)
+    H = resid.shape[-1]
+    assert resid.dtype == torch.float32 and resid.is_contiguous() and history.dtype == torch.float32
+    assert history.dim() == 3 and history.shape[2] == H and history.stride(1) == H and history.stride(2) == 1
+    assert history.shape[0] > index if keep else history.shape[0] >= index
+    _f32(avg_weights, "avg_weights")
+    assert avg_weights.shape == (index + 1,) and avg_weights.is_contiguous()
+    n = resid.shape[0]
+    if parts is not None:
+        if parts.dim() == 2:
+            parts = parts.unsqueeze(0)
+        assert parts.dtype == torch.float32 and parts.stride(2) == 1 and parts.shape[2] == H and parts.shape[1] == n
+    if post_weight is not None:
+        assert post_weight.shape == (H,) and post_weight.is_contiguous()
+    if history_rows is not None:
+        _i32(history_rows, "history_rows")
+        assert history_rows.numel() == n
+    else:
+        assert history.shape[1] == n
+    update = rows is None
+    if rows is not None:
+        _i32(rows, "rows")
+        n = rows.numel()
+    if out is not None:
+        assert weight is not None and weight.shape == (H,) and out.is_contiguous() and out.shape == (n, H)
+    lib = core()
+    _check(lib, lib.coheryn_depth_average_norm(
+        _ptr(resid), _ptr(parts), c_int(parts.shape[0] if parts is not None else 0), c_long(parts.stride(0) if parts is not None else 0),
+        c_long(parts.stride(1) if parts is not None else 0), _ptr(post_weight), c_int(_code(post_weight) if post_weight is not None else F32),
+        _ptr(history), c_long(history.stride(0)), _ptr(avg_weights), c_int(index), _ptr(rows), _ptr(history_rows),
+        _ptr(weight if out is not None else None), c_int(_code(weight) if weight is not None else F32), c_float(eps), _ptr(out),
+        c_int(_code(out) if out is not None else F32), c_int(n), c_int(H), c_int(1 if update else 0),
+        c_int(1 if keep and update and history_rows is None else 0), _stream()))
 
 
 def rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, cos_sin: torch.Tensor,
@@ -1392,12 +1446,17 @@ def set_grouped_tc(on: bool) -> None:
     GROUPED_TC = bool(on)
 
 
+ROUTER_SCORES = {"softmax": 0, "logits": 1, "sigmoid": 2}
+
+
 def route_select(logits: torch.Tensor, correction: Optional[torch.Tensor], n_groups: int, keep: int, top: int,
-                 scale: float, chosen_softmax: bool = False):
+                 scale: float, scores: str = "softmax", group_score: str = "max", renormalize: bool = True):
     """From router logits (float32 [T, N]) the chosen outputs per token (int32 [T, top], by choice score = softmax +
     correction, only within the ``keep`` best of ``n_groups`` equal groups of neighbours) and their weights (float32
-    [T, top]: the chosen probabilities over their sum, times ``scale``).  ``chosen_softmax``: the choice scores are the
-    logits themselves plus ``correction`` (a bias), and the weights the softmax over the chosen scores alone."""
+    [T, top]: the chosen probabilities over their sum, times ``scale``).  ``scores`` "logits": the choice scores are the
+    logits themselves plus ``correction`` (a bias), and the weights the softmax over the chosen scores alone; "sigmoid": a
+    sigmoid per output takes the softmax's place.  ``group_score`` "two": a group counts with the sum of its two largest
+    choice scores instead of its largest.  ``renormalize`` False: the weights are the chosen scores times ``scale``."""
     _dev(logits, correction)
     _f32(logits, "logits")
     T, N = logits.shape
@@ -1410,7 +1469,8 @@ def route_select(logits: torch.Tensor, correction: Optional[torch.Tensor], n_gro
     _check(lib, lib.coheryn_route_select(_ptr(logits), c_long(logits.stride(0)), _ptr(correction),
                                          c_int(_code(correction) if correction is not None else F32), c_int(T), c_int(N),
                                          c_int(n_groups), c_int(keep), c_int(top), c_float(scale),
-                                         c_int(1 if chosen_softmax else 0), _ptr(ids), _ptr(weights), _stream()))
+                                         c_int(ROUTER_SCORES[scores]), c_int(1 if group_score == "two" else 0),
+                                         c_int(1 if renormalize else 0), _ptr(ids), _ptr(weights), _stream()))
     return ids, weights
 
 
@@ -1669,11 +1729,12 @@ def pooled_tc_lib(dk: int, dv: int):
 
 def pooled_prepare(proj: torch.Tensor, positions: torch.Tensor, freq_k: Optional[torch.Tensor], rot: int,
                    freq_v: Optional[torch.Tensor], slots: Optional[torch.Tensor], k_cache, v_cache, heads: int, kv_heads: int,
-                   dk: int, dv: int, page_size: int, dtype: torch.dtype) -> torch.Tensor:
+                   dk: int, dv: int, page_size: int, dtype: torch.dtype, value_eps: Optional[float] = None) -> torch.Tensor:
     """``proj`` float32 [T, >= heads * dk + kv_heads * (dk + dv)]: queries, keys, values side by side.  The first ``rot``
     channels of every query and key head are rotated by the row's position (``freq_k`` float32 [rot/2, 2], high and low
     part of each pair's frequency), all ``dv`` channels of every value head by ``freq_v`` ([dv/2, 2]; None: values stay as
-    they are); keys and values go to the cache at ``slots`` (None: only queries are made).  Returns q [T, heads * dk]."""
+    they are); ``value_eps``: every value head is first divided by sqrt(mean of its squares + value_eps).  Keys and values go
+    to the cache at ``slots`` (None: only queries are made).  Returns q [T, heads * dk]."""
     _dev(proj, positions, freq_k, freq_v, slots, k_cache, v_cache)
     _f32(proj, "proj"); _i32(positions, "positions")
     T = proj.shape[0]
@@ -1690,7 +1751,7 @@ def pooled_prepare(proj: torch.Tensor, positions: torch.Tensor, freq_k: Optional
     _check(lib, lib.coheryn_pooled_prepare(
         _ptr(proj), c_long(proj.stride(0)), _ptr(positions), _ptr(freq_k), c_int(rot if freq_k is not None else 0), _ptr(freq_v),
         _ptr(q), c_long(q.stride(0)), c_int(_CODES[dtype]), _ptr(slots), _ptr(k_cache), _ptr(v_cache), c_int(T), c_int(heads),
-        c_int(kv_heads), c_int(dk), c_int(dv), c_int(page_size), _stream()))
+        c_int(kv_heads), c_int(dk), c_int(dv), c_int(page_size), c_float(-1.0 if value_eps is None else value_eps), _stream()))
     return q
 
 
@@ -1716,18 +1777,21 @@ def pooled_attention(q: torch.Tensor, out: torch.Tensor, k_cache, v_cache, pk_ca
                      pool_group: Optional[int], heads: int, kv_heads: int, dk: int, dv: int, page_size: int,
                      window: Optional[int], pool: Optional[int], scale: float, softcap: Optional[float],
                      temps: Optional[torch.Tensor], sinks: Optional[torch.Tensor], gates: Optional[torch.Tensor],
-                     freq_v: Optional[torch.Tensor]) -> None:
+                     freq_v: Optional[torch.Tensor], log_bias=None) -> None:
     """Attention of every row of the step over the last ``window`` positions of its request and the means of the blocks
     of ``pool`` positions that lie wholly before them (see csrc/attention_pooled.cu).  q [T, heads * dk], out
     [T, heads * dv] in the caches' dtype; ``temps``, ``sinks`` float32 [heads]; ``gates`` float32 [T, heads * dv] (rows may
-    be strided): the output passes sigmoid(gates); ``freq_v``: the values were rotated, the output is turned back."""
+    be strided): the output passes sigmoid(gates); ``freq_v``: the values were rotated, the output is turned back;
+    ``log_bias``: (r1, r2) float32 [heads] each, the score of a key d positions back loses r1 ln(1 + r2 d) (without blocks)."""
     tables = step.block_tables[group]
     ptables = step.block_tables[pool_group] if pool else None
     _dev(q, out, k_cache, v_cache, pk_cache, pv_cache, tables, ptables, step.token_req, step.positions, temps, sinks, gates, freq_v)
     T = q.shape[0]
     assert q.stride(1) == 1 and out.stride(1) == 1 and q.shape[1] == heads * dk and out.shape == (T, heads * dv)
     assert k_cache.dtype == q.dtype and v_cache.dtype == q.dtype and out.dtype == q.dtype
-    for v in (temps, sinks):
+    r1, r2 = log_bias if log_bias is not None else (None, None)
+    _dev(r1, r2)
+    for v in (temps, sinks, r1, r2):
         if v is not None:
             assert v.dtype == torch.float32 and v.is_contiguous() and v.numel() == heads
     if gates is not None:
@@ -1746,7 +1810,7 @@ def pooled_attention(q: torch.Tensor, out: torch.Tensor, k_cache, v_cache, pk_ca
             _ptr(q), c_long(q.stride(0)), _ptr(out), c_long(out.stride(0)), _ptr(k_cache), _ptr(v_cache), _ptr(pk_cache),
             _ptr(pv_cache), _ptr(tables), c_int(tables.shape[1]), _ptr(ptables), c_int(ptables.shape[1] if ptables is not None else 0),
             _ptr(step.cu_q), _ptr(step.kv_lens), _ptr(temps), _ptr(sinks), _ptr(gates),
-            c_long(gates.stride(0) if gates is not None else 0), _ptr(freq_v), c_int(len(q_lens)), c_int(max(q_lens)), c_int(heads),
+            c_long(gates.stride(0) if gates is not None else 0), _ptr(freq_v), _ptr(r1), _ptr(r2), c_int(len(q_lens)), c_int(max(q_lens)), c_int(heads),
             c_int(kv_heads), c_int(page_size), c_int(window or 0), c_int(pool or 0), c_int(pk_cache.shape[2] if pool else 0),
             c_float(scale), c_float(softcap or 0.0), _stream()))
         return
@@ -1758,6 +1822,58 @@ def pooled_attention(q: torch.Tensor, out: torch.Tensor, k_cache, v_cache, pk_ca
         _ptr(q), c_long(q.stride(0)), _ptr(out), c_long(out.stride(0)), _ptr(k_cache), _ptr(v_cache), _ptr(pk_cache),
         _ptr(pv_cache), c_int(_code(q)), _ptr(tables), c_int(tables.shape[1]), _ptr(ptables),
         c_int(ptables.shape[1] if ptables is not None else 0), _ptr(step.token_req), _ptr(step.positions), _ptr(temps), _ptr(sinks),
-        _ptr(gates), c_long(gates.stride(0) if gates is not None else 0), _ptr(freq_v), c_int(T), c_int(heads), c_int(kv_heads),
+        _ptr(gates), c_long(gates.stride(0) if gates is not None else 0), _ptr(freq_v), _ptr(r1), _ptr(r2), c_int(T), c_int(heads), c_int(kv_heads),
         c_int(dk), c_int(dv), c_int(page_size), c_int(window or 0), c_int(pool or 0),
         c_int(pk_cache.shape[2] if pool else 0), c_float(scale), c_float(softcap or 0.0), _ptr(scratch), c_long(floats), _stream()))
+
+
+# ------------------------------------------------------------------------------------
+# Gated linear attention (csrc/linear_attention.cu, a library of its own that is compiled when a model with such a mixer
+# is first run).
+_linear_attention = None
+
+
+def linear_attention():
+    global _linear_attention
+    if _linear_attention is None:
+        lib = build.linear_attention_library()
+        lib.coheryn_last_error.restype = ctypes.c_char_p
+        lib.coheryn_launch_count.restype = ctypes.c_ulonglong
+        lib.coheryn_gla_scratch.restype = ctypes.c_long
+        _linear_attention = lib
+    return _linear_attention
+
+
+# A step whose longest run of tokens is at most this takes the tokens one by one with the state in registers; longer runs
+# take the kernels over chunks of 64 tokens.
+GLA_FEW_TOKENS = int(os.environ.get("COHERYN_GLA_FEW_TOKENS", "8"))
+
+
+def gated_linear_attention(q, k, v, gate, a1, a2, a2_bias, tau: float, q_scale: float, state: torch.Tensor, step, heads: int, dk: int,
+                           dv: int, norm_weight: torch.Tensor, eps: float, out: torch.Tensor, gate_activation: str = "silu") -> None:
+    """S_t = diag(exp(l_t)) S_(t-1) + k_t v_t^T, o_t = S_t^T (q_scale q_t) per request and head, with
+    l_t = log sigmoid(a2 a1_t + a2_bias) / tau per head and key channel; out_t = o_t / rms(o_t) * norm_weight * act(gate_t).
+    ``q``, ``k`` float32 [T, heads * dk], ``v``, ``gate`` float32 [T, heads * dv], ``a1`` float32 [T, rank] (column slices
+    are fine); ``a2`` [heads * dk, rank], ``a2_bias`` [heads * dk] or None; ``state`` float32 [slots, heads * dk * dv] (rows
+    may be strided), read at a request's first token of the step and written behind its last; ``norm_weight`` [dv];
+    ``out`` [T, heads * dv] float32 or bfloat16."""
+    _dev(q, k, v, gate, a1, a2, a2_bias, state, norm_weight, out, step.cu_q, step.state_slots)
+    T = q.shape[0]
+    for name, t, n in (("q", q, heads * dk), ("k", k, heads * dk), ("v", v, heads * dv), ("gate", gate, heads * dv), ("a1", a1, a2.shape[1])):
+        assert t.dtype == torch.float32 and t.stride(1) == 1 and t.shape == (T, n), name
+    assert a2.shape[0] == heads * dk and a2.is_contiguous() and norm_weight.shape == (dv,) and norm_weight.is_contiguous()
+    if a2_bias is not None:
+        assert a2_bias.shape == (heads * dk,) and a2_bias.is_contiguous()
+    _f32(state, "state")
+    assert state.shape[1] == heads * dk * dv and state.stride(1) == 1 and out.shape == (T, heads * dv) and out.stride(1) == 1
+    lib = linear_attention()
+    B, longest, few = step.num_requests, int(step.max_q_len), GLA_FEW_TOKENS
+    floats = int(lib.coheryn_gla_scratch(c_int(T), c_int(B), c_int(longest), c_int(few), c_int(heads), c_int(dk), c_int(dv)))
+    scratch = torch.empty(floats, dtype=torch.float32, device=q.device) if floats else None
+    _check(lib, lib.coheryn_gla(
+        _ptr(q), c_long(q.stride(0)), _ptr(k), c_long(k.stride(0)), _ptr(v), c_long(v.stride(0)), _ptr(gate), c_long(gate.stride(0)),
+        _ptr(a1), c_long(a1.stride(0)), _ptr(a2), c_int(_code(a2)), _ptr(a2_bias), c_int(_code(a2_bias) if a2_bias is not None else F32),
+        c_int(a2.shape[1]), c_float(tau), c_float(q_scale), _ptr(state), c_long(state.stride(0)), _ptr(step.cu_q), _ptr(step.state_slots),
+        _ptr(norm_weight), c_int(_code(norm_weight)), c_float(eps), c_int({"sigmoid": 0, "silu": 1}[gate_activation]), _ptr(out),
+        c_int(_code(out)), c_long(out.stride(0)), _ptr(scratch), c_long(floats), c_int(T), c_int(B), c_int(heads), c_int(dk), c_int(dv),
+        c_int(longest), c_int(few), _stream()))

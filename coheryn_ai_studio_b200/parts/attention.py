@@ -17,7 +17,7 @@ import torch
 from .. import ops
 from ..config.spec import PartSpec
 from ..weights.spec import TensorSpec
-from .base import LayerCache, Mixer, PagedKV, Position, Runtime, StepContext, register_mixer
+from .base import LayerCache, Mixer, PagedKV, Position, Runtime, StepContext, need_halves, register_mixer
 
 
 class Attention(Mixer):
@@ -32,6 +32,7 @@ class Attention(Mixer):
         self.hidden_size, self.num_heads, self.num_kv_heads = hidden_size, num_heads, num_kv_heads
         self.head_dim, self.qkv_bias, self.o_bias = head_dim, bool(qkv_bias), bool(o_bias)
         self.window, self.scale, self.position = window, float(scale), position
+        need_halves(position, "attention")
         self.q_size = num_heads * head_dim
         self.kv_size = num_kv_heads * head_dim
         self.w_qkv = self.b_qkv = self.w_o = self.b_o = None
@@ -269,6 +270,7 @@ class MapsAttention(Mixer):
         self.head_norm = bool(head_norm) if head_norm is not None else self.maps == 2
         self.out_factor = float(out_factor) * float(out_scale) * ((1.0 - self.lambda_init) if self.maps == 2 else 1.0)
         self.own_kv, self.position = bool(own_kv), position
+        need_halves(position, "attention_maps")
         if position is not None and position.rotary_dim > self.dk:
             raise ValueError(f"{position.rotary_dim} rotated channels do not fit a map of {self.dk}")
         self.out_dtype = torch.float32 if float32_output else None
@@ -380,7 +382,8 @@ class LatentAttention(Mixer):
 
     so the attention itself is a multi-query attention over the cached rows whose values are the first ``kv_rank``
     channels of its keys.  The rotated parts turn over their first ``position.rotary_dim`` channels (the encoding's
-    amplitude multiplies cos and sin; ``scale`` is taken as given).  Options: ``sink`` (one more term exp(sink_h) in the
+    amplitude multiplies cos and sin; ``scale`` is taken as given; pairs of neighbouring channels become halves by a
+    permutation of the projections' rows when the weights are bound).  Options: ``sink`` (one more term exp(sink_h) in the
     softmax's denominator with a learned score per head, tensor ``sink``, that carries no value) and ``gate`` (head h's
     output is multiplied by sigmoid(g x)_h, tensor ``g`` [heads, width], the same input as the projections).  A layer
     without keys of its own reads the rows (latent and rotated key) that an earlier one wrote, with its own uk and uv.
@@ -429,6 +432,14 @@ class LatentAttention(Mixer):
 
     def bind(self, tensors):
         H = self.num_heads
+        tensors = dict(tensors)
+        if self.position is not None and self.position.pairs != "halves":
+            # both sides of the rotated part's products in the order the kernels turn
+            order = self.position.halves_order() + list(range(self.position.rotary_dim, self.rd))
+            q, at = tensors["q"].view(H, self.dim + self.rd, self.hidden_size), torch.tensor(order, device=tensors["q"].device)
+            tensors["q"] = torch.cat([q[:, :self.dim], q[:, self.dim + at]], dim=1).reshape(-1, self.hidden_size)
+            if self.own_kv:
+                tensors["dkv"] = torch.cat([tensors["dkv"][:self.rank], tensors["dkv"][self.rank + at]], dim=0)
         # one product for everything that reads the layer's input: queries, latent + key, gate logits
         mats = [tensors["q"]] + ([tensors["dkv"]] if self.own_kv else []) + ([tensors["g"]] if self.gate else [])
         self.w_in = torch.cat(mats, dim=0).contiguous() if len(mats) > 1 else mats[0]
@@ -582,10 +593,15 @@ class PooledWindowAttention(Mixer):
     * ``softcap``: score <- cap tanh(score / cap);
     * ``sink``: the softmax's denominator has one more term exp(sink_h), a learned number per head (tensor ``sink``)
       without key or value, neither scaled nor capped;
-    * ``gate``: the concatenated heads are multiplied by sigmoid(W_g x) (tensor ``g``), x being the mixer's input.
+    * ``gate``: the concatenated heads are multiplied by sigmoid(W_g x) (tensor ``g``), x being the mixer's input;
+    * ``value_eps``: every value head is divided by sqrt(mean of its squares + ``value_eps``), without a weight, before it is
+      rotated and cached;
+    * ``log_bias`` (without blocks): the score of a key d positions back loses r1_h ln(1 + r2_h d) (after the cap; two learned
+      numbers per head, tensors ``r1`` and ``r2``).
 
     The cache is two sets of pages: keys and values of every position, and one row per block (``PagedKV.stride``) that
-    the step which completes a block fills from the cached rows."""
+    the step which completes a block fills from the cached rows.  Without blocks it is one set, whose pages are given back
+    as the window passes them."""
 
     output_parts = 1
 
@@ -593,7 +609,8 @@ class PooledWindowAttention(Mixer):
                  v_head_dim: Optional[int], scale: float, window: Optional[int] = None, pool: Optional[int] = None,
                  qkv_bias: bool = False, rotate_values: bool = False, value_base: Optional[float] = None,
                  head_temps: bool = False, softcap: Optional[float] = None, sink: bool = False, gate: bool = False,
-                 float32_output: bool = True, position: Optional[Position] = None):
+                 value_eps: Optional[float] = None, log_bias: bool = False, float32_output: bool = True,
+                 position: Optional[Position] = None):
         super().__init__(runtime)
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads do not divide into {num_kv_heads} kv heads")
@@ -607,7 +624,11 @@ class PooledWindowAttention(Mixer):
         self.scale, self.window, self.pool = float(scale), window, pool
         self.qkv_bias, self.head_temps, self.sink, self.gate = bool(qkv_bias), bool(head_temps), bool(sink), bool(gate)
         self.softcap = float(softcap) if softcap else None
+        self.value_eps, self.log_bias = float(value_eps) if value_eps is not None else None, bool(log_bias)
+        if self.log_bias and pool is not None:
+            raise ValueError("a bias by distance is not defined for block means")
         self.position = position
+        need_halves(position, "pooled_window_attention")
         if position is not None and position.rotary_dim > self.dk:
             raise ValueError(f"{position.rotary_dim} rotated channels do not fit a head of {self.dk}")
         self.value_position = None
@@ -620,12 +641,13 @@ class PooledWindowAttention(Mixer):
             from .base import POSITIONS, build_part
             self.value_position = build_part(POSITIONS, "position", PartSpec("rope_computed", dict(rotary_dim=self.dv, theta=float(base))), runtime)
         self.out_dtype = torch.float32 if float32_output else None
-        self.w_in = self.b_in = self.w_o = self.temps = self.sinks = None
+        self.w_in = self.b_in = self.w_o = self.temps = self.sinks = self.bias_factors = None
 
     def cache_requirement(self):
-        kv = PagedKV(self.num_kv_heads, self.dk, None, None if self.dv == self.dk else self.dv)
         if self.pool is None:
-            return kv
+            return PagedKV(self.num_kv_heads, self.dk, self.window, None if self.dv == self.dk else self.dv)
+        # a block needs its keys until it is complete: no window gives pages back
+        kv = PagedKV(self.num_kv_heads, self.dk, None, None if self.dv == self.dk else self.dv)
         return (kv, PagedKV(self.num_kv_heads, self.dk, None, None if self.dv == self.dk else self.dv, stride=self.pool))
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
@@ -642,6 +664,8 @@ class PooledWindowAttention(Mixer):
             specs["sink"] = TensorSpec((H,), role="vector", init="bias")
         if self.gate:
             specs["g"] = TensorSpec((H * dv, W))
+        if self.log_bias:
+            specs.update({n: TensorSpec((H,), role="vector", init="norm") for n in ("r1", "r2")})
         return specs
 
     def bind(self, tensors):
@@ -655,6 +679,8 @@ class PooledWindowAttention(Mixer):
         self.w_o = tensors["o"]
         self.temps = tensors["temp"].to(torch.float32).contiguous() if self.head_temps else None
         self.sinks = tensors["sink"].to(torch.float32).contiguous() if self.sink else None
+        if self.log_bias:
+            self.bias_factors = tuple(tensors[n].to(torch.float32).contiguous() for n in ("r1", "r2"))
 
     def output_weights(self):
         return [self.w_o]
@@ -679,7 +705,7 @@ class PooledWindowAttention(Mixer):
         freq_v = self.value_position.frequency_pairs() if self.value_position is not None else None
         q = ops.pooled_prepare(proj, step.positions, pos.frequency_pairs() if pos is not None else None,
                                pos.rotary_dim if pos is not None else 0, freq_v, step.slots[kv.group], kv.k, kv.v, H, G, dk, dv,
-                               kv.page_size, self.runtime.dtype)
+                               kv.page_size, self.runtime.dtype, value_eps=self.value_eps)
         if blocks is not None:
             ops.pooled_means(kv.k, kv.v, blocks.k, blocks.v, step, kv.group, blocks.group, G, dk, dv, kv.page_size, self.pool)
         return q, proj
@@ -692,7 +718,7 @@ class PooledWindowAttention(Mixer):
         ops.pooled_attention(q, out, kv.k, kv.v, blocks.k if blocks is not None else None,
                              blocks.v if blocks is not None else None, step, kv.group,
                              blocks.group if blocks is not None else None, H, G, dk, dv, kv.page_size, self.window, self.pool,
-                             self.scale, self.softcap, self.temps, self.sinks, gates, freq_v)
+                             self.scale, self.softcap, self.temps, self.sinks, gates, freq_v, log_bias=self.bias_factors)
 
     def forward_open(self, x: torch.Tensor, step: StepContext, cache: LayerCache, outs) -> None:
         """The gated heads in front of the output product into ``outs[0]`` [T, heads * vdim]."""

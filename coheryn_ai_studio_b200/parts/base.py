@@ -161,6 +161,36 @@ class PostNormed:
 
 
 @dataclass
+class DepthAverage:
+    """What a schedule entry with ``average`` hands on: the stream, once ``pending`` (a tensor, a stack of partial sums, a
+    :class:`PostNormed`, or None) is added to it, is the entry's result X_index; what follows reads
+    sum_{j < index} weights[j] history[j] + weights[index] X_index.  ``history`` float32 [> index, T, H] holds X_0 (the
+    embedding output) and the earlier entries' results; the norm that forms the average stores X_index there too when a
+    later entry needs it (``keep``).  ``rows``: the history's rows of the stream's rows, when the stream holds only some of
+    the step's."""
+
+    pending: object
+    history: torch.Tensor
+    weights: torch.Tensor
+    index: int
+    keep: bool = True
+    rows: Optional[torch.Tensor] = None
+
+    def resolve(self, residual: torch.Tensor) -> torch.Tensor:
+        """The averaged stream itself, by library operations (traces and tests)."""
+        p = self.pending
+        if p is None or isinstance(p, StreamCopy):
+            x = residual
+        elif hasattr(p, "resolve"):
+            x = residual + p.resolve()
+        else:
+            x = residual + (p.sum(0) if p.dim() == 3 else p.float())
+        h = self.history[:self.index] if self.rows is None else self.history[:self.index, self.rows.long()]
+        w = self.weights.float()
+        return (w[:self.index, None, None] * h).sum(0) + w[self.index] * x
+
+
+@dataclass
 class StreamCopy:
     """What an arrangement hands on in the place of a pending delta when nothing is pending: the float32 stream is
     complete, and ``value`` is the same stream in the compute dtype, ready for the next matrix products (the stream
@@ -240,14 +270,15 @@ class Norm(Part):
 
 class Embedder(Part):
     """Turns the step's token ids into the float32 stream when that takes more than a table row: ``forward(step,
-    state, out)`` fills ``out`` [T, width] and returns a copy in the compute dtype (or ``out`` itself when that is
-    float32).  ``state_requirement()``: a :class:`FixedState` per request that the embedder keeps (for instance the last
+    state, out, status, keep)`` fills ``out`` [T, width] (and ``keep``, when given, with the same rows) and returns a copy in
+    the compute dtype (``out`` itself when that is float32) or None: nothing but the stream.  ``state_requirement()``: a :class:`FixedState` per request that the embedder keeps (for instance the last
     token of the request's previous step), or None.  Its tensors are named in full."""
 
     def state_requirement(self):
         return None
 
-    def forward(self, step: StepContext, state: Optional[LayerCache], out: torch.Tensor, status: torch.Tensor) -> torch.Tensor:
+    def forward(self, step: StepContext, state: Optional[LayerCache], out: torch.Tensor, status: torch.Tensor,
+                keep: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
         raise NotImplementedError
 
 
@@ -255,7 +286,25 @@ class Position(Part):
     """What the stock attention asks of an encoding that turns pairs (i, i + rotary_dim / 2) of a
     head's first ``rotary_dim`` elements: the attribute ``rotary_dim`` and ``cos_sin()``, a float32
     device table [positions, rotary_dim / 2, 2] of (cos, sin).  A mixer of another kind may ask its
-    position part for anything else."""
+    position part for anything else.
+
+    ``pairs``: how the channels that turn together lie in a head, "halves" (i, i + rotary_dim / 2) or "neighbours"
+    (2i, 2i + 1).  The kernels turn halves; ``halves_order`` is how a mixer serves neighbours with them."""
+
+    pairs = "halves"
+
+    def halves_order(self) -> List[int]:
+        """The order of the first ``rotary_dim`` channels that makes the pairs halves: the old index of every new one.  A
+        score does not depend on the order of the channels it is summed over, so a mixer may permute the rows of the
+        projections in front of BOTH its sides by it, once, when the weights are loaded."""
+        n = self.rotary_dim
+        return list(range(n)) if self.pairs == "halves" else list(range(0, n, 2)) + list(range(1, n, 2))
+
+
+def need_halves(position: Optional["Position"], what: str) -> None:
+    """For mixers that hand their channels to the kernels as the checkpoint orders them."""
+    if position is not None and getattr(position, "pairs", "halves") != "halves":
+        raise ValueError(f"{what} turns pairs (i, i + rotary_dim / 2); an encoding of neighbouring channels is not built for it")
 
 
 class Arrangement:

@@ -42,7 +42,7 @@ class PreNormResidual(Arrangement):
         return nb
 
     def forward(self, residual, delta, step, cache):
-        if ops.NATIVE_BLOCK:
+        if ops.NATIVE_BLOCK and (delta is None or isinstance(delta, torch.Tensor)):
             nb = self._native_block()
             if nb:
                 out = nb.run(residual, delta, step, cache)   # the whole block from one call into the library

@@ -5,6 +5,8 @@ row ``buckets`` of ``pair`` (its last) for the first token of a sequence, then o
 before the first one of a step's portion is the last token of the request's previous step: one int32 word of fixed state
 per request, written by the same step after it was read.  One kernel makes the float32 stream and its copy in the
 compute dtype.
+
+``position_table_embedding``: x_t = table[id_t] (* scale) + positions[p_t], a learned row per position.
 """
 from __future__ import annotations
 
@@ -48,7 +50,10 @@ class PairHashEmbedding(Embedder):
     def state_requirement(self):
         return FixedState((1,), torch.int32) if self.pair_name is not None else None
 
-    def forward(self, step: StepContext, state: Optional[LayerCache], out: torch.Tensor, status: torch.Tensor) -> torch.Tensor:
+    def forward(self, step: StepContext, state: Optional[LayerCache], out: torch.Tensor, status: torch.Tensor,
+                keep: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if keep is not None:
+            raise ValueError("pair_hash_embedding: a second copy of the embedding output is not built")
         cast = out if self.runtime.dtype == torch.float32 else torch.empty(out.shape, dtype=self.runtime.dtype, device=out.device)
         last = state.state if state is not None else None
         ops.embed_pair(self.table, self.pair, step, last, self.mul_prev, self.mul_cur, self.buckets, self.scale, self.norm,
@@ -58,4 +63,27 @@ class PairHashEmbedding(Embedder):
         return cast
 
 
+class PositionTableEmbedding(Embedder):
+    def __init__(self, runtime: Runtime, vocab_size: int, hidden_size: int, table: str, positions: str, max_positions: int,
+                 scale: Optional[float] = None):
+        """``table``, ``positions``: full tensor names ([vocab, width], [max_positions, width])."""
+        super().__init__(runtime)
+        self.vocab_size, self.hidden_size, self.max_positions = int(vocab_size), int(hidden_size), int(max_positions)
+        self.table_name, self.positions_name, self.scale = str(table), str(positions), scale
+        self.table = self.rows = None
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        return {self.table_name: TensorSpec((self.vocab_size, self.hidden_size)),
+                self.positions_name: TensorSpec((self.max_positions, self.hidden_size))}
+
+    def bind(self, tensors):
+        self.table, self.rows = tensors[self.table_name], tensors[self.positions_name]
+
+    def forward(self, step: StepContext, state: Optional[LayerCache], out: torch.Tensor, status: torch.Tensor,
+                keep: Optional[torch.Tensor] = None) -> None:
+        ops.embed_gather(self.table, step.token_ids, out, status, scale=self.scale, pos_table=self.rows, positions=step.positions,
+                         copy=keep)
+
+
+register_embedder("position_table_embedding", PositionTableEmbedding)
 register_embedder("pair_hash_embedding", PairHashEmbedding)

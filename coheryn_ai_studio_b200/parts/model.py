@@ -12,7 +12,7 @@ from .. import ops
 from ..config.spec import ModelSpec
 from ..weights.spec import TensorSpec
 from . import attention, block, embedding, feedforward, norm, position, recurrent, routed  # noqa: F401  (register the stock parts)
-from .base import (ARRANGEMENTS, EMBEDDERS, FEED_FORWARDS, MIXERS, NORMS, POSITIONS, LayerCache, Part,
+from .base import (ARRANGEMENTS, EMBEDDERS, FEED_FORWARDS, MIXERS, NORMS, POSITIONS, DepthAverage, LayerCache, Part,
                    Runtime, StepContext, StreamCopy, build_part)
 
 
@@ -116,6 +116,9 @@ class DecoderModel:
         self.head = tensors[self._matrix_name(s.head_name)] if s.head_name is not None else self.embedding
         self.head_bias = tensors[s.head_bias_name] if s.head_bias_name is not None else None
         self.extra = {name: tensors[name] for name in s.extra_tensors}
+        for e in s.schedule:      # what enters the residual sum is float32
+            if e.average is not None:
+                self.extra[e.average] = self.extra[e.average].to(torch.float32).contiguous()
         self.status = torch.zeros(1, dtype=torch.int32, device=self.runtime.device)
 
     # ------------------------------------------------------------------ cache needs
@@ -140,15 +143,25 @@ class DecoderModel:
         step.native = None      # a step object may be run again (warm-up, then capture): on another stream
         residual = torch.empty((T, H), dtype=torch.float32, device=self.runtime.device)
         delta = None
+        last = len(self.spec.schedule) - 1
+        # the results that averages over depth read: the embedding output, then every entry's that a later average needs
+        averaged = [i for i, e in enumerate(self.spec.schedule) if e.average is not None]
+        history = None
+        if averaged:
+            history = torch.empty((averaged[-1] + 1, T, H), dtype=torch.float32, device=self.runtime.device)
+        keep = history[0] if history is not None else None
         if self.embedder is not None:
             own = caches[len(self.spec.schedule)] if len(caches) > len(self.spec.schedule) else None
-            delta = StreamCopy(self.embedder.forward(step, own, residual, self.status))
+            copy = self.embedder.forward(step, own, residual, self.status, keep)
+            delta = StreamCopy(copy) if copy is not None else None
         else:
-            ops.embed_gather(self.embedding, step.token_ids, residual, self.status, scale=self.spec.embedding_scale)
-        last = len(self.spec.schedule) - 1
+            ops.embed_gather(self.embedding, step.token_ids, residual, self.status, scale=self.spec.embedding_scale, copy=keep)
         tailed = False
         for i, (entry, cache) in enumerate(zip(self.spec.schedule, caches)):
             layer = self.layers[entry.layer]
+            if entry.inject is not None and isinstance(delta, DepthAverage):
+                norm.apply_depth_average(residual, delta, None, 0.0, None)      # the stream itself, nothing pending
+                delta = None
             if entry.inject is not None and entry.inject.mix is not None:
                 # the stream, with what is pending, beside the embedding output: one kernel makes the product's input,
                 # the product's float32 result is the new stream and nothing is pending
@@ -169,9 +182,14 @@ class DecoderModel:
                 tailed = True
             else:
                 residual, delta = layer.forward(residual, delta, step, cache)
+            if history is not None and residual is not None and i <= averaged[-1]:
+                delta = DepthAverage(None if isinstance(delta, StreamCopy) else delta, history, self.extra[entry.average], i + 1,
+                                     keep=i < averaged[-1], rows=step.tail_rows if tailed else None)
             if self.layer_observer is not None:
                 if delta is None or isinstance(delta, StreamCopy):
                     out = residual
+                elif isinstance(delta, DepthAverage):
+                    out = delta.resolve(residual)
                 elif hasattr(delta, "resolve"):      # a summand that is normalised before it is added
                     out = residual + delta.resolve()
                 else:

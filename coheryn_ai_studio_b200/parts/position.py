@@ -46,8 +46,9 @@ class RotateHalfRope(Position):
 
 
 class ComputedRope(Position):
-    """Rotate-half rotary encoding whose angles the kernels compute from the position (no table, so no bound on
-    positions): pair i of the first ``rotary_dim`` channels turns by position * f_i, f_i = theta^(-2i / rotary_dim).
+    """Rotary encoding whose angles the kernels compute from the position (no table, so no bound on positions): pair i
+    of the first ``rotary_dim`` channels turns by position * f_i, f_i = theta^(-2i / rotary_dim).  ``pairs``: pair i is
+    channels (i, i + rotary_dim / 2) ("halves") or (2i, 2i + 1) ("neighbours", see ``Position.halves_order``).
 
     ``scaling`` (optional) is the YaRN interpolation by parts: with d(t) = rotary_dim * ln(original / (2 pi t)) /
     (2 ln theta), lo = max(floor(d(fast)), 0), hi = min(ceil(d(slow)), rotary_dim - 1) and
@@ -58,8 +59,11 @@ class ComputedRope(Position):
     forms position * (high + low) without losing the low part, so the angle is good to float32's last bit at any
     position."""
 
-    def __init__(self, runtime: Runtime, rotary_dim: int, theta: float, scaling=None):
+    def __init__(self, runtime: Runtime, rotary_dim: int, theta: float, scaling=None, pairs: str = "halves"):
         super().__init__(runtime)
+        if pairs not in ("halves", "neighbours"):
+            raise ValueError(f"pairs {pairs!r} is not built (halves, neighbours)")
+        self.pairs = pairs
         if rotary_dim % 2 or rotary_dim < 2:
             raise ValueError(f"rotary_dim {rotary_dim} must be even and positive")
         if not theta > 1:

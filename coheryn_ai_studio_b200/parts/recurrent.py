@@ -19,6 +19,10 @@ that runs several mixers side by side.
   r = sigmoid(A_b u_b + a_b), i = sigmoid(B_b u_b + c_b) with square matrices.  log a = -``rate`` r softplus(lam);
   S_t = a S_(t-1) + sqrt(1 - a^2) i u, from S = 0 (no special case for the first token); the output is W_o (S * y).
   State: S (one float32 per channel) and the convolution's last taps-1 inputs.
+* ``GatedLinearAttention`` (kind ``gated_linear_attention``): linear attention with a decay per head and key channel.
+  q = W_q h * d^(-1/2), k = W_k h, v = W_v h;  z = W_a2 (W_a1 h) + b, alpha = sigmoid(z)^(1 / tau);
+  S_t = diag(alpha_t) S_(t-1) + k_t v_t^T from S = 0, o_t = S_t^T q_t.  Each head's o is divided by its root mean square,
+  multiplied by a weight shared by the heads and by silu(W_g h), then W_o.
 * ``SideBySide`` (kind ``side_by_side``): mixers that read the same input; the result is the weighted sum of
   theirs.  Each child multiplies its own output by its weight before its output projection, and the
   children's outputs go to the next norm as separate summands.
@@ -281,6 +285,68 @@ class GatedLinearRecurrence(_StateMixer):
         ops.gated_scan(gates, self.b_r, self.b_i, u, proj[:, :C], self.lam, self.rate, bs, state[:, :C], step, outs[0])
 
 
+class GatedLinearAttention(_StateMixer):
+    def __init__(self, runtime: Runtime, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, tau: float, eps: float,
+                 decay_rank: Optional[int] = None, gate_activation: str = "silu", float32_output: bool = True):
+        """``decay_rank``: the inner size of the decay's two-step projection; None takes it from the checkpoint."""
+        super().__init__(runtime)
+        self.hidden_size, self.num_heads = int(hidden_size), int(num_heads)
+        self.dk, self.dv, self.tau, self.eps = int(head_dim), int(v_head_dim), float(tau), float(eps)
+        if min(self.num_heads, self.dk, self.dv) < 1 or not self.tau > 0:
+            raise ValueError("a gated linear attention needs positive head counts, sizes and tau")
+        if gate_activation not in ("sigmoid", "silu"):
+            raise ValueError("gated_linear_attention: gate_activation is 'sigmoid' or 'silu'")
+        self.decay_rank, self.gate_activation = decay_rank, gate_activation
+        self.out_dtype = torch.float32 if float32_output else None
+        self.stacked = self.w_a2 = self.b_a2 = self.norm_w = self.w_o = None
+
+    def cache_requirement(self):
+        return FixedState((self.num_heads * self.dk * self.dv,), torch.float32)     # S of every head, [dk, dv] rows first
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        W, H, dk, dv, r = self.hidden_size, self.num_heads, self.dk, self.dv, self.decay_rank or -1     # -1: as the checkpoint has it
+        return {"q": TensorSpec((H * dk, W)), "k": TensorSpec((H * dk, W)), "v": TensorSpec((H * dv, W)), "g": TensorSpec((H * dv, W)),
+                "o": TensorSpec((W, H * dv)), "norm": TensorSpec((dv,), role="vector", init="norm"), "a1": TensorSpec((r, W)),
+                "a2": TensorSpec((H * dk, r)), "a2.b": TensorSpec((H * dk,), role="vector", init="bias")}
+
+    def bind(self, tensors):
+        if tensors["a1"].shape[0] != tensors["a2"].shape[1]:
+            raise ValueError("the two steps of the decay's projection do not fit each other")
+        self.stacked = _StackedInput([(n, tensors[n]) for n in ("q", "k", "v", "g", "a1")])     # one product for all that reads h
+        self.w_a2, self.b_a2, self.norm_w, self.w_o = tensors["a2"].contiguous(), tensors["a2.b"], tensors["norm"], tensors["o"]
+
+    def output_weights(self):
+        return [self.w_o]
+
+    def forward_open(self, x: torch.Tensor, step: StepContext, cache: Optional[LayerCache], outs) -> None:
+        """The normalised, gated heads in front of the output product into ``outs[0]`` [T, heads * dv]."""
+        state = self._state_of(cache)
+        st, proj = self.stacked, self.stacked.project(x)
+        ops.gated_linear_attention(st.cut(proj, "q"), st.cut(proj, "k"), st.cut(proj, "v"), st.cut(proj, "g"), st.cut(proj, "a1"),
+                                   self.w_a2, self.b_a2, self.tau, self.dk ** -0.5, state, step, self.num_heads, self.dk, self.dv,
+                                   self.norm_w, self.eps, outs[0], gate_activation=self.gate_activation)
+
+    def _open(self, x, step, cache) -> torch.Tensor:
+        o = torch.empty((x.shape[0], self.num_heads * self.dv), dtype=self.runtime.dtype, device=x.device)
+        self.forward_open(x, step, cache, [o])
+        return o
+
+    def forward_into(self, x: torch.Tensor, step: StepContext, cache: Optional[LayerCache], out: torch.Tensor) -> None:
+        ops.linear(self._open(x, step, cache), self.w_o, out=out[0])
+
+    def forward(self, x: torch.Tensor, step: StepContext, cache: Optional[LayerCache]) -> torch.Tensor:
+        return ops.linear(self._open(x, step, cache), self.w_o, out_dtype=self.out_dtype, partial_ok=self.partial_output)
+
+    supports_tail = True
+
+    def forward_tail(self, x: torch.Tensor, step: StepContext, cache: Optional[LayerCache]) -> Optional[torch.Tensor]:
+        """The state passes every row; the output product runs for the wanted rows only."""
+        o = self._open(x, step, cache)
+        if not step.tail.num_tokens:
+            return None
+        return ops.linear(ops.gather_rows(o, step.tail_rows), self.w_o, out_dtype=self.out_dtype, partial_ok=self.partial_output)
+
+
 class SideBySide(Mixer):
     def __init__(self, runtime: Runtime, hidden_size: int, mixers: Sequence[Tuple[str, PartSpec, float]], position=None,
                  combine: str = "sum", eps: float = 1e-6):
@@ -367,5 +433,6 @@ class SideBySide(Mixer):
 
 register_mixer("matrix_memory", MatrixMemory)
 register_mixer("gated_delta_rule", GatedDeltaRule)
+register_mixer("gated_linear_attention", GatedLinearAttention)
 register_mixer("gated_linear_recurrence", GatedLinearRecurrence)
 register_mixer("side_by_side", SideBySide)

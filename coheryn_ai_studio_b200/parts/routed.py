@@ -11,7 +11,10 @@ their sum (+ 1e-20) times ``scale``; the result is the weighted sum of the chose
 
 ``selection = "top_softmax"`` is the other common router: the choice scores are the logits themselves (plus a bias
 ``router.b`` when ``router_bias``), the ``top`` largest are chosen and the weights are the softmax over the chosen logits
-alone (times ``scale``); groups and identity outputs work as above, ``correction`` does not apply.  ``shared``: one more
+alone (times ``scale``); groups and identity outputs work as above, ``correction`` does not apply.  ``selection =
+"sigmoid_top"``: s = sigmoid(z) per output in the softmax's place.  Independent of the selection: ``group_score = "two"``
+(a group's score is the sum of its two largest choice scores) and, where the weights are scores, ``renormalize`` False
+(they are taken as they are, times ``scale``).  ``shared``: one more
 expert of the same form (tensors ``shared.gate``, ``shared.up``, ``shared.down``; its own size and activation constant)
 that every token uses; with ``gate`` its output is multiplied by sigmoid(w . x), one number per token (tensor
 ``shared.sg`` [1, width]), before it is added.
@@ -39,16 +42,22 @@ from .base import FeedForward, Runtime, StepContext, register_feed_forward
 
 class RoutedExperts(FeedForward):
     output_parts = 1
+    SCORES = {"softmax_top": "softmax", "top_softmax": "logits", "sigmoid_top": "sigmoid"}     # selection -> ops.ROUTER_SCORES
 
     def __init__(self, runtime: Runtime, hidden_size: int, expert_size: int, experts: int, top: int, identity: int = 0,
                  groups: int = 1, keep: Optional[int] = None, scale: float = 1.0, correction: bool = True,
                  activation: str = "silu", expert_prefix: str = "e", tensors=("gate", "up", "down"),
                  activation_constant: Optional[float] = None, selection: str = "softmax_top", router_bias: bool = False,
-                 shared: Optional[dict] = None):
+                 shared: Optional[dict] = None, group_score: str = "max", renormalize: bool = True):
         """``shared``: None or {"size": .., "activation_constant": .. (None: the experts'), "gate": bool}."""
         super().__init__(runtime)
-        if selection not in ("softmax_top", "top_softmax"):
-            raise ValueError(f"router selection {selection!r} is not built (softmax_top, top_softmax)")
+        if selection not in self.SCORES:
+            raise ValueError(f"router selection {selection!r} is not built ({', '.join(self.SCORES)})")
+        if group_score not in ("max", "two"):
+            raise ValueError(f"group score {group_score!r} is not built (max, two)")
+        if selection == "top_softmax" and not renormalize:
+            raise ValueError("the weights of selection 'top_softmax' are a softmax over the chosen logits: they sum to one")
+        self.group_score, self.renormalize = group_score, bool(renormalize)
         self.selection, self.router_bias = selection, bool(router_bias)
         if selection == "top_softmax":
             correction = False
@@ -121,7 +130,8 @@ class RoutedExperts(FeedForward):
         """(ids, weights, pre-activation of the shared expert's gate [T] or None)."""
         logits = ops.linear(x, self.w_router, out_dtype=torch.float32)
         ids, weights = ops.route_select(logits[:, :self.outputs], self.w_correction, self.groups, self.keep, self.top, self.scale,
-                                        chosen_softmax=self.selection == "top_softmax")
+                                        scores=self.SCORES[self.selection], group_score=self.group_score,
+                                        renormalize=self.renormalize)
         return ids, weights, logits[:, self.outputs] if logits.shape[1] > self.outputs else None
 
     def forward(self, x: torch.Tensor, step: StepContext) -> torch.Tensor:

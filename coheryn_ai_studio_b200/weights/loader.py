@@ -131,7 +131,7 @@ def random_tensors(expected: Dict[str, TensorSpec], seed: int, policy: InitPolic
             out[name] = torch.zeros(spec.shape, dtype=torch.int32, device=device)
             continue
         dt = store
-        if spec.init == "norm" and vector_dtype is not None:
+        if spec.init in ("norm", "centered") and vector_dtype is not None:
             dt = vector_dtype
         if spec.init == "zeros":
             out[name] = torch.zeros(spec.shape, dtype=dt, device=device)
@@ -140,7 +140,7 @@ def random_tensors(expected: Dict[str, TensorSpec], seed: int, policy: InitPolic
             raise ValueError(f"tensor {name}: a size that only a checkpoint gives must be named to make random weights")
         try:
             mean, deviation = {"normal": (0.0, policy.matrix_std), "bias": (0.0, policy.bias_std),
-                               "norm": (1.0, policy.norm_jitter), "conv": (0.0, policy.conv_std)}[spec.init]
+                               "norm": (1.0, policy.norm_jitter), "centered": (0.0, policy.norm_jitter), "conv": (0.0, policy.conv_std)}[spec.init]
         except KeyError:
             raise ValueError(f"tensor {name}: unknown init {spec.init!r}") from None
         out[name] = seeded_tensor(seed, name, spec.shape, mean, deviation, dtype=dt, device=device)

@@ -16,7 +16,8 @@ class TensorSpec:
     * ``int_table`` – integer tables, kept as int32.
 
     ``init`` names how the random-weights mode fills it: ``normal`` (matrix_std),
-    ``bias`` (bias_std), ``norm`` (1 + norm_jitter * N(0,1)), ``zeros``.
+    ``bias`` (bias_std), ``norm`` (1 + norm_jitter * N(0,1)), ``centered`` (norm_jitter * N(0,1)),
+    ``conv`` (conv_std), ``zeros``.
     """
 
     shape: Tuple[int, ...]

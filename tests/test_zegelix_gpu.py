@@ -193,7 +193,7 @@ def test_router_takes_the_largest_logits_and_weighs_the_chosen_alone(experts, to
     z = rng.normal(0, 2.0, (T, experts)).astype(np.float32)
     b = rng.normal(0, bias, experts).astype(np.float32)
     wide = dev(np.concatenate([z, rng.normal(0, 9.0, (T, 2)).astype(np.float32)], axis=1))     # columns behind the logits are not read
-    ids, weights = ops.route_select(wide[:, :experts], dev(b), 1, 1, top, 1.0, chosen_softmax=True)
+    ids, weights = ops.route_select(wide[:, :experts], dev(b), 1, 1, top, 1.0, scores="logits")
     total = z.astype(np.float64) + b
     order = np.argsort(-total, axis=1, kind="stable")[:, :top]
     chosen = np.take_along_axis(total, order, axis=1)
