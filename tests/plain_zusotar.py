@@ -179,7 +179,29 @@ def route(h, W, p, router):
     return ids, np.take_along_axis(s, ids, axis=-1)
 
 
-def expert_mixture(h, W, p, mlp, rounder=_same):
+def route_margin(h, W, p, router):
+    """How close the router's choices are, per token: the smaller of the gaps between the last chosen and the first refused
+    score, and between the last kept and the first refused group (infinite where there is nothing to refuse)."""
+    s = sigmoid(h @ W[p + "router"].T)
+    T, n = s.shape
+    gap, allowed = np.full(T, np.inf), np.ones((T, n), dtype=bool)
+    groups = router.get("groups")
+    if groups is not None and groups["keep"] < groups["count"]:
+        per, keep = n // groups["count"], groups["keep"]
+        best = np.sort(s.reshape(T, groups["count"], per), axis=-1)[..., -2:].sum(-1)
+        order = np.sort(best, axis=-1)[:, ::-1]
+        gap = order[:, keep - 1] - order[:, keep]
+        allowed = np.repeat(best >= order[:, keep - 1:keep], per, axis=-1)
+    for t in range(T):
+        order = np.sort(s[t, allowed[t]])[::-1]
+        if router["top"] < len(order):
+            gap[t] = min(gap[t], order[router["top"] - 1] - order[router["top"]])
+    return gap
+
+
+def expert_mixture(h, W, p, mlp, rounder=_same, margins=None):
+    if margins is not None:
+        margins.append(route_margin(h, W, p, mlp["router"]))
     ids, weights = route(h, W, p, mlp["router"])
     out = np.zeros(h.shape)
     for t in range(h.shape[0]):
@@ -194,7 +216,7 @@ def expert_mixture(h, W, p, mlp, rounder=_same):
 MIXERS = {"latent_attention": latent_attention, "attention": log_bias_attention, "gla": gated_linear_attention}
 
 
-def layer(x, W, cfg, index, rounder=_same):
+def layer(x, W, cfg, index, rounder=_same, margins=None):
     """The layer's result, before the depth average."""
     L, eps, m, p = cfg["layers"][index], cfg["norm"]["eps"], cfg["residual_mult"], f"l{index}."
     y = MIXERS[L["type"]](rounder(rms_around_zero(x, W[p + "norm1"], eps)), W, p + "mix.", L["mixer"], eps, rounder)
@@ -202,13 +224,14 @@ def layer(x, W, cfg, index, rounder=_same):
     mlp = L.get("mlp")
     if mlp is not None:
         h = rounder(rms_around_zero(x, W[p + "norm2"], eps))
-        y = gated(h, W, p + "mlp.", rounder) if mlp["kind"] == "dense" else expert_mixture(h, W, p + "mlp.", mlp, rounder)
+        y = gated(h, W, p + "mlp.", rounder) if mlp["kind"] == "dense" else expert_mixture(h, W, p + "mlp.", mlp, rounder, margins)
         x = x + m * rms_around_zero(y, W[p + "norm2b"], eps)
     return x
 
 
-def forward(tokens, W, cfg, layer_outputs=None, rounded=False):
-    """Logits [T, vocab] of a whole sequence; ``layer_outputs`` (a list) receives what every layer hands on.
+def forward(tokens, W, cfg, layer_outputs=None, rounded=False, margins=None):
+    """Logits [T, vocab] of a whole sequence; ``layer_outputs`` (a list) receives what every layer hands on, ``margins`` (a
+    list) how close every router's choices are.
     ``rounded``: everything a part hands to the next in 16 bits is rounded to bfloat16 (the yardstick of what 8-bit
     mantissas between the parts cost by themselves)."""
     rounder = round_bf16 if rounded else _same
@@ -216,7 +239,7 @@ def forward(tokens, W, cfg, layer_outputs=None, rounded=False):
     x = embedding(tokens, W)
     results = [x]
     for i in range(len(cfg["layers"])):
-        results.append(layer(x, W, cfg, i, rounder))
+        results.append(layer(x, W, cfg, i, rounder, margins))
         x = depth_average(results, W[f"l{i}.dwa"])
         if layer_outputs is not None:
             layer_outputs.append(x.copy())

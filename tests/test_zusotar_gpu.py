@@ -1,0 +1,772 @@
+"""The Zusotar decoder on the GPU against the plain implementation (``plain_zusotar.py``): each mechanism's kernels
+alone, then whole models through the step function, the cache and the scheduler, in float32 and in bfloat16."""
+import types
+
+import numpy as np
+import pytest
+import torch
+
+import plain_zusotar as plain
+import zusotar_cases as sc
+
+pytestmark = pytest.mark.gpu
+DTYPES = ["float32", "bfloat16"]
+NAMES = ["S1", "S2", "S3"]
+DEV = "cuda:0"
+TORCH = {"float32": torch.float32, "bfloat16": torch.bfloat16}
+
+
+@pytest.fixture(scope="module")
+def folders(tmp_path_factory):
+    base = tmp_path_factory.mktemp("zusotar")
+    return {n: sc.make_folder(base, n) for n in NAMES}
+
+
+@pytest.fixture(scope="module")
+def models(folders):
+    from coheryn_ai_studio_b200.engine import load_model
+    cache = {}
+
+    def get(name, dtype):
+        if (name, dtype) not in cache:
+            cache[(name, dtype)] = load_model(folders[name], dtype)[1]
+        return cache[(name, dtype)]
+    return get
+
+
+def vocab(name):
+    return sc.CASES[name][0]["vocab"]
+
+
+def dev(a, dtype=torch.float32):
+    return torch.as_tensor(np.asarray(a), dtype=dtype).to(DEV)
+
+
+def bf(a):
+    return plain.round_bf16(np.asarray(a, dtype=np.float64))
+
+
+def f32(a):
+    return np.asarray(a, dtype=np.float32).astype(np.float64)
+
+
+def stored(dtype):
+    """How test values are rounded so that the device holds them exactly."""
+    return bf if dtype == "bfloat16" else f32
+
+
+def same(a):
+    return a
+
+
+def host(t):
+    return t.float().cpu().numpy().astype(np.float64)
+
+
+def runtime(dtype):
+    from coheryn_ai_studio_b200.parts.base import Runtime
+    return Runtime(TORCH[dtype], torch.device(DEV))
+
+
+def bind(part, W, prefix, dtype):
+    """Hand a part its tensors from a dict of float64 arrays, kept as the loader keeps them."""
+    from coheryn_ai_studio_b200.weights.loader import kept_dtype
+    part.bind({n: dev(W[prefix + n]).to(kept_dtype(s, TORCH[dtype], TORCH[dtype])).contiguous() for n, s in part.tensor_specs().items()})
+    return part
+
+
+class Pages:
+    """A hand-made cache for one attention: requests whose pages are handed out in a scrambled order and full of noise, and
+    steps over any runs of their positions.  With a ``window`` the pages that lie wholly before every window of a step are
+    -1 in its block table, as a cache that has given them back leaves it."""
+
+    def __init__(self, lengths, G, dk, dv, page, dtype, window=None, seed=0):
+        from coheryn_ai_studio_b200.parts.base import LayerCache
+        self.page, self.window = page, window
+        pages = [-(-n // page) for n in lengths]
+        order = np.random.default_rng(seed).permutation(sum(pages) + 3)
+        self.table = np.full((len(lengths), max(pages) + 1), -1, dtype=np.int32)
+        at = 0
+        for r, n in enumerate(pages):
+            self.table[r, :n] = order[at:at + n]
+            at += n
+        noise = lambda *shape: torch.randn(shape, device=DEV).mul_(7.0).to(TORCH[dtype])
+        self.k = noise(sum(pages) + 3, G, page, dk)
+        self.v = noise(sum(pages) + 3, G, page, dv) if dv else None
+        self.cache = LayerCache(kind="paged", group=0, page_size=page, k=self.k, v=self.v, writes=True)
+
+    def step(self, runs):
+        """``runs``: (request, first position, tokens) in batch order; the requests' lengths are first + tokens."""
+        req = np.concatenate([np.full(n, i) for i, (_, _, n) in enumerate(runs)]).astype(np.int32)
+        pos = np.concatenate([np.arange(s, s + n) for _, s, n in runs]).astype(np.int32)
+        cu = np.concatenate([[0], np.cumsum([n for _, _, n in runs])]).astype(np.int32)
+        tab = np.stack([self.table[r] for r, _, _ in runs])
+        if self.window is not None:
+            for b, (_, s, _) in enumerate(runs):
+                tab[b, :max(0, s - self.window + 1) // self.page] = -1
+        slots = np.concatenate([self.table[r][np.arange(s, s + n) // self.page] * self.page + np.arange(s, s + n) % self.page
+                                for r, s, n in runs]).astype(np.int32)
+        kv = [s + n for _, s, n in runs]
+        return types.SimpleNamespace(
+            num_requests=len(runs), num_tokens=int(cu[-1]), token_req=dev(req, torch.int32), positions=dev(pos, torch.int32),
+            cu_q=dev(cu, torch.int32), kv_lens=dev(kv, torch.int32), block_tables=[dev(tab, torch.int32)],
+            slots=[dev(slots, torch.int32)], q_lens=[n for _, _, n in runs], kv_lens_host=kv,
+            max_q_len=max(n for _, _, n in runs), max_kv_len=max(kv), prior_positions_settled=True, tail=None, tail_rows=None)
+
+
+def state_step(runs, slots):
+    """A step without pages: ``runs`` as above; ``slots``: the state slot of every request."""
+    cu = np.concatenate([[0], np.cumsum([n for _, _, n in runs])]).astype(np.int32)
+    return types.SimpleNamespace(num_requests=len(runs), num_tokens=int(cu[-1]), cu_q=dev(cu, torch.int32),
+                                 state_slots=dev([slots[r] for r, _, _ in runs], torch.int32), tail=None, tail_rows=None,
+                                 max_q_len=max(n for _, _, n in runs))
+
+
+def cuts(lengths, portions):
+    """Steps of a schedule: request r joins at step r and advances by portions[r][k] tokens in its k-th step."""
+    at = [0] * len(lengths)
+    steps, k = [], 0
+    while any(a < n for a, n in zip(at, lengths)):
+        runs = []
+        for r, n in enumerate(lengths):
+            if at[r] < n and k >= r:
+                take = min(portions[r][(k - r) % len(portions[r])], n - at[r])
+                runs.append((r, at[r], take))
+                at[r] += take
+        steps.append(runs)
+        k += 1
+    return steps
+
+
+def run_mixer(mixer, hs, steps, make_step, cache, dtype, width, before=None):
+    got = [np.zeros((len(h), width)) for h in hs]
+    for runs in steps:
+        if before is not None:
+            before(runs)
+        x = dev(np.concatenate([hs[r][s:s + n] for r, s, n in runs]), TORCH[dtype])
+        out = mixer.forward(x, make_step(runs), cache)
+        out, o = host(out), 0
+        for r, s, n in runs:
+            got[r][s:s + n] = out[o:o + n]
+            o += n
+    return got
+
+
+# ------------------------------------------------------------------------------ the embedding, the average over depth
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H", [64, 100, 1100])
+def test_embedding_with_a_row_per_position_and_its_copy(dtype, H):
+    from coheryn_ai_studio_b200 import ops
+    rng = np.random.default_rng(H)
+    V, P, T = 50, 70, 33
+    table, pos = bf(rng.normal(0, 1, (V, H))), bf(rng.normal(0, 1, (P, H)))
+    ids, at = rng.integers(0, V, T), rng.integers(0, P, T)
+    at[0], at[1] = 0, P - 1
+    out, copy = torch.empty((T, H), device=DEV), torch.empty((T, H), device=DEV)
+    status = torch.zeros(1, dtype=torch.int32, device=DEV)
+    ops.embed_gather(dev(table, TORCH[dtype]), dev(ids, torch.int32), out, status, scale=1.5, pos_table=dev(pos, TORCH[dtype]),
+                     positions=dev(at, torch.int32), copy=copy)
+    assert np.abs(host(out) - (table[ids] * 1.5 + pos[at])).max() < 1e-5 and torch.equal(out, copy) and status.item() == 0
+    ops.embed_gather(dev(table, TORCH[dtype]), dev(ids, torch.int32), out, status, copy=copy)
+    assert np.array_equal(host(copy), table[ids]) and torch.equal(out, copy)
+    at[3] = P                                  # the host refuses such a position; the kernel flags it and reads nothing
+    ops.embed_gather(dev(table, TORCH[dtype]), dev(ids, torch.int32), out, status, pos_table=dev(pos, TORCH[dtype]), positions=dev(at, torch.int32))
+    assert status.item() == 1 and host(out)[3].any() == False  # noqa: E712
+
+
+@pytest.mark.parametrize("H", [64, 100, 1536, 5000])
+@pytest.mark.parametrize("n", [1, 3, 11])
+def test_average_over_depth_with_the_add_before_and_the_norm_behind(H, n):
+    """Every form of what is pending (nothing, a summand, a stack of partial sums; normalised or not), the stream updated or
+    read through a row gather, the history's rows the stream's or others."""
+    from coheryn_ai_studio_b200 import ops
+    rng = np.random.default_rng(H + n)
+    T, eps = 37, 1e-5
+    x = rng.normal(0, 1, (T, H)).astype(np.float32)
+    hist = rng.normal(0, 1, (n + 2, T, H)).astype(np.float32)
+    avg = rng.normal(0, 0.5, n + 1).astype(np.float32)
+    post, w = f32(rng.normal(0.3, 0.2, H)), bf(rng.normal(1, 0.2, H))
+    parts3 = rng.normal(0, 0.02, (3, T, H)).astype(np.float32)        # small: the eps inside the root counts
+    for parts in (None, parts3[0], parts3):
+        for normed in ((False,) if parts is None else (False, True)):
+            y = 0.0 if parts is None else parts.astype(np.float64).reshape(-1, T, H).sum(0)
+            X = x + (plain.rms(y, eps) * post if normed else y)
+            S = plain.depth_average([h for h in hist[:n].astype(np.float64)] + [X], avg)
+            want = plain.rms(S, eps) * w
+            kw = dict(post_weight=dev(post) if normed else None, avg_weights=dev(avg), index=n, weight=dev(w, torch.bfloat16), eps=eps)
+            stream, h = dev(x), dev(hist)
+            for out_dtype, tol in ((torch.float32, 2e-5), (torch.bfloat16, 2e-2)):
+                stream, h = dev(x), dev(hist)
+                out = torch.empty((T, H), dtype=out_dtype, device=DEV)
+                ops.depth_average_norm(stream, dev(parts) if parts is not None else None, history=h, out=out, **kw)
+                assert np.abs(host(out) - want).max() <= tol * np.abs(want).max()
+            assert np.abs(host(stream) - S).max() <= 2e-5 * np.abs(S).max() and np.abs(host(h[n]) - X).max() <= 2e-5 * np.abs(X).max()
+            assert torch.equal(h[:n], dev(hist[:n])) and torch.equal(h[n + 1:], dev(hist[n + 1:]))
+            # only some rows: nothing is written but the output
+            rows = rng.permutation(T)[:9]
+            stream, h = dev(x), dev(hist)
+            out = torch.empty((9, H), dtype=torch.float32, device=DEV)
+            ops.depth_average_norm(stream, dev(parts) if parts is not None else None, history=h, out=out, rows=dev(rows, torch.int32), **kw)
+            assert np.abs(host(out) - want[rows]).max() <= 2e-5 * np.abs(want).max() and torch.equal(stream, dev(x)) and torch.equal(h, dev(hist))
+            # a stream of some rows beside the whole step's history
+            kept = dev(x[rows])
+            out = torch.empty((9, H), dtype=torch.float32, device=DEV)
+            part_rows = None if parts is None else dev(np.ascontiguousarray(parts[..., rows, :]))
+            ops.depth_average_norm(kept, part_rows, history=h, out=out, history_rows=dev(rows, torch.int32), keep=False, **kw)
+            assert np.abs(host(out) - want[rows]).max() <= 2e-5 * np.abs(want).max() and np.abs(host(kept) - S[rows]).max() <= 2e-5 * np.abs(S).max()
+            assert torch.equal(h, dev(hist))
+            # no norm behind it: the stream alone
+            stream = dev(x)
+            ops.depth_average_norm(stream, dev(parts) if parts is not None else None, post_weight=kw["post_weight"], history=h,
+                                   avg_weights=kw["avg_weights"], index=n, weight=None, eps=eps, out=None)
+            assert np.abs(host(stream) - S).max() <= 2e-5 * np.abs(S).max()
+
+
+# ------------------------------------------------------------------------------ gated linear attention
+def gla_weights(rng, width, H, dk, dv, rank, r8, bias):
+    return {"m.q": r8(rng.normal(0, 0.2, (H * dk, width))), "m.k": r8(rng.normal(0, 0.2, (H * dk, width))),
+            "m.v": r8(rng.normal(0, 0.2, (H * dv, width))), "m.g": r8(rng.normal(0, 0.2, (H * dv, width))),
+            "m.o": r8(rng.normal(0, 0.2, (width, H * dv))), "m.norm": r8(rng.normal(1, 0.2, dv)),
+            "m.a1": r8(rng.normal(0, 0.2, (rank, width))), "m.a2": r8(rng.normal(0, 0.2, (H * dk, rank))), "m.a2.b": r8(bias)}
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("width,H,dk,dv,rank,tau", [(64, 2, 32, 64, 16, 16.0), (100, 3, 12, 22, 5, 1.0), (48, 1, 130, 144, 7, 4.0),
+                                                    (64, 2, 64, 32, 40, 0.5), (32, 1, 257, 20, 3, 8.0)])
+def test_gated_linear_attention_in_portions_and_decoded(dtype, width, H, dk, dv, rank, tau):
+    """Two requests in portions of many sizes (across chunks of 64, down to one token, beside each other) over state slots
+    full of noise.  Decays from nearly 1 (a loud first token is still there hundreds of tokens later) to channels that
+    forget more within a chunk than float32's exponents hold."""
+    from coheryn_ai_studio_b200.parts.base import LayerCache
+    from coheryn_ai_studio_b200.parts.recurrent import GatedLinearAttention
+    rng, r8 = np.random.default_rng(dk * dv), stored(dtype)
+    bias = rng.permutation(np.linspace(-12.0 if tau <= 1 else -4.0, 12.0, H * dk))
+    W = gla_weights(rng, width, H, dk, dv, rank, r8, bias)
+    mixer = bind(GatedLinearAttention(runtime(dtype), width, H, dk, dv, tau, 1e-6), W, "m.", dtype)
+    lengths = [331, 45]
+    hs = [r8(rng.normal(0, 1.0, (n, width))) for n in lengths]
+    hs[0][0] *= 12.0
+    m = {"heads": H, "dim": dk, "vdim": dv, "tau": tau}
+    want = [plain.gated_linear_attention(h, W, "m.", m, 1e-6) for h in hs]
+    lost = plain.gated_linear_attention(np.concatenate([hs[0][:1] / 12.0, hs[0][1:]]), W, "m.", m, 1e-6)
+    assert np.abs(lost[-1] - want[0][-1]).max() > 0.01 * np.abs(want[0][-1]).max()        # a lost state would show
+    if tau <= 1:          # ... and channels reach the part of the kernel that carries keys forward by the tokens' own decays
+        z = hs[0] @ W["m.a1"].T @ W["m.a2"].T + W["m.a2.b"]
+        assert (-np.logaddexp(0.0, -z) / tau)[:64].sum(0).min() < -100
+    slots = [3, 1]
+    schedules = [cuts(lengths, [[130, 2, 1, 67, 31, 33, 1, 1, 1, 64], [7, 1, 2, 30, 1]]), cuts(lengths, [[331], [45]]),
+                 cuts(lengths, [[64, 65, 63, 8, 9], [8]])]
+    for steps in schedules:
+        state = torch.randn((5, H * dk * dv), device=DEV) * 3.0
+        fresh = set()
+
+        def admit(runs):
+            for r, _, _ in runs:
+                if r not in fresh:
+                    state[slots[r]].zero_()          # what admission does
+                    fresh.add(r)
+
+        got = run_mixer(mixer, hs, steps, lambda runs: state_step(runs, slots), LayerCache(kind="state", state=state, writes=True),
+                        dtype, width, before=admit)
+        for g, w in zip(got, want):
+            tol = 4e-5 if dtype == "float32" else 4e-2
+            assert np.abs(g - w).max() <= tol * np.abs(w).max(), np.abs(g - w).max() / np.abs(w).max()
+
+
+def test_linear_attention_long_memories_do_not_drift():
+    """A thousand tokens through decays within 1e-4 of 1, one token at a time and in chunks: the error of the state stays at
+    float32's rounding, it does not grow with the position."""
+    from coheryn_ai_studio_b200 import ops
+    rng = np.random.default_rng(4)
+    T, H, dk, dv = 1000, 2, 16, 16
+    q, k, v, g = (rng.normal(0, 1, (T, H * d)) for d in (dk, dk, dv, dv))
+    a2, bias = np.zeros((H * dk, 1)), np.full(H * dk, 9.0)
+    la = np.tile(-np.log1p(np.exp(-9.0)), (T, H, dk))
+    o = plain.linear_attention_scan(f32(q).reshape(T, H, dk), f32(k).reshape(T, H, dk), f32(v).reshape(T, H, dv), la)
+    want = (plain.rms(o, 1e-6)).reshape(T, H * dv) * plain.silu(f32(g))
+    for portion in (1, T):
+        state = torch.zeros((1, H * dk * dv), device=DEV)
+        out = torch.empty((T, H * dv), device=DEV)
+        for t in range(0, T, portion):
+            s = slice(t, t + portion)
+            ops.gated_linear_attention(dev(q[s]), dev(k[s]), dev(v[s]), dev(g[s]), torch.zeros((portion, 1), device=DEV), dev(a2), dev(bias),
+                                       1.0, 1.0, state, state_step([(0, t, portion)], [0]), H, dk, dv, torch.ones(dv, device=DEV), 1e-6, out[s])
+        d = np.abs(host(out) - want).max(1)
+        assert d.max() <= 2e-5 * np.abs(want).max() and d[-100:].mean() <= 4.0 * d[50:150].mean() + 1e-6, (portion, d.max())
+
+
+# ------------------------------------------------------------------------------ the router and the experts
+@pytest.mark.parametrize("experts,top,groups", [(16, 3, (4, 2)), (5, 2, (5, 3)), (8, 3, (2, 1)), (9, 9, None), (40, 7, (8, 3)), (6, 2, (2, 2)), (3, 1, None)])
+def test_router_takes_the_best_groups_and_the_scores_as_weights(experts, top, groups):
+    from coheryn_ai_studio_b200 import ops
+    rng = np.random.default_rng(experts * 10 + top)
+    T = 90
+    z = rng.normal(0, 2.0, (T, experts)).astype(np.float32)
+    wide = dev(np.concatenate([z, rng.normal(0, 9.0, (T, 2)).astype(np.float32)], axis=1))     # columns behind the logits are not read
+    count, keep = groups or (1, 1)
+    ids, weights = ops.route_select(wide[:, :experts], None, count, keep, top, 1.0, scores="sigmoid", group_score="two", renormalize=False)
+    router = {"experts": experts, "top": top}
+    if groups:
+        router["groups"] = {"count": count, "keep": keep}
+    want_ids, want = plain.route(z.astype(np.float64), {"r.router": np.eye(experts)}, "r.", router)
+    assert np.array_equal(ids.cpu().numpy(), want_ids) and np.abs(host(weights) - want).max() < 1e-6
+    if groups and keep < count and experts // count > 2:        # the sum of two chooses other groups than the largest alone
+        by_max, _ = ops.route_select(wide[:, :experts], None, count, keep, top, 1.0, scores="sigmoid", renormalize=False)
+        assert not np.array_equal(by_max.cpu().numpy(), want_ids)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("width,ff,experts,top,groups,shared,T", [(64, 32, 8, 3, (4, 2), 48, 77), (100, 50, 5, 2, (5, 3), 10, 33),
+                                                                  (128, 64, 4, 2, None, None, 300), (64, 16, 6, 6, (2, 2), 16, 2)])
+def test_expert_mixture_with_a_shared_expert(dtype, width, ff, experts, top, groups, shared, T):
+    from coheryn_ai_studio_b200.parts.routed import RoutedExperts
+    rng, r8 = np.random.default_rng(width + T), stored(dtype)
+    W = {"f.router": r8(rng.normal(0, 0.3, (experts, width)))}
+    for e in [f"e{i}" for i in range(experts)] + (["shared"] if shared else []):
+        n = shared if e == "shared" else ff
+        W[f"f.{e}.gate"], W[f"f.{e}.up"] = r8(rng.normal(0, 0.3, (n, width))), r8(rng.normal(0, 0.3, (n, width)))
+        W[f"f.{e}.down"] = r8(rng.normal(0, 0.3, (width, n)))
+    router = {"experts": experts, "top": top}
+    if groups:
+        router["groups"] = {"count": groups[0], "keep": groups[1]}
+    count, keep = groups or (1, 1)
+    part = bind(RoutedExperts(runtime(dtype), width, ff, experts, top, groups=count, keep=keep, correction=False, selection="sigmoid_top",
+                              group_score="two", renormalize=False, shared=dict(size=shared) if shared else None), W, "f.", dtype)
+    h = r8(rng.normal(0, 1.0, (T, width)))
+    want = plain.expert_mixture(h, W, "f.", {"router": router, "shared": {"ff": shared} if shared else None})
+    got = host(part.forward(dev(h, TORCH[dtype]), None))
+    # a near tie of two scores (or groups) may fall the other way in float32 sums: few rows, left out
+    tol = 3e-5 if dtype == "float32" else 3e-2
+    d = np.abs(got - want).max(1) / np.abs(want).max()
+    assert np.median(d) <= tol and (d > tol).mean() <= 0.05, (d.max(), (d > tol).mean())
+
+
+# ------------------------------------------------------------------------------ window attention with the logarithmic bias
+def run_window(q, k, v, lengths, steps, size, page, scale, r1, r2, dtype, G, value_eps=None):
+    """Write k and v through ``pooled_prepare``, attend; rows [sum lengths][H, dv]."""
+    from coheryn_ai_studio_b200 import ops
+    H, dk, dv = q[0].shape[1], q[0].shape[2], v[0].shape[2]
+    pages = Pages(lengths, G, dk, dv, page, dtype, window=size, seed=len(steps))
+    got = [np.zeros((n, H, dv)) for n in lengths]
+    for runs in steps:
+        st = pages.step(runs)
+        proj = np.concatenate([np.concatenate([a[r][s:s + n].reshape(n, -1) for a in (q, k, v)], axis=1) for r, s, n in runs])
+        qd = ops.pooled_prepare(dev(proj), st.positions, None, 0, None, st.slots[0], pages.k, pages.v, H, G, dk, dv, page, TORCH[dtype],
+                                value_eps=value_eps)
+        out = torch.empty((qd.shape[0], H * dv), dtype=TORCH[dtype], device=DEV)
+        ops.pooled_attention(qd, out, pages.k, pages.v, None, None, st, 0, None, H, G, dk, dv, page, size, None, scale, None, None, None,
+                             None, None, log_bias=(dev(r1), dev(r2)))
+        o = 0
+        for r, s, n in runs:
+            got[r][s:s + n] = host(out[o:o + n]).reshape(n, H, dv)
+            o += n
+    return got
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("size,page,H,G,dk,dv", [(24, 16, 4, 2, 32, 16), (7, 16, 3, 3, 20, 14), (5, 8, 6, 2, 10, 6), (1, 16, 6, 1, 16, 48),
+                                                 (36, 64, 2, 1, 80, 256), (72, 16, 8, 4, 48, 48), (33, 8, 4, 1, 16, 128)])
+def test_one_key_that_stands_out_at_the_windows_edges(dtype, size, page, H, G, dk, dv):
+    """A marked position j*: its key and the queries of ALL rows carry one large component, so a row puts nearly all its
+    weight on j* while its window holds it and none from the next row on.  Marks at position 0, on both sides of page borders
+    and far in; whole, in portions and decoded, over block tables whose passed pages are gone."""
+    from coheryn_ai_studio_b200 import ops
+    rng, r8 = np.random.default_rng(size * 100 + dk), stored(dtype)
+    T, marks = 170, [0, 47, 96]
+    q, k, v = r8(rng.normal(0, 0.3, (T, H, dk))), r8(rng.normal(0, 0.3, (T, G, dk))), r8(rng.normal(0, 1.0, (T, G, dv)))
+    q[:, :, 0] = 9.0
+    for j in marks:
+        k[j, :, 0] = 9.0
+    r1, r2 = f32(rng.uniform(0.1, 2.0, H)), f32(rng.uniform(0.05, 0.5, H))
+    want = plain.attend_log_bias(q, k, v, size, 0.2, r1, r2)
+    for j in marks:          # the last row that sees the mark differs from the next one
+        assert np.abs(want[j + size - 1] - want[j + size]).max() > 0.2, j
+    tol = 2e-5 if dtype == "float32" else 3e-2
+    for tensor_cores in ((True, False) if dtype == "bfloat16" else (True,)):      # bfloat16 portions: both kernels
+        ops.set_pooled_tc(tensor_cores)
+        try:
+            for steps in ([[(0, 0, T)]], cuts([T], [[40, 1, 1, 1, 17, 2, 1, 3, 64, 1, 1, 1, 1, 6]]), [[(0, t, 1)] for t in range(T)]):
+                got = run_window([q], [k], [v], [T], steps, size, page, 0.2, r1, r2, dtype, G)[0]
+                d = np.abs(got - want).max(axis=(1, 2))
+                assert d.max() <= tol * np.abs(want).max(), (tensor_cores, int(d.argmax()), d.max())
+        finally:
+            ops.set_pooled_tc(True)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_the_bias_weighs_distances_as_powers(dtype):
+    """Equal products everywhere: what is left is the bias.  A long window, so that slight and strong biases differ by far."""
+    rng, r8 = np.random.default_rng(9), stored(dtype)
+    T, H, G, dk, dv, size = 400, 4, 2, 16, 16, 300
+    q, k, v = np.zeros((T, H, dk)), np.zeros((T, G, dk)), r8(rng.normal(0, 1, (T, G, dv)))
+    v[5] *= 40.0             # a loud value far back: the tail of the weights shows
+    r1, r2 = f32([0.0, 0.02, 1.0, 2.5]), f32([0.3, 0.4, 0.1, 5.0])
+    want = plain.attend_log_bias(q, k, v, size, 1.0, r1, r2)
+    for steps in ([[(0, 0, T)]], cuts([T], [[250, 1, 1, 1, 90, 1]])):
+        got = run_window([q], [k], [v], [T], steps, size, 16, 1.0, r1, r2, dtype, G)[0]
+        for h in range(H):
+            assert np.abs(got[:, h] - want[:, h]).max() <= (2e-5 if dtype == "float32" else 2e-2) * np.abs(want[:, h]).max(), h
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_values_are_cached_divided_by_their_root_mean_square(dtype):
+    from coheryn_ai_studio_b200 import ops
+    rng, r8 = np.random.default_rng(10), stored(dtype)
+    for G, dk, dv in ((2, 16, 48), (3, 10, 7), (11, 8, 130)):
+        T = 20
+        pages = Pages([T], G, dk, dv, 8, dtype)
+        st = pages.step([(0, 0, T)])
+        proj = rng.normal(0, 1, (T, (1 * G + G) * dk + G * dv)).astype(np.float32)
+        proj[3] *= 1e-4                         # the eps inside the root counts
+        proj[4] = 0.0
+        ops.pooled_prepare(dev(proj), st.positions, None, 0, None, st.slots[0], pages.k, pages.v, G, G, dk, dv, 8, TORCH[dtype], value_eps=1e-5)
+        v = proj[:, 2 * G * dk:].astype(np.float64).reshape(T, G, dv)
+        want = plain.rms(v, 1e-5)
+        for t in range(T):
+            page, off = pages.table[0][t // 8], t % 8
+            d = np.abs(host(pages.v[page, :, off]) - want[t]).max()
+            assert d <= (1e-6 if dtype == "float32" else 4e-3) * max(1.0, np.abs(want[t]).max()), t
+            assert np.abs(host(pages.k[page, :, off]) - proj[t, G * dk:2 * G * dk].reshape(G, dk)).max() <= (0 if dtype == "float32" else 2e-2)
+
+
+MIXERS = [({"heads": 4, "kv_heads": 2, "dim": 32, "vdim": 16, "mask": {"size": 24}, "scale": 0.3}, 64, 16),
+          ({"heads": 3, "kv_heads": 3, "dim": 20, "vdim": 14, "mask": {"size": 7}, "scale": 0.4}, 100, 16),
+          ({"heads": 6, "kv_heads": 1, "dim": 16, "vdim": 48, "mask": {"size": 1}, "scale": 0.3}, 64, 8),
+          ({"heads": 2, "kv_heads": 1, "dim": 144, "vdim": 112, "mask": {"size": 50}, "scale": 0.1}, 128, 64)]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("m,width,page", MIXERS)
+def test_window_attention_mixer_in_portions_and_decoded(dtype, m, width, page):
+    """The whole mixer (projections, value norm, bias by distance, gate, output product) for two requests cut into portions."""
+    from coheryn_ai_studio_b200.parts.attention import PooledWindowAttention
+    rng, r8 = np.random.default_rng(m["dim"] + m["vdim"]), stored(dtype)
+    H, G, dk, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    W = {"m.q": r8(rng.normal(0, 0.25, (H * dk, width))), "m.k": r8(rng.normal(0, 0.25, (G * dk, width))),
+         "m.v": r8(rng.normal(0, 0.25, (G * dv, width))), "m.g": r8(rng.normal(0, 0.25, (H * dv, width))),
+         "m.o": r8(rng.normal(0, 0.25, (width, H * dv))), "m.r1": r8(rng.uniform(0.1, 2.5, H)), "m.r2": r8(rng.uniform(0.05, 0.5, H))}
+    mixer = bind(PooledWindowAttention(runtime(dtype), width, H, G, dk, dv, m["scale"], window=m["mask"]["size"], gate=True, value_eps=1e-6,
+                                       log_bias=True), W, "m.", dtype)
+    lengths = [139, 30]
+    hs = [r8(rng.normal(0, 1.0, (n, width))) for n in lengths]
+    want = [plain.log_bias_attention(h, W, "m.", m, 1e-6, rounder=r8 if dtype == "bfloat16" else same) for h in hs]
+    pages = Pages(lengths, G, dk, dv, page, dtype, window=m["mask"]["size"], seed=width)
+    steps = cuts(lengths, [[33, 2, 1, 17, 1, 1, 1, 40, 2, 1, 1, 1], [5, 1, 1, 20, 1]])
+    got = run_mixer(mixer, hs, steps, pages.step, pages.cache, dtype, width)
+    for g, w in zip(got, want):
+        tol = 3e-5 if dtype == "float32" else 4e-2
+        assert np.abs(g - w).max() <= tol * np.abs(w).max(), np.abs(g - w).max() / np.abs(w).max()
+
+
+# ------------------------------------------------------------------------------ latent attention, neighbouring pairs
+LATENTS = [({"heads": 4, "dim": 32, "rot_dim": 16, "vdim": 16, "kv_rank": 48, "scale": 0.25, "rot": {"dims": 16, "base": 1000.0}}, 64, 16),
+           ({"heads": 5, "dim": 12, "rot_dim": 6, "vdim": 10, "kv_rank": 22, "scale": 0.3, "rot": {"dims": 6, "base": 77.0}}, 100, 8),
+           ({"heads": 1, "dim": 48, "rot_dim": 64, "vdim": 80, "kv_rank": 272, "scale": 0.1, "rot": {"dims": 64, "base": 5e5}}, 128, 64),
+           ({"heads": 8, "dim": 16, "rot_dim": 32, "vdim": 32, "kv_rank": 96, "scale": 0.2, "rot": {"dims": 20, "base": 9.0}}, 64, 16)]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("m,width,page", LATENTS)
+def test_latent_attention_mixer_with_a_far_key_in_portions_and_decoded(dtype, m, width, page):
+    """The whole mixer for two requests in portions and decoded; the tokens at positions 2 and 40 share a direction with the
+    queries of the last rows (in the unrotated part), so those rows put most of their weight on keys far back; sinks from
+    far below to above the scores."""
+    from coheryn_ai_studio_b200.config.spec import PartSpec
+    from coheryn_ai_studio_b200.parts.attention import LatentAttention
+    from coheryn_ai_studio_b200.parts.base import POSITIONS, build_part
+    rng, r8 = np.random.default_rng(m["dim"] + m["kv_rank"]), stored(dtype)
+    H, dim, rd, vd, rank = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    W = {"m.q": rng.normal(0, 0.2, (H * (dim + rd), width)), "m.dkv": rng.normal(0, 0.2, (rank + rd, width)), "m.dkv.norm": rng.normal(1, 0.2, rank),
+         "m.uk": rng.normal(0, 0.3, (H * dim, rank)), "m.uv": rng.normal(0, 0.3, (H * vd, rank)), "m.o": rng.normal(0, 0.2, (width, H * vd)),
+         "m.sink": np.linspace(-8.0, 3.0, H)}
+    lengths = [311, 45]
+    hs = [rng.normal(0, 1.0, (n, width)) for n in lengths]
+    # input 0 makes latent channel 0 and input 1 the queries' component along what latent channel 0 gives every head's keys
+    W["m.dkv"][0, 0], W["m.dkv"][rank:, 0], W["m.dkv.norm"][0] = 3.0, 0.0, 1.5
+    for h in range(H):
+        u = W["m.uk"][h * dim:(h + 1) * dim, 0]
+        u[:] = np.sign(u + 1e-9) * 0.5
+        W["m.q"][h * (dim + rd):h * (dim + rd) + dim, 1] = u * (8.0 / (m["scale"] * dim))
+    hs[0][:, 0], hs[0][:, 1] = 0.0, 0.0
+    hs[0][[2, 40], 0] = 6.0
+    hs[0][-60:, 1] = 1.0
+    W, hs = {n: r8(w) for n, w in W.items()}, [r8(h) for h in hs]
+    rounder = r8 if dtype == "bfloat16" else same
+    want = [plain.latent_attention(h, W, "m.", m, 1e-6, rounder) for h in hs]
+    changed = hs[0].copy()
+    changed[2] = hs[0][3]
+    assert np.abs(plain.latent_attention(changed, W, "m.", m, 1e-6)[-60:] - want[0][-60:]).max() > 0.2 * np.abs(want[0]).max()
+    rt = runtime(dtype)
+    pos = build_part(POSITIONS, "position", PartSpec("rope_computed", dict(rotary_dim=m["rot"]["dims"], theta=m["rot"]["base"], pairs="neighbours")), rt)
+    mixer = bind(LatentAttention(rt, width, H, dim, rd, vd, rank, m["scale"], 1e-6, sink=True, position=pos), W, "m.", dtype)
+    for steps in (cuts(lengths, [[33, 2, 1, 217, 1, 1, 1, 40, 2, 1, 1, 1], [5, 1, 1, 20, 1]]), cuts(lengths, [[311], [45]])):
+        pages = Pages(lengths, 1, rank + rd, 0, page, dtype, seed=width)
+        got = run_mixer(mixer, hs, steps, pages.step, pages.cache, dtype, width)
+        for g, w in zip(got, want):
+            tol = 4e-5 if dtype == "float32" else 5e-2
+            assert np.abs(g - w).max() <= tol * np.abs(w).max(), np.abs(g - w).max() / np.abs(w).max()
+
+
+# ------------------------------------------------------------------------------ whole models
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_whole_prompts(name, dtype, folders, models):
+    for i, n in enumerate([1, 2, 23, 97]):
+        seq = sc.clear_prompt(folders[name], 30 + i, n)
+        r = sc.noisy_replay(folders[name], dtype, 128, models(name, dtype))
+        r.step([("r", seq, list(range(n)))], end=["r"])
+        sc.check_rows(r.rows, folders[name], {"r": seq}, dtype, f"whole {n}")
+
+
+def test_layer_outputs_equal_the_plain_layers(folders, models):
+    for name in NAMES:
+        seq = sc.clear_prompt(folders[name], 3, 29)
+        config, w = sc.read_model(folders[name])
+        want = []
+        plain.forward(seq, w, config, layer_outputs=want)
+        r = sc.noisy_replay(folders[name], "float32", 64, models(name, "float32"), layer_outputs=True)
+        r.step([("r", seq[:20], [19])])
+        r.step([("r", seq[20:], [8])])
+        for t in range(29):
+            got = r.layers[("r", t)]
+            assert len(got) == len(want)
+            for i in range(len(want)):
+                assert np.abs(got[i] - want[i][t]).max() <= 2e-4 * max(1.0, np.abs(want[i][t]).max()), (name, i, t)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_prompt_then_token_by_token(name, dtype, folders, models):
+    n = 120
+    seq = sc.clear_prompt(folders[name], 41, n)
+    r = sc.noisy_replay(folders[name], dtype, 128, models(name, dtype))
+    r.step([("r", seq[:n - 50], list(range(0, n - 50, 3)))])
+    for t in range(n - 50, n):
+        r.step([("r", [seq[t]], [0])])
+    sc.check_rows(r.rows, folders[name], {"r": seq}, dtype, "tail")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_every_token_decoded(name, dtype, folders, models):
+    """From the first token on, one by one (the first tokens of a sequence, then a long decode over many pages and windows
+    that give their pages back)."""
+    n = 70 if dtype == "bfloat16" else 260
+    seq = sc.clear_prompt(folders[name], 42, n)
+    r = sc.noisy_replay(folders[name], dtype, 272, models(name, dtype))
+    for t in range(n):
+        r.step([("r", [seq[t]], [0] if t < 4 or t % 4 == 0 or t > n - 5 else [])])
+    sc.check_rows(r.rows, folders[name], {"r": seq}, dtype, "decoded")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_portions_down_to_two_tokens(name, dtype, folders, models):
+    portions = [7, 2, 16, 3, 2, 33, 1, 15, 2, 17, 2, 5, 1, 1, 2, 40, 2, 70, 9]
+    n = sum(portions)
+    seq = sc.clear_prompt(folders[name], 43, n)
+    r = sc.noisy_replay(folders[name], dtype, 240, models(name, dtype), page_size=8)
+    o = 0
+    for p in portions:
+        r.step([("r", seq[o:o + p], list(range(p)))])
+        o += p
+    sc.check_rows(r.rows, folders[name], {"r": seq}, dtype, "portions")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_unequal_requests_in_one_batch_with_pages_and_slots_used_again(name, dtype, folders, models):
+    """Five requests over three state slots and a pool of 14 pages of 16: portions of some beside single tokens of others;
+    a request that ends gives its pages and its slot (with the state it left) to the next, which must not see them."""
+    seqs = {f"s{i}": sc.clear_prompt(folders[name], 50 + i, n) for i, n in enumerate([61, 9, 130, 33, 47])}
+    r = sc.noisy_replay(folders[name], dtype, 14 * 16, models(name, dtype), max_requests=3)
+    at = {k: 0 for k in seqs}
+
+    def take(rid, n):
+        toks = seqs[rid][at[rid]:at[rid] + n]
+        want = [i for i in range(len(toks)) if (at[rid] + i) % 3 == 0 or at[rid] + i == len(seqs[rid]) - 1]
+        at[rid] += len(toks)
+        return (rid, toks, want)
+
+    def done(*rids):
+        return [x for x in rids if at[x] == len(seqs[x])]
+
+    r.step([take("s0", 20), take("s1", 2)])
+    r.step([take("s0", 1), take("s1", 1), take("s2", 50)])
+    r.step([take("s0", 40), take("s1", 6), take("s2", 1)], end=["s0", "s1"])
+    r.step([take("s2", 1), take("s3", 33)], end=["s3"])
+    r.step([take("s4", 2), take("s2", 30)])
+    while at["s2"] < 130 or at["s4"] < 47:
+        batch = [take(x, 1 if x == "s2" else 5) for x in ("s2", "s4") if at[x] < len(seqs[x])]
+        r.step(batch, end=done(*[b[0] for b in batch]))
+    assert all(at[k] == len(seqs[k]) for k in seqs)
+    sc.check_rows(r.rows, folders[name], seqs, dtype, "mixed")
+    assert len(r.cache.requests) == 0 and r.cache.available_pages() == [14] * len(r.cache.groups)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["S1", "S3"])
+def test_batched_rows_equal_the_rows_of_each_request_alone(name, dtype, folders, models):
+    """What a request's rows are does not depend on what else is in the batch, nor on pages and slots, beyond rounding."""
+    a, b = sc.clear_prompt(folders[name], 60, 45), sc.clear_prompt(folders[name], 61, 18)
+    alone = sc.noisy_replay(folders[name], dtype, 128, models(name, dtype))
+    alone.step([("a", a[:30], list(range(30)))])
+    alone.step([("a", a[30:], list(range(15)))])
+    both = sc.noisy_replay(folders[name], dtype, 128, models(name, dtype))
+    both.step([("b", b[:10], [9]), ("a", a[:30], list(range(30)))])
+    both.step([("a", a[30:], list(range(15))), ("b", b[10:], [7])])
+    far = [p for p in range(45) if np.abs(alone.rows[("a", p)] - both.rows[("a", p)]).max()
+           > (1e-4 if dtype == "float32" else 0.05) * np.std(alone.rows[("a", p)])]
+    # in bfloat16 other product kernels (by row count) can turn a router's near tie
+    assert len(far) <= (0 if dtype == "float32" else 3), far
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_few_wanted_rows_take_the_last_layers_shortcut(name, dtype, folders, models):
+    """Steps that want few rows (or none) run the last layer behind its cache or state for those rows only (S1: a window
+    attention; S2: a latent attention without feed-forward; S3: a recurrence), the average over depth included: the logits
+    equal the plain implementation's, and switching the shortcut off changes nothing beyond rounding."""
+    n = 131
+    seq, other = sc.clear_prompt(folders[name], 33, n), sc.clear_prompt(folders[name], 34, 40)
+    runs = {}
+    for shortcut in (True, False):
+        r = sc.noisy_replay(folders[name], dtype, 256, models(name, dtype))
+        r.runner.tail_shortcut = shortcut
+        r.step([("r", seq[:30], [])])
+        r.step([("r", seq[30:60], [29, 3]), ("o", other[:20], [19])])
+        r.step([("r", seq[60:n - 5], [0]), ("o", other[20:], [])])
+        r.step([("r", seq[n - 5:], list(range(5)))])
+        assert set(k for k in r.rows if k[0] == "r") == {("r", p) for p in [59, 33, 60] + list(range(n - 5, n))}
+        sc.check_rows(r.rows, folders[name], {"r": seq, "o": other}, dtype, f"shortcut {shortcut}")
+        runs[shortcut] = r.rows
+    assert models(name, dtype).layers[-1].supports_tail
+    near = [np.abs(row - runs[False][key]).max() <= (2e-4 * max(1.0, np.std(row)) if dtype == "float32" else 0.08 * np.std(row))
+            for key, row in runs[True].items()]
+    assert all(near) if dtype == "float32" else np.mean(near) > 0.7
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_long_prompts_and_their_expanded_latents(dtype, tmp_path):
+    """A prompt of 600 tokens at once (latent rows expanded per head in bfloat16), then portions behind it and decoded tokens."""
+    from coheryn_ai_studio_b200.engine import load_model
+    cfg = sc._config(200, 64, 700, 1e-6, 0.5, [
+        sc._latent(2, 16, 16, 16, 112, 300.0, 0.25, mlp=sc._dense(64)), sc._gla(2, 16, 16, 4.0, 8, mlp=None),
+        sc._window(2, 1, 16, 16, 100, 0.3, mlp=None), sc._latent(2, 32, 16, 32, 96, 10000.0, 0.2, mlp=sc._moe(32, 4, 2, groups=(2, 1), shared=16))])
+    folder = sc.make_folder(tmp_path, "long", cfg, 71)
+    model = load_model(folder, dtype)[1]
+    seq = sc.clear_prompt(folder, 90, 660)
+    r = sc.noisy_replay(folder, dtype, 768, model)
+    r.step([("r", seq[:600], list(range(0, 600, 23)) + [599])])
+    r.step([("r", seq[600:640], [0, 1, 20, 39])])
+    for t in range(640, 660):
+        r.step([("r", [seq[t]], [0])])
+    sc.check_rows(r.rows, folder, {"r": seq}, dtype, "long")
+
+
+def test_tensor_core_attention_equals_the_float32_arithmetic_one_in_a_model(folders, models):
+    """The same bfloat16 steps with the tensor-core attentions switched off: rows agree within rounding."""
+    from coheryn_ai_studio_b200 import ops
+    for name in ("S1", "S3"):
+        seq, other = sc.clear_prompt(folders[name], 62, 150), sc.clear_prompt(folders[name], 63, 70)
+        rows = {}
+        for on in (True, False):
+            ops.set_pooled_tc(on)
+            ops.set_maps_tc(on)
+            try:
+                r = sc.noisy_replay(folders[name], "bfloat16", 256, models(name, "bfloat16"))
+                r.step([("r", seq[:91], list(range(0, 91, 2)))])
+                r.step([("r", seq[91:140], list(range(0, 49, 3))), ("o", other, [69, 5])])
+                for t in range(140, 150):
+                    r.step([("r", [seq[t]], [0])])
+                rows[on] = r.rows
+            finally:
+                ops.set_pooled_tc(True)
+                ops.set_maps_tc(True)
+        sc.check_rows(rows[True], folders[name], {"r": seq, "o": other}, "bfloat16", "tensor cores")
+        near = [np.abs(rows[True][k] - rows[False][k]).max() <= 0.06 * np.std(rows[False][k]) for k in rows[True]]
+        assert np.mean(near) > 0.85          # a router's near tie may fall the other way at single rows
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["S1", "S3"])
+def test_greedy_generation_through_the_engine(name, dtype, folders):
+    """The Python entry point with its scheduler, continuous batching, portions of 16 tokens and decode steps replayed
+    from CUDA graphs: every generated token is the plain implementation's first maximum given the tokens before it (in
+    bfloat16: or a near tie)."""
+    from coheryn_ai_studio_b200.engine import Engine
+    eng = Engine.from_folder(folders[name], dtype, context=128, max_num_seqs=3, max_num_batched_tokens=16, page_size=8)
+    prompts = [sc.clear_prompt(folders[name], 70 + i, n) for i, n in enumerate((3, 29, 50, 1))]
+    res = eng.generate(prompts, max_tokens=12)
+    for p, out in zip(prompts, res):
+        ids = list(p)
+        assert out.completion_tokens == 12 and out.finish_reason == "length"
+        for tok in out.token_ids:
+            ref = sc.plain_rows(folders[name], ids)[-1]
+            best = int(np.argmax(ref))
+            if tok != best:
+                gap = float(ref[best] - ref[tok]) / float(np.std(ref))
+                assert gap <= (1e-3 if dtype == "float32" else 0.4) or (dtype == "bfloat16" and not sc.clear_rows(folders[name], ids)[-1]), \
+                    (name, len(ids), tok, best, gap)
+            ids.append(tok)
+    eng.cache.check()
+    assert len(eng.cache.requests) == 0
+
+
+def test_positions_end_where_the_position_table_ends(folders, models):
+    name = "S2"
+    seq = sc.clear_prompt(folders[name], 75, 290)
+    r = sc.noisy_replay(folders[name], "float32", 304, models(name, "float32"))
+    r.step([("r", seq[:288], [287])])
+    r.step([("r", seq[288:], [0, 1])])                      # the table's last row
+    sc.check_rows(r.rows, folders[name], {"r": seq}, "float32", "last position")
+    with pytest.raises(ValueError):
+        r.step([("r", [1], [0])])
+
+
+def test_trace_program_replays_a_schedule(folders, tmp_path):
+    """bin/trace_run on a folder of this design: portions, a second request, an ended request, a step that wants nothing."""
+    import json, os, subprocess, sys
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    name = "S2"
+    a, b = sc.clear_prompt(folders[name], 80, 40), sc.clear_prompt(folders[name], 81, 12)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:25], "want": [0, 24]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": a[25:27], "want": []}, {"id": "b", "tokens": b, "want": [11]}], "end": ["b"]},
+             {"step": 2, "entries": [{"id": "a", "tokens": a[27:], "want": [12]}], "end": ["a"]}]
+    out = tmp_path / "out"
+    p = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", folders[name], "--dtype", "float32",
+                        "--out", str(out), "--max-tokens", "128"], input="\n".join(json.dumps(s) for s in steps) + "\n",
+                       capture_output=True, text=True, timeout=900)
+    assert p.returncode == 0, p.stderr[-2000:]
+    assert [l for l in p.stdout.splitlines() if l.startswith("done")] == ["done 0", "done 1", "done 2"]
+    V = vocab(name)
+    got0 = np.fromfile(out / "0.f32", dtype="<f4").reshape(2, V)
+    got1 = np.fromfile(out / "1.f32", dtype="<f4").reshape(1, V)
+    got2 = np.fromfile(out / "2.f32", dtype="<f4").reshape(1, V)
+    rows = {("a", 0): got0[0], ("a", 24): got0[1], ("b", 11): got1[0], ("a", 39): got2[0]}
+    sc.check_rows(rows, folders[name], {"a": a, "b": b}, "float32", "trace")
+
+
+def test_command_line_runs_and_inspects_the_design(folders):
+    import os, subprocess, sys
+    from coheryn_ai_studio_b200 import api
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    name = "S1"
+    p = sc.clear_prompt(folders[name], 85, 27)
+    r = subprocess.run([sys.executable, os.path.join(root, "bin", "coheryn"), "run", folders[name], "--tokens", ",".join(map(str, p)),
+                        "--max-tokens", "5", "--context", "64", "--dtype", "float32", "--stream"], capture_output=True, text=True, timeout=900)
+    assert r.returncode == 0, r.stderr[-2000:]
+    got = [int(t) for t in r.stdout.split()]
+    ids = list(p)
+    for tok in got:
+        assert tok == int(np.argmax(sc.plain_rows(folders[name], ids)[-1]))
+        ids.append(tok)
+    assert api.generate(folders[name], [p], max_tokens=5, context=64, dtype="float32")[0]["token_ids"] == got
+    r = subprocess.run([sys.executable, os.path.join(root, "bin", "coheryn"), "models", "inspect", folders[name]], capture_output=True,
+                       text=True, timeout=900)
+    assert r.returncode == 0 and "Zusotar" in r.stdout, r.stderr[-2000:]
+
+
+def test_zz_report():
+    print(f"\nZusotar rows against the plain implementation: float32 largest |d| = {sc.WORST['float32']:.2e} of the spread; "
+          f"bfloat16 largest median distance = {sc.WORST['bfloat16']:.2f} of the bound")
