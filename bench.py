@@ -29,7 +29,9 @@ decode through the step function, and the mixers' kernels alone.  ``--workload t
 design (differential attention over chunks, attention with a sink beside a gated delta rule, norms before and after each
 sub-layer), its kernels beside the like kernels of the other models.  ``--workload zegelix`` does the same for the Zegelix
 design (gated linear recurrences, window attention over positions and block means, routed experts with a shared expert, a
-repeated span of layers).  ``--workload guvusun`` does the same for the Guvusun
+repeated span of layers).  ``--workload zusotar`` does the same for the Zusotar design (latent attention, gated linear
+attention, window attention with a logarithmic bias by distance, routed experts, an average over depth behind every layer)
+beside Guvusun at equal sizes and Qwen2.  ``--workload guvusun`` does the same for the Guvusun
 design (latent attention with a learned sink and head gates, routed experts, norms after the sum) beside Qwen2 with a dense
 feed-forward of the experts' active size.
 """
@@ -960,6 +962,183 @@ def zegelix_workload(args) -> int:
     return 0
 
 
+# Sizes of --workload zusotar: linear attention, latent attention and window attention in the proportion 1 : 2 : 1, a dense
+# feed-forward in the first layer and routed experts with a shared one in the others.  Beside each the closest other design,
+# Guvusun: as many layers of the same latent attention and the same routed experts at equal width; and Qwen2 with a dense
+# feed-forward of (top + shared) rows and the window attention's heads.
+ZUSOTAR_SIZES = {
+    "w2048": dict(width=2048, vocab=32000, layers="glwlglwl", gla=(8, 128, 256, 16), latent=(16, 96, 32, 128, 224), window=(16, 4, 128, 1024),
+                  experts=32, top=4, groups=(4, 2), ff=1024, shared=1024, dense=5120),
+    "w4096": dict(width=4096, vocab=32000, layers="glwl", gla=(16, 128, 256, 32), latent=(32, 128, 64, 128, 512), window=(32, 8, 128, 2048),
+                  experts=64, top=6, groups=(8, 4), ff=1408, shared=2816, dense=11264),
+}
+
+
+def zusotar_config(z, positions):
+    H, dk, dv, rank = z["gla"]
+    gla = {"type": "gla", "mixer": {"heads": H, "dim": dk, "vdim": dv, "tau": 16.0, "a_rank": rank}}
+    H, dim, rd, vd, r = z["latent"]
+    latent = {"type": "latent_attention", "mixer": {"heads": H, "dim": dim, "rot_dim": rd, "vdim": vd, "kv_rank": r, "scale": (dim + rd) ** -0.5,
+                                                    "rot": {"base": 500000.0, "dims": rd}}}
+    H, G, d, size = z["window"]
+    window = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": size}}}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"]}, "shared": {"ff": z["shared"]},
+           "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": z["groups"][0], "keep": z["groups"][1]}}}
+    kinds = {"g": gla, "l": latent, "w": window}
+    return {"architecture": "Zusotar", "vocab": z["vocab"], "width": z["width"], "max_positions": positions, "norm": {"eps": 1e-6},
+            "residual_mult": 0.5, "layers": [dict(kinds[c], mlp=moe if i else {"kind": "dense", "ff": z["dense"]})
+                                             for i, c in enumerate(z["layers"])]}
+
+
+def zusotar_workload(args) -> int:
+    """Prefill and decode throughput of Zusotar, of Guvusun and of Qwen2 at equal sizes through the step function, and the
+    design's own kernels alone beside the like kernels of the other models, each with its share of the roofline.  One JSON
+    line."""
+    import torch
+
+    from coheryn_ai_studio_b200 import ops
+    from coheryn_ai_studio_b200.config import Qwen2Config
+    from coheryn_ai_studio_b200.config.guvusun import GuvusunConfig
+    from coheryn_ai_studio_b200.config.zusotar import ZusotarConfig
+    from coheryn_ai_studio_b200.engine import random_model_on_device
+
+    tools = model_bench_tools(args)
+    pk, hbm, flops_peak, dev = tools.pk, tools.hbm, tools.flops_peak, tools.dev
+    tokens, batch, context = tools.tokens, tools.batch, tools.context
+    timed, step_like = tools.timed, tools.step_like
+    fma_peak = 148 * 128 * 2 * 1.965e9        # float32 FMA lanes x 2 x the SM clock: what float32 arithmetic is bound by
+
+    def kernels(z):
+        out = {}
+        W, page = z["width"], args.page_size
+        f = lambda *shape: torch.randn(shape, device=dev)
+        b16 = lambda *shape: f(*shape).to(torch.bfloat16)
+        for name, lengths, starts in (("prefill", [tokens], [0]), ("decode", [1] * batch, [context] * batch)):
+            B, T = len(lengths), sum(lengths)
+            per = -(-max(s + n for s, n in zip(starts, lengths)) // page)
+            tables = torch.arange(B * per, dtype=torch.int32, device=dev).view(B, per)
+            st = step_like(lengths, starts, tables)
+            st.block_tables, st.max_q_len = [tables, tables], max(lengths)
+            st.slots = [(tables[st.token_req.long(), (st.positions // page).long()] * page + st.positions % page).to(torch.int32)]
+            seen = sum(p + 1 for s, n in zip(starts, lengths) for p in range(s, s + n))
+            held = sum(s + n for s, n in zip(starts, lengths))
+
+            def record(label, fn, by=None, flops=None, peak=None, peak_name="of_bf16_peak"):
+                ms = timed(fn)
+                e = out[f"{name}.{label}"] = {"ms": round(ms, 4)}
+                if by is not None:
+                    e["of_hbm"] = round(by / (ms / 1e3) / hbm, 4)
+                if flops is not None:
+                    e["tflops"] = round(flops / ms / 1e9, 1)
+                    e[peak_name] = round(flops / (ms / 1e3) / peak, 4)
+
+            # gated linear attention, and the delta rule with a decay per key channel at the same heads
+            H, dk, dv, rank = z["gla"]
+            wide = f(T, 2 * H * (dk + dv))       # one projection, as the mixers have it
+            q, k, v, g = wide.split([H * dk, H * dk, H * dv, H * dv], dim=1)
+            a1 = f(T, rank)
+            a2, a2b, nw = b16(H * dk, rank), f(H * dk), f(dv)
+            state = torch.zeros((B, H * dk * dv), dtype=torch.float32, device=dev)
+            o = torch.empty((T, H * dv), dtype=torch.bfloat16, device=dev)
+            state_bytes = 8.0 * B * H * dk * dv
+            # what the recurrence itself needs per token and head: the state's update and its product with the query
+            record("gated_linear_attention", lambda: ops.gated_linear_attention(
+                q, k, v, g, a1, a2, a2b, 16.0, dk ** -0.5, state, st, H, dk, dv, nw, 1e-6, o),
+                by=state_bytes + T * H * (8.0 * dk + 10.0 * dv), flops=4.0 * T * H * dk * dv, peak=fma_peak, peak_name="of_fma_peak")
+            if dk <= 256 and dv <= 256:
+                beta, sp, rl, sb = f(T, H), f(T, H * dk), f(H), f(H * dk)
+                record("delta_rule_decay_per_channel", lambda: ops.gated_delta_scan(
+                    q, k, v, beta, sp, sb, rl, state, st, H, H, dk, dv, o, nw, g, 1e-6, 1.0, decay_per_channel=True, gate_activation="silu"),
+                    by=state_bytes + T * H * (12.0 * dk + 10.0 * dv), flops=8.0 * T * H * dk * dv, peak=fma_peak, peak_name="of_fma_peak")
+            # window attention with the logarithmic bias; with blocks, cap, rotated values and sink (Zegelix); Qwen2's
+            H, G, d, size = z["window"]
+            met = sum(min(p + 1, size) for s, n in zip(starts, lengths) for p in range(s, s + n))
+            rows_read = sum(min(s + n, size + n) for s, n in zip(starts, lengths))
+            io = 4.0 * d * G * rows_read + 4.0 * T * H * d
+            kc, vc = b16(B * per + 1, G, page, d), b16(B * per + 1, G, page, d)
+            qa, oa = b16(T, H * d), torch.empty((T, H * d), dtype=torch.bfloat16, device=dev)
+            gates, r1, r2 = f(T, H * d), f(H).abs(), f(H).abs()
+            record("window_attention_log_bias", lambda: ops.pooled_attention(
+                qa, oa, kc, vc, None, None, st, 0, None, H, G, d, d, page, size, None, d ** -0.5, None, None, None, gates, None,
+                log_bias=(r1, r2)), by=io, flops=4.0 * H * d * met, peak=flops_peak)
+            fv = torch.stack([torch.pow(torch.tensor(10000.0), -2.0 * torch.arange(d // 2) / d), torch.zeros(d // 2)], dim=1).to(dev).contiguous()
+            temps, sinks = f(H).abs() + 0.5, f(H)
+            record("zegelix_window_attention_cap_and_turned_values", lambda: ops.pooled_attention(
+                qa, oa, kc, vc, None, None, st, 0, None, H, G, d, d, page, size, None, d ** -0.5, 50.0, temps, sinks, gates, fv),
+                by=io, flops=4.0 * H * d * met, peak=flops_peak)
+            record("qwen2_attention_same_window", lambda: ops.attention_rows(
+                qa, oa, kc, vc, tables, st.token_req, st.positions, H, G, d, page, size, d ** -0.5, cu_q=st.cu_q, kv_lens=st.kv_lens,
+                q_lens=st.q_lens, max_kv_len=st.max_kv_len), by=io, flops=4.0 * H * d * met, peak=flops_peak)
+            proj = f(T, (H + 2 * G) * d + H * d)
+            record("value_norm_and_cache_write", lambda: ops.pooled_prepare(
+                proj, st.positions, None, 0, None, st.slots[0], kc, vc, H, G, d, d, page, torch.bfloat16, value_eps=1e-6), by=T * (H + 2 * G) * d * 6.0)
+            record("zegelix_rotate_and_cache_write", lambda: ops.pooled_prepare(
+                proj, st.positions, fv, d, fv, st.slots[0], kc, vc, H, G, d, d, page, torch.bfloat16), by=T * (H + 2 * G) * d * 6.0)
+            # latent attention (Guvusun's kernels; without gates here): over the latent rows, and expanded per head for whole prompts
+            H, dim, rd, vd, rank = z["latent"]
+            row, hd = rank + rd, dim + rd
+            kl, ql, ol, sk = b16(B * per + 1, 1, page, row), b16(T, H * row), torch.empty((T, H * rank), dtype=torch.bfloat16, device=dev), f(H)
+            record("latent_attention_sink", lambda: ops.attention_maps(
+                ql, ol, kl, None, st, 0, H, 1, row, rank, 1, page, None, None, True, hd ** -0.5, 0.0, False, 1e-6, 1.0, sink_scores=sk,
+                values_in_keys=True), by=2.0 * row * held + 2.0 * T * H * (row + rank), flops=2.0 * H * (row + rank) * seen, peak=flops_peak)
+            # the average over depth with the add in front of it and the norm behind it, early and late in the stack
+            x, y, w1, w2 = f(T, W), f(T, W), f(W), f(W)
+            h = torch.empty((T, W), dtype=torch.bfloat16, device=dev)
+            hist = f(len(z["layers"]) + 1, T, W)
+            for n in (1, len(z["layers"])):
+                avg = f(n + 1)
+                record(f"average_over_{n}_earlier_results_add_and_norm", lambda: ops.depth_average_norm(x, y, w1, hist, avg, n, w2, 1e-6, h),
+                       by=T * W * (4.0 * n + 4 + 4 + 4 + 4 + 2))
+            record("tutunex_add_of_a_normalised_summand_and_norm", lambda: ops.add_normed_rmsnorm(x, y, None, 1.0, w1, w2, 1e-6, h), by=T * W * 14.0)
+            # embedding rows with positions; the router
+            table, pos = b16(z["vocab"], W), b16(context + tokens + 64, W)
+            ids, status = torch.randint(0, z["vocab"], (T,), dtype=torch.int32, device=dev), torch.zeros(1, dtype=torch.int32, device=dev)
+            record("embedding_with_positions_written_twice", lambda: ops.embed_gather(table, ids, x, status, pos_table=pos, positions=st.positions, copy=y),
+                   by=T * W * 12.0)
+            record("qwen2_embedding", lambda: ops.embed_gather(table, ids, x, status), by=T * W * 6.0)
+            logits = f(T, z["experts"])
+            record("router_sigmoid_groups_of_two", lambda: ops.route_select(
+                logits, None, z["groups"][0], z["groups"][1], z["top"], 1.0, scores="sigmoid", group_score="two", renormalize=False),
+                by=T * (z["experts"] * 4.0 + z["top"] * 8.0))
+            corr = f(z["experts"]) * 0.01
+            record("guvusun_router", lambda: ops.route_select(logits, corr, z["groups"][0], z["groups"][1], z["top"], 2.5),
+                   by=T * (z["experts"] * 4.0 + z["top"] * 8.0))
+        return out
+
+    sampler = ClockSampler()
+    sampler.start()
+    t0 = time.time()
+    results = {}
+    for name in [n for n in ZUSOTAR_SIZES if not args.sizes or n in args.sizes.split(",")]:
+        z = ZUSOTAR_SIZES[name]
+        entry = {}
+
+        def run(label, config):
+            model = random_model_on_device(config, seed=0, dtype="bfloat16", device="cuda:0")
+            entry[label] = tools.run_model(model, z["vocab"])
+            del model
+            torch.cuda.empty_cache()
+        run("zusotar", ZusotarConfig.from_dict(zusotar_config(z, max(context, tokens) + 1024)))
+        H, dim, rd, vd, r = z["latent"]
+        run("guvusun_equal_size", GuvusunConfig.from_dict(guvusun_config(dict(
+            width=z["width"], vocab=z["vocab"], layers=len(z["layers"]), heads=H, dim=dim, rot_dim=rd, vdim=vd, kv_rank=r, experts=z["experts"],
+            identity=0, top=z["top"], groups=z["groups"], ff=z["ff"], side_dim=64, buckets=100003))))
+        H, G, d, _ = z["window"]
+        run("qwen2_equal_size", Qwen2Config(
+            vocab_size=z["vocab"], hidden_size=z["width"], intermediate_size=z["top"] * z["ff"] + z["shared"], num_hidden_layers=len(z["layers"]),
+            num_attention_heads=H, num_key_value_heads=G, head_dim=d, max_position_embeddings=32768, rms_norm_eps=1e-6, rope_theta=1e6,
+            tie_word_embeddings=False))
+        if not args.no_kernels:
+            entry["kernels"] = kernels(z)
+        results[name] = entry
+    clocks = ClockSampler.summary(sampler.window(t0, time.time()))
+    sampler.stop()
+    print(json.dumps({"workload": "zusotar", "dtype": "bf16", "data": "synthetic", "prefill_tokens": tokens, "decode_batch": batch,
+                      "decode_context": context, "decode_steps": tools.steps, "peaks": pk, "clocks": clocks,
+                      "l2": "flushed before each timed kernel", "gpu_launches": ops.total_launch_count(), "sizes": results}))
+    return 0
+
+
 def timeline(args, make_engine, StepEntry, ops, torch) -> int:
     """Where a decode step's time goes, kernel by kernel, measured inside graph-replayed steps (the
     kernels overlap through programmatic dependent launch, so a kernel's own duration says little):
@@ -1027,10 +1206,10 @@ def main() -> int:
     ap.add_argument("--page-size", type=int, default=16)
     ap.add_argument("--skip-points", action="store_true", help="skip the batch 1 / 64 points")
     ap.add_argument("--no-graphs", action="store_true")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serving-7b", "long-14b", "chat-1.5b", "kapudra", "tutunex", "guvusun", "zegelix"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "serving-7b", "long-14b", "chat-1.5b", "kapudra", "tutunex", "guvusun", "zegelix", "zusotar"],
                     help="decode: the contract's line (default); the others: see the header")
-    ap.add_argument("--sizes", default="", help="--workload kapudra / tutunex / guvusun / zegelix: which of its sizes (comma separated; default all)")
-    ap.add_argument("--no-kernels", action="store_true", help="--workload guvusun / zegelix: the models only, not the kernels alone")
+    ap.add_argument("--sizes", default="", help="--workload kapudra / tutunex / guvusun / zegelix / zusotar: which of its sizes (comma separated; default all)")
+    ap.add_argument("--no-kernels", action="store_true", help="--workload guvusun / zegelix / zusotar: the models only, not the kernels alone")
     ap.add_argument("--timeline-raw", action="store_true", help="with --timeline: also every kernel's start and end")
     ap.add_argument("--timeline", action="store_true",
                     help="instead of the benchmark: the kernels of one graph-replayed decode step with their times "
@@ -1055,6 +1234,8 @@ def main() -> int:
         return guvusun_workload(args)
     if args.workload == "zegelix":
         return zegelix_workload(args)
+    if args.workload == "zusotar":
+        return zusotar_workload(args)
     if args.workload != "decode":
         return other_workload(args)
 
