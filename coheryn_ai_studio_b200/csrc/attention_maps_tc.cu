@@ -12,8 +12,8 @@
 // w = e_0 / l_0 - lambda e_1 / l_1 in float32 and accumulates w V once.  No accumulator is ever rescaled, two maps
 // cost one accumulator, and the difference of the maps is taken before anything is rounded.
 //
-// Decoding (`maps_decode_kernel` + `maps_combine_kernel`): the rows of a tile are the query heads of ONE key/value
-// head for one token, the visible keys are cut into at most sixteen splits at absolute multiples of the split size,
+// Decoding (`maps_decode_kernel` + `maps_combine_kernel`): the rows of a tile are (up to sixteen of) the query heads of
+// ONE key/value head for one token, the visible keys are cut into at most sixteen splits at absolute multiples of the split size,
 // each of a CTA's four warps takes a quarter of a split (an online softmax over its tiles, one map after the other)
 // and leaves (maximum, sum, unnormalised output) per head and map; a second kernel merges the parts in order, adds
 // the sink, takes the difference of the maps, normalises and writes.
@@ -390,21 +390,24 @@ __global__ void __launch_bounds__(WARPS * 32, CO_MAPS_MIN_CTAS) maps_tiles_kerne
 }
 
 // ---------------------------------------------------------------------------------
-// Decoding: requests that bring ONE token.  grid: (requests, kv heads, splits).  A part = (split, warp).
+// Decoding: requests that bring ONE token.  grid: (requests, kv heads * blocks of sixteen query heads, splits).  A part =
+// (split, warp).
 // scratch: [request][query head][map][splits * WARPS parts][DV + 2] = (output[DV], maximum, sum).
 // ---------------------------------------------------------------------------------
 __global__ void __launch_bounds__(WARPS * 32) maps_decode_kernel(MapsArgs A, float* __restrict__ scratch, int split_keys, int n_splits) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
-  bf16* qs = reinterpret_cast<bf16*>(smem_raw);        // [16][KS]: the query heads of the kv head, then zero rows
+  bf16* qs = reinterpret_cast<bf16*>(smem_raw);        // [16][KS]: the CTA's query heads, then zero rows
   bf16* kall = qs + 16 * KS;                           // [WARPS][BN][KS]
   bf16* vall = kall + WARPS * BN * KS;                 // [WARPS][BN][VS]
   co_pdl_launch_dependents();
   co_pdl_wait();
-  const int r = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z;
+  const int per_kv = A.nh / A.nkv, blocks = (per_kv + 15) / 16;
+  const int r = blockIdx.x, kvh = blockIdx.y / blocks, split = blockIdx.z;
   const int q0 = A.cu_q[r], q_len = A.cu_q[r + 1] - q0;
   if (q_len != 1) return;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int group = A.nh / A.nkv;
+  const int first_head = kvh * per_kv + (blockIdx.y % blocks) * 16;      // the CTA's query heads: this one and the next ones
+  const int group = min(16, (kvh + 1) * per_kv - first_head);
   const int p = A.kv_lens[r] - 1, f = first_visible(p, A.window, A.chunk);
   const int key_lo = (f / split_keys + split) * split_keys;      // splits at absolute multiples of their size
   if (key_lo > p) return;                                         // the combine kernel knows which splits exist
@@ -412,7 +415,7 @@ __global__ void __launch_bounds__(WARPS * 32) maps_decode_kernel(MapsArgs A, flo
   for (int c = tid; c < 16 * (KROW / 8); c += WARPS * 32) {
     const int row = c / (KROW / 8), ch = c % (KROW / 8);
     const bool ok = row < group;
-    cp_async16(qs + row * KS + ch * 8, A.q + (size_t)q0 * A.ldq + (size_t)(kvh * group + (ok ? row : 0)) * KROW + ch * 8, ok ? 16 : 0);
+    cp_async16(qs + row * KS + ch * 8, A.q + (size_t)q0 * A.ldq + (size_t)(first_head + (ok ? row : 0)) * KROW + ch * 8, ok ? 16 : 0);
   }
   cp_commit();
   bf16* kw = kall + warp * BN * KS;
@@ -470,7 +473,7 @@ __global__ void __launch_bounds__(WARPS * 32) maps_decode_kernel(MapsArgs A, flo
       const int row = (lane >> 2) + 8 * rr;
       const float l = quad_sum(sum[rr]);
       if (row < group) {
-        float* part = scratch + ((((size_t)r * A.nh + kvh * group + row) * MAPS + m) * (n_splits * WARPS) + split * WARPS + warp) * (DV + 2);
+        float* part = scratch + ((((size_t)r * A.nh + first_head + row) * MAPS + m) * (n_splits * WARPS) + split * WARPS + warp) * (DV + 2);
 #pragma unroll
         for (int nt = 0; nt < OT; ++nt) {
           part[vc * DVC + nt * 8 + 2 * (lane & 3)] = o[nt][2 * rr];
@@ -589,8 +592,8 @@ CO_EXPORT int coheryn_attention_maps_bf16(const void* q, long ldq, void* out, lo
   if ((ldq & 7) || (ldo & 1) || ((uintptr_t)q & 15) || ((uintptr_t)out & 3) || ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15))
     CO_FAIL("attention_maps_bf16: rows of q must start on 16-byte boundaries, rows of out on 4-byte ones");
   if (head_norm && NCH > 1) CO_FAIL("attention_maps_bf16: a normalised output needs values of at most 256 channels (%d)", DV);
-  const int group = nh / nkv;
-  const bool decode = any_single && group <= 16;
+  const int blocks = (nh / nkv + 15) / 16;             // of query heads per kv head
+  const bool decode = any_single != 0;
   MapsArgs A{(const bf16*)q, ldq, (bf16*)out, ldo, (const bf16*)k_cache, (const bf16*)v_cache, block_tables, max_blocks, cu_q,
              kv_lens, nh, nkv, page_size, window, chunk, sink, head_norm, decode ? 1 : 0, 0,
              scale * 1.4426950408889634f, lambda, eps, out_scale, sink_scores, gates, gates_ld};
@@ -612,7 +615,7 @@ CO_EXPORT int coheryn_attention_maps_bf16(const void* q, long ldq, void* out, lo
     decode_plan(max_kv_len, window, chunk, &split_keys, &n_splits);
     const size_t smem = ((size_t)16 * KS + (size_t)WARPS * BN * (KS + VROW)) * sizeof(bf16);
     if (smem > 48 * 1024) cudaFuncSetAttribute(maps_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    co_launch(maps_decode_kernel, dim3(B, nkv, n_splits), dim3(WARPS * 32), smem, stream, A, scratch, split_keys, n_splits);
+    co_launch(maps_decode_kernel, dim3(B, nkv * blocks, n_splits), dim3(WARPS * 32), smem, stream, A, scratch, split_keys, n_splits);
     CO_CHECK_LAUNCH("maps_decode");
     co_launch(maps_combine_kernel, dim3(B, nh), dim3(DV >= 128 ? 128 : (DV > 32 ? (DV + 31) / 32 * 32 : 64)), 0, stream, A, (const float*)scratch, split_keys, n_splits);
     CO_CHECK_LAUNCH("maps_combine");

@@ -68,7 +68,7 @@ __global__ void pooled_prepare_kernel(const float* __restrict__ proj, long ld, c
       if (lane == 0) v_mult[g] = 1.0f / sqrtf(ss / (float)dv + v_eps);
     }
   }
-  __syncthreads();
+  if (hk) __syncthreads();       // without a rotation queries and keys need not wait for the values' sums
   size_t k_at = 0, v_at = 0;
   if (slots) {
     const int slot = slots[t];
@@ -92,6 +92,7 @@ __global__ void pooled_prepare_kernel(const float* __restrict__ proj, long ld, c
     }
   }
   if (!slots) return;
+  __syncthreads();
   const int per_v = dv - hv;
   const float* vrow = row + (size_t)(H + G) * dk;
   for (int e = threadIdx.x; e < G * per_v; e += blockDim.x) {

@@ -233,20 +233,23 @@ __global__ void __launch_bounds__(256) gla_chunk_state_kernel(GlaArgs A, bool ve
   const int h = blockIdx.z / (nk * nv), kt = (blockIdx.z / nv) % nk, vt = blockIdx.z % nv;
   const int d0 = kt * 64, c0 = vt * VT;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  for (int e = threadIdx.x; e < CH * 64; e += 256) {
-    const int t = e >> 6, d = e & 63;
+#pragma unroll 8
+  for (int i = 0; i < CH * 64 / 256; ++i) {
+    const int e = threadIdx.x + 256 * i, t = e >> 6, d = e & 63;
     const bool in = t < ck.n && d0 + d < dk;
     const size_t ch = (size_t)h * dk + d0 + d, row = (size_t)ck.first + t;
     Ks[t * TP + d] = in ? A.k[row * A.ldk + ch] : 0.f;
     Ls[d * SP + t] = in ? A.log_decay[row * ((size_t)A.H * dk) + ch] : 0.f;
   }
-  for (int e = threadIdx.x; e < CH * (VT / 4); e += 256) {
-    const int t = e / (VT / 4), c4 = e % (VT / 4);
+#pragma unroll
+  for (int i = 0; i < CH * (VT / 4) / 256; ++i) {
+    const int e = threadIdx.x + 256 * i, t = e / (VT / 4), c4 = e % (VT / 4);
     const float4 x = t < ck.n ? gla_load4(A.v + ((size_t)ck.first + t) * A.ldv + (size_t)h * dv, c0 + 4 * c4, dv, vec)
                               : make_float4(0.f, 0.f, 0.f, 0.f);
     *reinterpret_cast<float4*>(Vs + t * VT + 4 * c4) = x;
   }
   __syncthreads();
+#pragma unroll 4
   for (int i = 0; i < 8; ++i) {          // a warp takes eight channels: sums of l over the tokens behind each token
     const int d = warp * 8 + i;
     float lo = Ls[d * SP + lane], hi = Ls[d * SP + 32 + lane];
@@ -366,23 +369,31 @@ __global__ void __launch_bounds__(256, 2) gla_chunk_out_kernel(GlaArgs A, bool v
   float a[4][4];
 #pragma unroll
   for (int i = 0; i < 4; ++i) a[i][0] = a[i][1] = a[i][2] = a[i][3] = 0.f;
+  float nq[CH / 8], nk[CH / 8], nl[CH / 8];      // the next slice's q, k, l: requested while the current one is used
+  auto fetch_slice = [&](int sl) {
+    const bool in_d = sl * SL + lane < dk;
+    const size_t ch = (size_t)h * dk + sl * SL + lane;
+#pragma unroll
+    for (int i = 0; i < CH / 8; ++i) {
+      const bool in = in_d && warp + 8 * i < ck.n;
+      const size_t row = (size_t)ck.first + warp + 8 * i;
+      nq[i] = in ? A.q[row * A.ldq + ch] : 0.f;
+      nk[i] = in ? A.k[row * A.ldk + ch] : 0.f;
+      nl[i] = in ? A.log_decay[row * ((size_t)A.H * dk) + ch] : 0.f;
+    }
+  };
+  fetch_slice(0);
   for (int sl = 0; sl < n_slices; ++sl) {
     const int d0 = sl * SL;
-    {
-      const int d = lane;
-      const bool in_d = d0 + d < dk;
-      const size_t ch = (size_t)h * dk + d0 + d;
 #pragma unroll
-      for (int i = 0; i < CH / 8; ++i) {
-        const int t = warp + 8 * i;
-        const bool in = in_d && t < ck.n;
-        const size_t row = (size_t)ck.first + t;
-        Qs[d * SP + t] = in ? A.q[row * A.ldq + ch] * A.q_scale : 0.f;
-        Kst[d * SP + t] = in ? A.k[row * A.ldk + ch] : 0.f;
-        Ls[d * SP + t] = in ? A.log_decay[row * ((size_t)A.H * dk) + ch] : 0.f;
-      }
+    for (int i = 0; i < CH / 8; ++i) {
+      const int t = warp + 8 * i;
+      Qs[lane * SP + t] = nq[i] * A.q_scale;
+      Kst[lane * SP + t] = nk[i];
+      Ls[lane * SP + t] = nl[i];
     }
     __syncthreads();
+    if (sl + 1 < n_slices) fetch_slice(sl + 1);
     bool far = false;
 #pragma unroll
     for (int i = 0; i < SL / 8; ++i) {

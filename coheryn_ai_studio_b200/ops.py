@@ -1297,7 +1297,7 @@ def attention_maps(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_
         _i32(step.cu_q, "cu_q"); _i32(step.kv_lens, "kv_lens")
         lib = maps_attention_lib(dk, dv, maps, values_in_keys)
         B = len(q_lens)
-        single = any(n == 1 for n in q_lens) and num_heads // num_kv_heads <= 16
+        single = any(n == 1 for n in q_lens)
         floats = int(lib.coheryn_maps_scratch_floats(c_int(B), c_int(num_heads), c_int(step.max_kv_len), c_int(window or 0),
                                                      c_int(chunk or 0))) if single else 0
         scratch = torch.empty(floats, dtype=torch.float32, device=q.device) if floats else None

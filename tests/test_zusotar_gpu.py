@@ -462,7 +462,10 @@ def test_window_attention_mixer_in_portions_and_decoded(dtype, m, width, page):
 LATENTS = [({"heads": 4, "dim": 32, "rot_dim": 16, "vdim": 16, "kv_rank": 48, "scale": 0.25, "rot": {"dims": 16, "base": 1000.0}}, 64, 16),
            ({"heads": 5, "dim": 12, "rot_dim": 6, "vdim": 10, "kv_rank": 22, "scale": 0.3, "rot": {"dims": 6, "base": 77.0}}, 100, 8),
            ({"heads": 1, "dim": 48, "rot_dim": 64, "vdim": 80, "kv_rank": 272, "scale": 0.1, "rot": {"dims": 64, "base": 5e5}}, 128, 64),
-           ({"heads": 8, "dim": 16, "rot_dim": 32, "vdim": 32, "kv_rank": 96, "scale": 0.2, "rot": {"dims": 20, "base": 9.0}}, 64, 16)]
+           ({"heads": 8, "dim": 16, "rot_dim": 32, "vdim": 32, "kv_rank": 96, "scale": 0.2, "rot": {"dims": 20, "base": 9.0}}, 64, 16),
+           # more query heads than the sixteen rows of a decode tile, in two blocks and in three
+           ({"heads": 18, "dim": 16, "rot_dim": 16, "vdim": 16, "kv_rank": 48, "scale": 0.25, "rot": {"dims": 16, "base": 50.0}}, 64, 16),
+           ({"heads": 48, "dim": 16, "rot_dim": 16, "vdim": 16, "kv_rank": 48, "scale": 0.25, "rot": {"dims": 16, "base": 50.0}}, 64, 16)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
