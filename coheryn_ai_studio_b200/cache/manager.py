@@ -4,7 +4,8 @@ per group of layers with the same needs, and slots for per-request state of fixe
 Schedule entries whose mixers ask for the same :class:`PagedKV` (kv heads, head size,
 window) form a group: they share page ids and block tables, and each has its own slice
 of the group's pool ``[entry, K/V, page, kv head, slot in page, head_dim]``.  A group
-with a window gives a page back as soon as every later query lies past it; a finished
+with a window gives a page back as soon as every later query lies past it (a window may keep
+the first positions of a sequence in sight: their pages stay); a finished
 request gives everything back.  Full, hashed pages of groups without a window can be
 found again by a later request with the same token prefix (the reference hands a whole
 session's keys and values to the next request with a common prefix, capped at
@@ -105,6 +106,8 @@ class CacheManager:
         # the writes of padding rows (a decode batch padded up to a captured width).
         for g in self.groups:
             n = g.need
+            if n.keep_first < 0 or (n.keep_first and n.window is None):
+                raise ValueError("kept first positions are those that a window would leave behind: they need a window")
             if n.stride < 1 or (n.stride > 1 and n.window is not None):
                 raise ValueError("rows that stand for blocks of positions need a positive stride and take no window")
             rows_pp = n.rows_per_page(self.page_size)      # rows of a page of this group (the books count positions)
@@ -130,7 +133,8 @@ class CacheManager:
         reuse = bool(prefix_reuse) and not self._state and all(g.need.window is None for g in self.groups)
         self._lib = host()
         windows, n_groups = _ints([g.need.window or 0 for g in self.groups])
-        self._book = self._lib.coheryn_book_new(page_size, num_pages, max_requests, 1 if reuse else 0, n_groups, windows)
+        kept, _ = _ints([g.need.keep_first for g in self.groups])
+        self._book = self._lib.coheryn_book_new(page_size, num_pages, max_requests, 1 if reuse else 0, n_groups, windows, kept)
         if not self._book:
             raise CacheError("the native cache book could not be made")
         for gi, g in enumerate(self.groups):

@@ -50,7 +50,7 @@ def _host():
         P, I, L = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
         IP, S = ctypes.POINTER(ctypes.c_int), ctypes.c_char_p
         sig = {
-            "coheryn_book_new": (P, [I, I, I, I, I, IP]), "coheryn_book_delete": (None, [P]),
+            "coheryn_book_new": (P, [I, I, I, I, I, IP, IP]), "coheryn_book_delete": (None, [P]),
             "coheryn_book_prefix_reuse": (I, [P]), "coheryn_book_set_prefix_reuse": (None, [P, I]),
             "coheryn_book_pool": (P, [P, I]), "coheryn_book_slots": (P, [P]), "coheryn_book_count": (I, [P]),
             "coheryn_book_has": (I, [P, S]), "coheryn_book_admit": (I, [P, S, IP, I, IP, IP, ctypes.POINTER(L)]),

@@ -19,6 +19,7 @@ from .tutunex import TutunexConfig, tutunex_model_spec
 from .guvusun import GuvusunConfig, guvusun_model_spec
 from .zegelix import ZegelixConfig, zegelix_model_spec
 from .zusotar import ZusotarConfig, zusotar_model_spec
+from .vilazen import VilazenConfig, vilazen_model_spec
 from .spec import ModelSpec
 
 
@@ -194,3 +195,4 @@ register_architecture("Tutunex", TutunexConfig.from_dict, tutunex_model_spec, ad
 register_architecture("Guvusun", GuvusunConfig.from_dict, guvusun_model_spec, adapter_id="guvusun-b200-v1")
 register_architecture("Zegelix", ZegelixConfig.from_dict, zegelix_model_spec, adapter_id="zegelix-b200-v1")
 register_architecture("Zusotar", ZusotarConfig.from_dict, zusotar_model_spec, adapter_id="zusotar-b200-v1")
+register_architecture("Vilazen", VilazenConfig.from_dict, vilazen_model_spec, adapter_id="vilazen-b200-v1")

@@ -60,6 +60,7 @@ constexpr int value_chunk(int dv) {
 constexpr int DVC = value_chunk(DV), NCH = DV / DVC;
 constexpr int NT = BN / 8, OT = DVC / 8;
 constexpr int MAX_SPLITS = 16;
+constexpr int MAX_PARTS = (MAX_SPLITS + 1) * WARPS;      // a split more for kept first positions
 typedef __nv_bfloat16 bf16;
 
 struct MapsArgs {
@@ -67,7 +68,7 @@ struct MapsArgs {
   const bf16* k_cache; const bf16* v_cache;
   const int* block_tables; int max_blocks;
   const int* cu_q; const int* kv_lens;
-  int nh, nkv, page_size, window, chunk, sink, head_norm, skip_single;
+  int nh, nkv, page_size, window, chunk, keep, sink, head_norm, skip_single;
   int table_cache;      // block-table entries a CTA of the prompt kernel may keep in shared memory
   float scale_log2, lambda, eps, out_scale;
   const float* sink_scores;     // [heads]: the sink's score per head (null: 0)
@@ -113,10 +114,12 @@ __device__ __forceinline__ float quad_sum(float v) {
   v += __shfl_xor_sync(0xffffffffu, v, 1);
   return v + __shfl_xor_sync(0xffffffffu, v, 2);
 }
-__device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
-  int f = window > 0 ? max(0, pos - window + 1) : 0;
-  if (chunk > 0) f = max(f, (pos / chunk) * chunk);
-  return f;
+// The first of the run of keys that ends at the row itself.  A window may keep the first `keep` positions of the sequence in
+// sight: they stand apart from that run, unless the two touch and the run then starts at 0.  (In order of the positions.)
+__device__ __forceinline__ int first_visible(const MapsArgs& A, int pos) {
+  int f = A.window > 0 ? max(0, pos - A.window + 1) : 0;
+  if (A.chunk > 0) f = max(f, (pos / A.chunk) * A.chunk);
+  return f <= A.keep ? 0 : f;
 }
 
 // 2^x by the hardware's approximation (two units in the last place; 2^-inf = 0).
@@ -200,14 +203,15 @@ __device__ __forceinline__ void weights_times_values(float (&o)[OT][4], const fl
 }
 
 // The scores of a tile in the log2 domain, masked: element (nt, e) belongs to row (e >> 1) of the thread's two rows
-// and to key key0 + nt * 8 + 2 (lane & 3) + (e & 1); a key outside [first, pos] of its row becomes -infinity.
-__device__ __forceinline__ void mask_scale(float (&s)[NT][4], int key0, int lane, const int (&pos)[2], const int (&first)[2], float scale_log2) {
+// and to key key0 + nt * 8 + 2 (lane & 3) + (e & 1); a key outside [first, pos] of its row that is not one of the first
+// `keep` becomes -infinity.
+__device__ __forceinline__ void mask_scale(float (&s)[NT][4], int key0, int lane, const int (&pos)[2], const int (&first)[2], int keep, float scale_log2) {
 #pragma unroll
   for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int j = key0 + nt * 8 + 2 * (lane & 3) + (e & 1), r = e >> 1;
-      s[nt][e] = (j <= pos[r] && j >= first[r]) ? s[nt][e] * scale_log2 : -INFINITY;
+      s[nt][e] = (j <= pos[r] && (j >= first[r] || j < keep)) ? s[nt][e] * scale_log2 : -INFINITY;
     }
 }
 
@@ -246,50 +250,58 @@ __global__ void __launch_bounds__(WARPS * 32, CO_MAPS_MIN_CTAS) maps_tiles_kerne
     const bool ok = row < rows;
     cp_async16(qs + row * KS + ch * 8, A.q + (size_t)(q0 + tile * BM + (ok ? row : 0)) * A.ldq + (size_t)h * KROW + ch * 8, ok ? 16 : 0);
   }
-  const int t_lo = first_visible(pos_lo, A.window, A.chunk) / BN, t_hi = pos_hi / BN, n_tiles = t_hi - t_lo + 1;
+  const int t_lo = first_visible(A, pos_lo) / BN, t_hi = pos_hi / BN;
+  // the tiles of the kept first positions, as far as they lie before the others, then tiles t_lo .. t_hi
+  const int n_kept = min(t_lo, (A.keep + BN - 1) / BN), n_tiles = n_kept + t_hi - t_lo + 1;
+  const int* kept_table = table;
   {   // the pages of the CTA's keys, looked up once: the tile loads then read shared memory
     const int e0 = (t_lo * BN) / A.page_size, e1 = min(t_hi * BN + BN - 1, kv_len - 1) / A.page_size;
-    if (e1 - e0 + 1 <= A.table_cache) {
-      for (int i = tid; i <= e1 - e0; i += WARPS * 32) tbl[i] = table[e0 + i];
+    const int kept = n_kept > 0 ? (n_kept * BN - 1) / A.page_size + 1 : 0;
+    if (e1 - e0 + 1 + kept <= A.table_cache) {
+      for (int i = tid; i < kept + e1 - e0 + 1; i += WARPS * 32) tbl[i] = table[i < kept ? i : e0 + i - kept];
       __syncthreads();
-      table = tbl - e0;
+      kept_table = tbl;
+      table = tbl + kept - e0;
     }
   }
+  auto first_key = [&](int i) { return (i < n_kept ? i : t_lo + i - n_kept) * BN; };
   int pos[2], first[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int row = warp * 16 + (lane >> 2) + 8 * i;
     pos[i] = row < rows ? pos_lo + row : -1;                      // -1: a row beyond the portion sees nothing
-    first[i] = row < rows ? first_visible(pos[i], A.window, A.chunk) : 0;
+    first[i] = row < rows ? first_visible(A, pos[i]) : 0;
   }
   const bf16* qw = qs + warp * 16 * KS;
   // what the warp's rows see together: a tile none of them sees is skipped, one all of them see whole needs no mask
   const bool whole_warp = warp * 16 + 15 < rows;
   const int wp_lo = pos_lo + warp * 16, wp_hi = min(pos_hi, wp_lo + 15);
-  const int wf_lo = first_visible(min(wp_lo, pos_hi), A.window, A.chunk), wf_hi = first_visible(wp_hi, A.window, A.chunk);
+  const int wf_lo = first_visible(A, min(wp_lo, pos_hi)), wf_hi = first_visible(A, wp_hi);
+  auto unseen_tile = [&](int key0) { return warp * 16 >= rows || key0 > wp_hi || (key0 + BN - 1 < wf_lo && key0 >= A.keep); };
+  auto open_tile = [&](int key0) { return whole_warp && key0 + BN - 1 <= wp_lo && (key0 >= wf_hi || key0 + BN <= A.keep); };
 
   // pass 1: maximum and sum of every row, per map
   float mx[MAPS][2], sum[MAPS][2];
 #pragma unroll
   for (int m = 0; m < MAPS; ++m) { mx[m][0] = mx[m][1] = -INFINITY; sum[m][0] = sum[m][1] = 0.f; }
-  load_keys<WARPS * 32>(ks, nullptr, A, table, kvh, t_lo * BN, kv_len, tid);
+  load_keys<WARPS * 32>(ks, nullptr, A, n_kept ? kept_table : table, kvh, first_key(0), kv_len, tid);
   cp_commit();
   for (int i = 0; i < n_tiles; ++i) {
-    if (i + 1 < n_tiles) load_keys<WARPS * 32>(ks + ((i + 1) & 1) * BN * KS, nullptr, A, table, kvh, (t_lo + i + 1) * BN, kv_len, tid);
+    if (i + 1 < n_tiles)
+      load_keys<WARPS * 32>(ks + ((i + 1) & 1) * BN * KS, nullptr, A, i + 1 < n_kept ? kept_table : table, kvh, first_key(i + 1), kv_len, tid);
     cp_commit();
     cp_wait<1>();
     __syncthreads();
     const bf16* kt = ks + (i & 1) * BN * KS;
-    const int key0 = (t_lo + i) * BN;
-    const bool unseen = warp * 16 >= rows || key0 > wp_hi || key0 + BN - 1 < wf_lo;
-    const bool open = whole_warp && key0 >= wf_hi && key0 + BN - 1 <= wp_lo;
+    const int key0 = first_key(i);
+    const bool unseen = unseen_tile(key0), open = open_tile(key0);
 #pragma unroll
     for (int m = 0; m < MAPS; ++m) {
       if (unseen) break;
       float s[NT][4];
       scores(s, qw, kt, m, lane);
       if (open) scale_only(s, A.scale_log2);
-      else mask_scale(s, key0, lane, pos, first, A.scale_log2);
+      else mask_scale(s, key0, lane, pos, first, A.keep, A.scale_log2);
 #pragma unroll
       for (int rr = 0; rr < 2; ++rr) {
         float tm = -INFINITY;
@@ -331,25 +343,25 @@ __global__ void __launch_bounds__(WARPS * 32, CO_MAPS_MIN_CTAS) maps_tiles_kerne
   float o[OT][4];
 #pragma unroll
   for (int nt = 0; nt < OT; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
-  load_keys<WARPS * 32>(ks, vs, A, table, kvh, t_lo * BN, kv_len, tid);
+  load_keys<WARPS * 32>(ks, vs, A, n_kept ? kept_table : table, kvh, first_key(0), kv_len, tid);
   cp_commit();
   for (int i = 0; i < n_tiles; ++i) {
     if (i + 1 < n_tiles)
-      load_keys<WARPS * 32>(ks + ((i + 1) & 1) * BN * KS, vs + ((i + 1) & 1) * BN * VS, A, table, kvh, (t_lo + i + 1) * BN, kv_len, tid);
+      load_keys<WARPS * 32>(ks + ((i + 1) & 1) * BN * KS, vs + ((i + 1) & 1) * BN * VS, A, i + 1 < n_kept ? kept_table : table, kvh,
+                            first_key(i + 1), kv_len, tid);
     cp_commit();
     cp_wait<1>();
     __syncthreads();
     const bf16* kt = ks + (i & 1) * BN * KS;
-    const int key0 = (t_lo + i) * BN;
-    const bool unseen = warp * 16 >= rows || key0 > wp_hi || key0 + BN - 1 < wf_lo;
-    const bool open = whole_warp && key0 >= wf_hi && key0 + BN - 1 <= wp_lo;
+    const int key0 = first_key(i);
+    const bool unseen = unseen_tile(key0), open = open_tile(key0);
     if (!unseen) {
     float w[NT][4];
     {
       float s[NT][4];
       scores(s, qw, kt, 0, lane);
       if (open) scale_only(s, A.scale_log2);
-      else mask_scale(s, key0, lane, pos, first, A.scale_log2);
+      else mask_scale(s, key0, lane, pos, first, A.keep, A.scale_log2);
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
@@ -357,7 +369,7 @@ __global__ void __launch_bounds__(WARPS * 32, CO_MAPS_MIN_CTAS) maps_tiles_kerne
       if (MAPS == 2) {
         scores(s, qw, kt, MAPS - 1, lane);
         if (open) scale_only(s, A.scale_log2);
-        else mask_scale(s, key0, lane, pos, first, A.scale_log2);
+        else mask_scale(s, key0, lane, pos, first, A.keep, A.scale_log2);
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
@@ -408,9 +420,11 @@ __global__ void __launch_bounds__(WARPS * 32) maps_decode_kernel(MapsArgs A, flo
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int first_head = kvh * per_kv + (blockIdx.y % blocks) * 16;      // the CTA's query heads: this one and the next ones
   const int group = min(16, (kvh + 1) * per_kv - first_head);
-  const int p = A.kv_lens[r] - 1, f = first_visible(p, A.window, A.chunk);
-  const int key_lo = (f / split_keys + split) * split_keys;      // splits at absolute multiples of their size
-  if (key_lo > p) return;                                         // the combine kernel knows which splits exist
+  const int p = A.kv_lens[r] - 1, f = first_visible(A, p);
+  const int n_run = p / split_keys - f / split_keys + 1;          // splits at absolute multiples of their size
+  const bool kept = split == n_run && f > 0 && A.keep > 0;        // ... and one behind them for the kept first positions
+  if (split >= n_run && !kept) return;                            // the combine kernel knows which splits exist
+  const int key_lo = kept ? 0 : (f / split_keys + split) * split_keys, last = kept ? A.keep - 1 : p;
   const int* table = A.block_tables + (size_t)r * A.max_blocks;
   for (int c = tid; c < 16 * (KROW / 8); c += WARPS * 32) {
     const int row = c / (KROW / 8), ch = c % (KROW / 8);
@@ -420,10 +434,10 @@ __global__ void __launch_bounds__(WARPS * 32) maps_decode_kernel(MapsArgs A, flo
   cp_commit();
   bf16* kw = kall + warp * BN * KS;
   bf16* vw = vall + warp * BN * VROW;
-  const int quarter = split_keys / WARPS;                         // a multiple of BN
-  const int w_lo = key_lo + warp * quarter, w_hi = min(w_lo + quarter, p + 1);
-  const int pos[2] = {(lane >> 2) < group ? p : -1, (lane >> 2) + 8 < group ? p : -1};
-  const int first[2] = {f, f};
+  const int quarter = kept ? (A.keep + WARPS * BN - 1) / (WARPS * BN) * BN : split_keys / WARPS;      // a multiple of BN
+  const int w_lo = key_lo + warp * quarter, w_hi = min(w_lo + quarter, last + 1);
+  const int pos[2] = {(lane >> 2) < group ? last : -1, (lane >> 2) + 8 < group ? last : -1};
+  const int first[2] = {kept ? 0 : f, kept ? 0 : f};
   if (w_lo < w_hi) load_keys<32>(kw, vw, A, table, kvh, w_lo, p + 1, lane);     // in flight with the queries
   cp_commit();
   cp_wait<0>();
@@ -444,7 +458,7 @@ __global__ void __launch_bounds__(WARPS * 32) maps_decode_kernel(MapsArgs A, flo
       }
       float s[NT][4];
       scores(s, qs, kw, m, lane);
-      mask_scale(s, key0, lane, pos, first, A.scale_log2);
+      mask_scale(s, key0, lane, pos, first, 0, A.scale_log2);
 #pragma unroll
       for (int rr = 0; rr < 2; ++rr) {
         float tm = -INFINITY;
@@ -489,24 +503,24 @@ __global__ void __launch_bounds__(WARPS * 32) maps_decode_kernel(MapsArgs A, flo
 // one thread each and turned into factors in shared memory; the outputs are then added with independent loads.
 __global__ void __launch_bounds__(128) maps_combine_kernel(MapsArgs A, const float* __restrict__ scratch, int split_keys, int n_splits) {
   __shared__ float red[33];
-  __shared__ float factor_s[MAPS][MAX_SPLITS * WARPS];
+  __shared__ float factor_s[MAPS][MAX_PARTS];
   __shared__ float coef_s[MAPS];
   co_pdl_launch_dependents();
   co_pdl_wait();
   const int r = blockIdx.x, h = blockIdx.y;
   const int q0 = A.cu_q[r], q_len = A.cu_q[r + 1] - q0;
   if (q_len != 1) return;
-  const int p = A.kv_lens[r] - 1, f = first_visible(p, A.window, A.chunk);
-  const int n_parts = (p / split_keys - f / split_keys + 1) * WARPS;
+  const int p = A.kv_lens[r] - 1, f = first_visible(A, p);
+  const int n_parts = (p / split_keys - f / split_keys + 1 + (f > 0 && A.keep > 0 ? 1 : 0)) * WARPS;
   const float* base = scratch + ((size_t)r * A.nh + h) * MAPS * (n_splits * WARPS) * (DV + 2);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (warp < MAPS) {                       // a warp per map: maxima and sums of its parts, merged in a fixed tree
     const float* parts = base + (size_t)warp * (n_splits * WARPS) * (DV + 2);
-    float m[(MAX_SPLITS * WARPS + 31) / 32], l[(MAX_SPLITS * WARPS + 31) / 32];
+    float m[(MAX_PARTS + 31) / 32], l[(MAX_PARTS + 31) / 32];
     const float sv = sink_log2(A, h);
     float M = A.sink ? sv : -INFINITY;
 #pragma unroll
-    for (int k = 0; k < (MAX_SPLITS * WARPS + 31) / 32; ++k) {
+    for (int k = 0; k < (MAX_PARTS + 31) / 32; ++k) {
       const int i = lane + 32 * k;
       m[k] = i < n_parts ? parts[i * (DV + 2) + DV] : -INFINITY;
       l[k] = i < n_parts ? parts[i * (DV + 2) + DV + 1] : 0.f;
@@ -515,7 +529,7 @@ __global__ void __launch_bounds__(128) maps_combine_kernel(MapsArgs A, const flo
     M = co_warp_max(M);
     float L = 0.f;
 #pragma unroll
-    for (int k = 0; k < (MAX_SPLITS * WARPS + 31) / 32; ++k) {
+    for (int k = 0; k < (MAX_PARTS + 31) / 32; ++k) {
       const int i = lane + 32 * k;
       const float fac = ex2(m[k] - M);                    // 0 for a part that saw no key
       if (i < n_parts) factor_s[warp][i] = fac;
@@ -557,23 +571,27 @@ CO_EXPORT int coheryn_maps_values_in_keys() { return V_IN_K ? 1 : 0; }
 
 // How the keys a decoded row can see are cut: the keys per split (a multiple of what a CTA's warps take in one round, cut at
 // absolute multiples of itself) and the most splits a row then has (its keys may straddle one boundary more than their
-// number fills).
-static void decode_plan(int max_kv_len, int window, int chunk, int* split_keys, int* n_splits) {
+// number fills), and one for kept first positions.
+static int most_visible(int max_kv_len, int window, int chunk, int keep) {
   int visible = max_kv_len;
   if (chunk > 0 && chunk < visible) visible = chunk;
-  if (window > 0 && window < visible) visible = window;
+  if (window > 0 && (long)window + keep < visible) visible = window + keep;
+  return visible;
+}
+static void decode_plan(int max_kv_len, int window, int chunk, int keep, int* split_keys, int* n_splits) {
+  const int visible = most_visible(max_kv_len, window, chunk, keep);
   const int unit = WARPS * BN;
   int keys = ((visible + (MAX_SPLITS - 1) - 1) / (MAX_SPLITS - 1) + unit - 1) / unit * unit;
   if (keys < unit) keys = unit;
   *split_keys = keys;
   int n = (visible + keys - 1) / keys + 1;
-  *n_splits = n > MAX_SPLITS ? MAX_SPLITS : n;
+  *n_splits = (n > MAX_SPLITS ? MAX_SPLITS : n) + (keep > 0 ? 1 : 0);
 }
 
 // Floats of scratch that the decode kernels need for `B` requests whose longest context is `max_kv_len`.
-CO_EXPORT long coheryn_maps_scratch_floats(int B, int nh, int max_kv_len, int window, int chunk) {
+CO_EXPORT long coheryn_maps_scratch_floats(int B, int nh, int max_kv_len, int window, int chunk, int keep) {
   int keys, n;
-  decode_plan(max_kv_len, window, chunk, &keys, &n);
+  decode_plan(max_kv_len, window, chunk, keep, &keys, &n);
   return (long)B * nh * MAPS * n * WARPS * (DV + 2);
 }
 
@@ -583,7 +601,7 @@ CO_EXPORT long coheryn_maps_scratch_floats(int B, int nh, int max_kv_len, int wi
 // gates_ld; head h's output of token t is multiplied by sigmoid(gates[t, h]).
 CO_EXPORT int coheryn_attention_maps_bf16(const void* q, long ldq, void* out, long ldo, const void* k_cache, const void* v_cache,
                                           const int* block_tables, int max_blocks, const int* cu_q, const int* kv_lens, int B,
-                                          int nh, int nkv, int page_size, int window, int chunk, int sink, float scale,
+                                          int nh, int nkv, int page_size, int window, int chunk, int keep, int sink, float scale,
                                           float lambda, int head_norm, float eps, float out_scale, int max_q_len, int max_kv_len,
                                           int any_single, int any_longer, float* scratch, long scratch_floats,
                                           const float* sink_scores, const float* gates, long gates_ld, cudaStream_t stream) {
@@ -591,17 +609,16 @@ CO_EXPORT int coheryn_attention_maps_bf16(const void* q, long ldq, void* out, lo
   if (nkv <= 0 || nh % nkv) CO_FAIL("attention_maps_bf16: %d heads do not group over %d kv heads", nh, nkv);
   if ((ldq & 7) || (ldo & 1) || ((uintptr_t)q & 15) || ((uintptr_t)out & 3) || ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15))
     CO_FAIL("attention_maps_bf16: rows of q must start on 16-byte boundaries, rows of out on 4-byte ones");
+  if (keep < 0 || (keep > 0 && (window <= 0 || chunk > 0))) CO_FAIL("attention_maps_bf16: kept first positions stand beside a window (%d kept)", keep);
   if (head_norm && NCH > 1) CO_FAIL("attention_maps_bf16: a normalised output needs values of at most 256 channels (%d)", DV);
   const int blocks = (nh / nkv + 15) / 16;             // of query heads per kv head
   const bool decode = any_single != 0;
   MapsArgs A{(const bf16*)q, ldq, (bf16*)out, ldo, (const bf16*)k_cache, (const bf16*)v_cache, block_tables, max_blocks, cu_q,
-             kv_lens, nh, nkv, page_size, window, chunk, sink, head_norm, decode ? 1 : 0, 0,
+             kv_lens, nh, nkv, page_size, window, chunk, keep, sink, head_norm, decode ? 1 : 0, 0,
              scale * 1.4426950408889634f, lambda, eps, out_scale, sink_scores, gates, gates_ld};
   if (any_longer || !decode) {
-    int visible = max_kv_len;                              // the most keys a row can see
-    if (chunk > 0 && chunk < visible) visible = chunk;
-    if (window > 0 && window < visible) visible = window;
-    const long entries = ((long)visible + BM + 2 * BN) / page_size + 2;
+    const int visible = most_visible(max_kv_len, window, chunk, keep);      // the most keys a row can see
+    const long entries = ((long)visible + BM + 3 * BN) / page_size + 3;
     A.table_cache = entries <= 4096 ? (int)entries : 0;    // a longer table is read from global memory
     const size_t smem = ((size_t)BM * KS + (size_t)2 * BN * KS + (size_t)2 * BN * VROW) * sizeof(bf16) + (size_t)A.table_cache * sizeof(int);
     if (smem > 48 * 1024) cudaFuncSetAttribute(maps_tiles_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -609,10 +626,10 @@ CO_EXPORT int coheryn_attention_maps_bf16(const void* q, long ldq, void* out, lo
     CO_CHECK_LAUNCH("maps_tiles");
   }
   if (decode) {
-    if (scratch_floats < coheryn_maps_scratch_floats(B, nh, max_kv_len, window, chunk))
+    if (scratch_floats < coheryn_maps_scratch_floats(B, nh, max_kv_len, window, chunk, keep))
       CO_FAIL("attention_maps_bf16: scratch of %ld floats is too small", scratch_floats);
     int split_keys, n_splits;
-    decode_plan(max_kv_len, window, chunk, &split_keys, &n_splits);
+    decode_plan(max_kv_len, window, chunk, keep, &split_keys, &n_splits);
     const size_t smem = ((size_t)16 * KS + (size_t)WARPS * BN * (KS + VROW)) * sizeof(bf16);
     if (smem > 48 * 1024) cudaFuncSetAttribute(maps_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     co_launch(maps_decode_kernel, dim3(B, nkv * blocks, n_splits), dim3(WARPS * 32), smem, stream, A, scratch, split_keys, n_splits);

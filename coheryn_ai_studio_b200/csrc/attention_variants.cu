@@ -5,7 +5,8 @@
 //     over the same values, and the head's output is a_0 - lambda a_1 (differential attention; maps = 1 is the
 //     ordinary case);
 //   * a mask by CHUNKS: position i sees j <= i with floor(i / chunk) = floor(j / chunk), chunks counted from
-//     position 0 of the sequence; or a window (i - j < window); or all j <= i;
+//     position 0 of the sequence; or a window (i - j < window), beside which the first `keep` positions of the sequence
+//     may stay in sight; or all j <= i;
 //   * a SINK: one more term exp(0) in the softmax's denominator that carries no value;
 //   * the head's output divided by its root mean square over the value channels, and a constant factor;
 //   * values of another head size than keys; values that are the first dv channels of the key row itself (a latent
@@ -13,9 +14,9 @@
 //   * a sink with a learned score per head instead of 0.
 //
 // And the kernel in front of it: queries and keys normalised per head (RMS over dk, one weight [dk] shared by the
-// heads) and/or rotated by position (rotate-half pairing over the first `rot` channels of every unit of dk, the
-// angle position * frequency computed here in float32 pairs, so no table bounds the positions), then keys and
-// values written into their cache pages.
+// heads) or over the whole projection (a weight per channel), and/or rotated by position (rotate-half pairing over the first `rot` channels of every unit of dk, the
+// angle position * frequency computed here in float32 pairs, so no table bounds the positions), values mixed with those
+// that an earlier layer made of the same token, then keys and values written into their cache pages.
 //
 // Everything is float32 arithmetic on float32 or bfloat16 storage; scores, weights and their sums never leave
 // float32.  A row's result depends on its position and the keys it sees only, in an order fixed by those.
@@ -27,6 +28,8 @@ namespace {
 // q_out[t, u, :] and the cache rows of token t.  A "unit" is dk consecutive channels of a projection that are
 // normalised and rotated together: q has q_units of them (heads x maps), k has k_units (kv heads x maps).
 // freq: [rot/2][2] float32 = (high, low) parts of each pair's frequency; angle = position * (high + low).
+// normalise: 0 none, 1 per unit (weights [dk]), 2 over all channels of q, and all of k, at once (weights [units * dk]).
+// v_first (null: none): values [T][nkv * dv] of row stride ldf; what is cached is keep_v v + mix_v v_first.
 // ---------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -34,8 +37,10 @@ unit_norm_rope_kv_write_kernel(const float* __restrict__ q, const float* __restr
                                const void* __restrict__ wq, const void* __restrict__ wk, int w_dtype, float eps, int normalise,
                                const int* __restrict__ positions, const float* __restrict__ freq, int rot, float rot_scale,
                                T* __restrict__ q_out, long ldq, const int* __restrict__ slots, T* __restrict__ k_cache,
-                               T* __restrict__ v_cache, int q_units, int k_units, int nkv, int dk, int dv, int page_size) {
+                               T* __restrict__ v_cache, int q_units, int k_units, int nkv, int dk, int dv, int page_size,
+                               const float* __restrict__ v_first, long ldf, float keep_v, float mix_v) {
   extern __shared__ __align__(16) float sm[];
+  __shared__ float whole_s[2];
   co_pdl_launch_dependents();
   co_pdl_wait();
   const size_t t = blockIdx.x;
@@ -71,11 +76,20 @@ unit_norm_rope_kv_write_kernel(const float* __restrict__ q, const float* __restr
     if (normalise) {
       float ss = 0.f;
       for (int d = lane; d < dk; d += 32) ss = fmaf(xs[u * dk + d], xs[u * dk + d], ss);
-      s = 1.0f / sqrtf(co_warp_sum(ss) / (float)dk + eps);
+      ss = co_warp_sum(ss);
+      s = normalise == 2 ? ss : 1.0f / sqrtf(ss / (float)dk + eps);
     }
     if (lane == 0) scale_s[u] = s;
   }
   __syncthreads();
+  if (normalise == 2 && warp < 2) {      // the sums of a side's units, added in a fixed order
+    const int u0 = warp ? q_units : 0, n = warp ? units - q_units : q_units;
+    float ss = 0.f;
+    for (int u = lane; u < n; u += 32) ss += scale_s[u0 + u];
+    ss = co_warp_sum(ss);
+    if (lane == 0) whole_s[warp] = n > 0 ? 1.0f / sqrtf(ss / ((float)n * (float)dk) + eps) : 0.f;
+  }
+  if (normalise == 2) __syncthreads();
   int slot = 0;
   size_t page = 0, off = 0;
   if (write) { slot = slots[t]; page = (size_t)(slot / page_size); off = (size_t)(slot % page_size); }
@@ -85,6 +99,7 @@ unit_norm_rope_kv_write_kernel(const float* __restrict__ q, const float* __restr
     const void* w = u < q_units ? wq : wk;
     auto val = [&](int dd) {
       const float x = xs[u * dk + dd];
+      if (normalise == 2) return (x * whole_s[u < q_units ? 0 : 1]) * co_load_any(w, w_dtype, (size_t)(u < q_units ? u : u - q_units) * dk + dd);
       return normalise ? (x * scale_s[u]) * co_load_any(w, w_dtype, dd) : x;
     };
     float y;
@@ -107,20 +122,21 @@ unit_norm_rope_kv_write_kernel(const float* __restrict__ q, const float* __restr
   const float* vr = v + t * ld;
   for (int e = threadIdx.x; e < nkv * dv; e += blockDim.x) {
     const int g = e / dv, d = e % dv;
-    v_cache[((page * nkv + g) * page_size + off) * dv + d] = co_from_float<T>(vr[e]);
+    const float x = v_first ? keep_v * vr[e] + mix_v * v_first[t * ldf + e] : vr[e];
+    v_cache[((page * nkv + g) * page_size + off) * dv + d] = co_from_float<T>(x);
   }
 }
 
 // ---------------------------------------------------------------------------------
 // One CTA per (token, query head); four warps each run an online softmax per map over the keys
-// first + warp, first + warp + 4, ..; their (maximum, sum, accumulator) triples are merged in warp order.
+// n = warp, warp + 4, .. (kept first positions, then those from the first visible one on); their (maximum, sum, accumulator) triples are merged in warp order.
 // ---------------------------------------------------------------------------------
 constexpr int WARPS = 4;
 constexpr int MAX_MAPS = 2;
 constexpr int WIDE_PER_LANE = 24; // head sizes up to 768, for a single map
 
 struct MapsShape {
-  int nh, nkv, dk, dv, maps, page_size, window, chunk, sink, head_norm;
+  int nh, nkv, dk, dv, maps, page_size, window, chunk, keep, sink, head_norm;
   float scale, lambda, eps, out_scale;
   const float* sink_scores;     // [heads]: the sink's score per head (null: 0)
   long v_row;                   // channels between two value rows (dv, or the key row's size when values live in the keys)
@@ -158,7 +174,9 @@ attention_maps_kernel(const T* __restrict__ q, long q_stride, T* __restrict__ ou
 #pragma unroll
     for (int i = 0; i < MAX_PER_LANE; ++i) acc[a][i] = 0.f;
   }
-  for (int kp = first + warp; kp <= pos; kp += WARPS) {
+  const int n_kept = min(S.keep, first), n_keys = n_kept + pos - first + 1;
+  for (int n = warp; n < n_keys; n += WARPS) {
+    const int kp = n < n_kept ? n : first + n - n_kept;
     const int page = table[kp / S.page_size];
     const size_t row = ((size_t)page * S.nkv + kvh) * S.page_size + (kp % S.page_size);
     const T* kr = k_cache + row * (size_t)(MAPS * dk);
@@ -302,14 +320,17 @@ latent_prepare_kernel(const float* __restrict__ q, const float* __restrict__ kv,
 }  // namespace
 
 
-// freq: float32 [rot/2][2] on the device (null when rot = 0).  wq / wk: [dk] (null when normalise = 0).  slots null: only the
+// freq: float32 [rot/2][2] on the device (null when rot = 0).  wq / wk: [dk], or [units * dk] with
+// normalise = 2 (null when normalise = 0).  slots null: only the
 // queries are made.  The key cache is [page][nkv][page_size][k_units / nkv * dk], the value cache [page][nkv][page_size][dv].
 CO_EXPORT int coheryn_unit_norm_rope_kv_write(const float* q, const float* k, const float* v, long ld, const void* wq,
                                               const void* wk, int w_dtype, float eps, int normalise, const int* positions,
                                               const float* freq, int rot, float rot_scale, void* q_out, int dtype, long ldq,
                                               const int* slots, void* k_cache, void* v_cache, int T, int q_units, int k_units,
-                                              int nkv, int dk, int dv, int page_size, cudaStream_t stream) {
+                                              int nkv, int dk, int dv, int page_size, const float* v_first, long ldf,
+                                              float keep_v, float mix_v, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (normalise < 0 || normalise > 2) CO_FAIL("unit_norm_rope_kv_write: unknown normalisation %d", normalise);
   if (q_units < 1 || dk < 1 || dv < 1 || page_size < 1 || rot < 0 || rot > dk || (rot & 1))
     CO_FAIL("unit_norm_rope_kv_write: bad sizes (units %d, channels %d, rotated %d)", q_units, dk, rot);
   if (slots && (nkv < 1 || k_units < nkv || k_units % nkv)) CO_FAIL("unit_norm_rope_kv_write: %d key units over %d kv heads", k_units, nkv);
@@ -322,7 +343,8 @@ CO_EXPORT int coheryn_unit_norm_rope_kv_write(const float* q, const float* k, co
     auto kern = unit_norm_rope_kv_write_kernel<TT>;                                                                   \
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);          \
     co_launch(kern, dim3(T), dim3(256), smem, stream, q, k, v, ld, wq, wk, w_dtype, eps, normalise, positions, freq, rot, \
-              rot_scale, (TT*)q_out, ldq, slots, (TT*)k_cache, (TT*)v_cache, q_units, k_units, nkv, dk, dv, page_size); \
+              rot_scale, (TT*)q_out, ldq, slots, (TT*)k_cache, (TT*)v_cache, q_units, k_units, nkv, dk, dv, page_size, v_first, \
+              ldf, keep_v, mix_v);                                                                                    \
   }
   if (dtype == CO_F32) GO(float)
   else if (dtype == CO_BF16) GO(__nv_bfloat16)
@@ -335,7 +357,7 @@ CO_EXPORT int coheryn_unit_norm_rope_kv_write(const float* q, const float* k, co
 CO_EXPORT int coheryn_attention_maps(const void* q, long q_stride, void* out, long out_stride, const void* k_cache,
                                      const void* v_cache, int dtype, const int* block_tables, int max_blocks,
                                      const int* token_req, const int* positions, int T, int nh, int nkv, int dk, int dv,
-                                     int maps, int page_size, int window, int chunk, int sink, float scale, float lambda,
+                                     int maps, int page_size, int window, int chunk, int keep, int sink, float scale, float lambda,
                                      int head_norm, float eps, float out_scale, const float* sink_scores, int values_in_keys,
                                      cudaStream_t stream) {
   if (T <= 0) return 0;
@@ -345,7 +367,8 @@ CO_EXPORT int coheryn_attention_maps(const void* q, long q_stride, void* out, lo
   if (values_in_keys && dv > maps * dk) CO_FAIL("attention_maps: %d value channels do not fit a key row of %d", dv, maps * dk);
   if (nkv <= 0 || nh % nkv != 0) CO_FAIL("attention_maps: %d heads do not group over %d kv heads", nh, nkv);
   if (maps < 1 || maps > MAX_MAPS) CO_FAIL("attention_maps: %d score maps per head (1..%d)", maps, MAX_MAPS);
-  MapsShape S{nh, nkv, dk, dv, maps, page_size, window, chunk, sink, head_norm, scale, lambda, eps, out_scale, sink_scores,
+  if (keep < 0 || (keep > 0 && (window <= 0 || chunk > 0))) CO_FAIL("attention_maps: kept first positions stand beside a window (%d kept)", keep);
+  MapsShape S{nh, nkv, dk, dv, maps, page_size, window, chunk, keep, sink, head_norm, scale, lambda, eps, out_scale, sink_scores,
               values_in_keys ? (long)maps * dk : (long)dv};
   if (values_in_keys) v_cache = k_cache;
   dim3 grid(T, nh);

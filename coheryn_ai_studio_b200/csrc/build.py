@@ -36,6 +36,7 @@ RECURRENT_SOURCES = ["recurrent.cu", "runtime.cu"]
 VARIANT_SOURCES = ["attention_variants.cu", "runtime.cu"]
 LINEAR_RECURRENCE_SOURCES = ["linear_recurrence.cu", "runtime.cu"]
 LINEAR_ATTENTION_SOURCES = ["linear_attention.cu", "runtime.cu"]
+LIGHTNING_SOURCES = ["lightning_attention.cu", "runtime.cu"]
 POOLED_ATTENTION_SOURCES = ["attention_pooled.cu", "runtime.cu"]
 HEADERS = ["common.cuh"]
 
@@ -264,6 +265,12 @@ def linear_attention_library() -> ctypes.CDLL:
     return load_library("linear_attention", LINEAR_ATTENTION_SOURCES)
 
 
+def lightning_library() -> ctypes.CDLL:
+    """The kernels of linear attention with a constant decay per head.  Compiled when a model with such a mixer is first
+    run."""
+    return load_library("lightning", LIGHTNING_SOURCES)
+
+
 def pooled_attention_library() -> ctypes.CDLL:
     """Window attention over positions and block means (float32 arithmetic) with the kernels that rotate and write its
     keys and values and keep the block means.  Compiled when a model with such a mixer is first run."""
@@ -309,7 +316,7 @@ def build_all(head_dims: Sequence[int] = (16, 32, 64, 128)) -> List[str]:
     paths = [build_host_library(), build_library("core", CORE_SOURCES), build_library("recurrent", RECURRENT_SOURCES),
              build_library("variants", VARIANT_SOURCES), build_library("routed", ROUTED_SOURCES),
              build_library("linear_recurrence", LINEAR_RECURRENCE_SOURCES),
-             build_library("linear_attention", LINEAR_ATTENTION_SOURCES),
+             build_library("linear_attention", LINEAR_ATTENTION_SOURCES), build_library("lightning", LIGHTNING_SOURCES),
              build_library("pooled_attention", POOLED_ATTENTION_SOURCES),
              build_library("pooled_tc_128_128", ["attention_pooled_tc.cu", "runtime.cu"], {"CO_PW_DK": 128, "CO_PW_DV": 128})]
     paths.append(build_library("maps_96_64_1_vk", ["attention_maps_tc.cu", "runtime.cu"],

@@ -156,8 +156,17 @@ __device__ __forceinline__ float co_gated(int e, float g, float u) {
   }
   return co_gate_act(e, g) * u;
 }
-// Whether an epilogue word is one the gated epilogues know.
-inline bool co_epilogue_known(int e) { return e >= 0 && ((e & 0xff) <= 2 ? e <= 2 : (e & 0xff) == CO_GATE_CLAMPED_SWISH); }
+// Words from CO_ACT_FIRST on are plain activations of the (biased) product, one output per column: 16 is the exact GELU,
+// z times the normal distribution function.  The two helpers split a word: the gate's part, and the plain activation.
+#define CO_ACT_FIRST 16
+#define CO_ACT_GELU 16
+__host__ __device__ __forceinline__ int co_gate_word(int e) { return (e & 0xff) < CO_ACT_FIRST ? e : 0; }
+__host__ __device__ __forceinline__ int co_plain_act(int e) { return (e & 0xff) < CO_ACT_FIRST ? 0 : e; }
+__device__ __forceinline__ float co_gelu(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
+// Whether an epilogue word is one the epilogues know.
+inline bool co_epilogue_known(int e) {
+  return e == CO_ACT_GELU || (e >= 0 && ((e & 0xff) <= 2 ? e <= 2 : (e & 0xff) == CO_GATE_CLAMPED_SWISH));
+}
 
 __device__ __forceinline__ float co_warp_sum(float v) {
 #pragma unroll

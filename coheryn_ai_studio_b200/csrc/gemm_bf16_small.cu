@@ -146,7 +146,7 @@ gemm_small_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __re
       v0 += red[wi * E + base];
       v1 += red[wi * E + base + 32];
     }
-    if (epilogue != 0) {
+    if (co_gate_word(epilogue) != 0) {
       // rows (n, n+1) = (gate_j, up_j), j = n / 2
       const float r = (epilogue & 0xff) == CO_GATE_CLAMPED_SWISH ? co_gated(epilogue, v0, v1)
                       : (epilogue == EPI_GATED_GELU_TANH ? co_gelu_tanh(v0) : v0 / (1.0f + __expf(-v0))) * v1;
@@ -160,6 +160,7 @@ gemm_small_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __re
       v0 += co_load_any(bias, bias_dtype, n);
       if (has1) v1 += co_load_any(bias, bias_dtype, n + 1);
     }
+    if (co_plain_act(epilogue)) { v0 = co_gelu(v0); v1 = co_gelu(v1); }
     const size_t o = (size_t)m * ldo + n;
     if (out_dtype == CO_BF16) {
       __nv_bfloat16* p = (__nv_bfloat16*)out + o;
@@ -314,7 +315,8 @@ int launch_small(const void* x, const void* w, const void* bias, int bias_dtype,
 
 // x: [M, K] bfloat16, row stride ldx (elements, a multiple of 8, base 16-byte aligned);
 // w: [N, K] bfloat16 contiguous; K a multiple of 8; M <= 64.
-// epilogue 0: out[M, N] (+ bias); 1: gated SiLU over interleaved rows, out[M, N/2].
+// epilogue 0: out[M, N] (+ bias); 1: gated SiLU over interleaved rows, out[M, N/2];
+// 16: out[M, N] = gelu(product + bias).
 CO_EXPORT int coheryn_gemm_bf16_small(const void* x, const void* w, const void* bias, int bias_dtype, void* out,
                                       int out_dtype, int M, int N, int K, long ldx, long ldo, int epilogue,
                                       cudaStream_t stream) {
@@ -322,7 +324,7 @@ CO_EXPORT int coheryn_gemm_bf16_small(const void* x, const void* w, const void* 
   if (M > 64) CO_FAIL("gemm_bf16_small: M = %d exceeds 64", M);
   if (K <= 0 || (K & 7) || (ldx & 7)) CO_FAIL("gemm_bf16_small: K = %d and the row stride %ld must be multiples of 8", K, ldx);
   if (((uintptr_t)x & 15) || ((uintptr_t)w & 15)) CO_FAIL("gemm_bf16_small: operands must be 16-byte aligned");
-  if (epilogue != 0 && (N & 1)) CO_FAIL("gemm_bf16_small: gated epilogue needs an even number of rows");
+  if (co_gate_word(epilogue) != 0 && (N & 1)) CO_FAIL("gemm_bf16_small: gated epilogue needs an even number of rows");
   if (!co_epilogue_known(epilogue)) CO_FAIL("gemm_bf16_small: unknown epilogue %d", epilogue);
   // Rows per CTA: as many as keep at least ~2 CTAs per SM (148 SMs); more rows per CTA
   // mean fewer re-reads of x through L2.  The warps of a CTA split K (a function of K

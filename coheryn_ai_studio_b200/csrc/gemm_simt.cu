@@ -12,7 +12,7 @@ constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;
 template <typename TX, typename TW, typename TO>
 __global__ void __launch_bounds__(256)
 gemm_simt_kernel(const TX* __restrict__ x, const TW* __restrict__ w, const void* __restrict__ bias,
-                 int bias_dtype, TO* __restrict__ out, int M, int N, int K, long ldx, long ldo) {
+                 int bias_dtype, TO* __restrict__ out, int M, int N, int K, long ldx, long ldo, int act) {
   __shared__ float xs[BK][BM + 4];
   __shared__ float ws[BK][BN + 4];
   const int tid = threadIdx.x;
@@ -59,6 +59,7 @@ gemm_simt_kernel(const TX* __restrict__ x, const TW* __restrict__ w, const void*
       if (gn >= N) continue;
       float v = acc[i][j];
       if (bias) v += co_load_any(bias, bias_dtype, gn);
+      if (act) v = co_gelu(v);
       out[(size_t)gm * ldo + gn] = co_from_float<TO>(v);
     }
   }
@@ -66,15 +67,17 @@ gemm_simt_kernel(const TX* __restrict__ x, const TW* __restrict__ w, const void*
 }  // namespace
 
 // x: [M, K] with row stride ldx; w: [N, K] contiguous; out: [M, N] with row stride ldo.
+// act 0: the (biased) product; CO_ACT_GELU: its exact GELU.
 CO_EXPORT int coheryn_gemm_simt(const void* x, int x_dtype, const void* w, int w_dtype, const void* bias,
                                 int bias_dtype, void* out, int out_dtype, int M, int N, int K, long ldx,
-                                long ldo, cudaStream_t stream) {
+                                long ldo, int act, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0) CO_FAIL("gemm_simt: K must be positive");
+  if (act != 0 && act != CO_ACT_GELU) CO_FAIL("gemm_simt: unknown activation %d", act);
   dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
 #define LAUNCH(TX, TW, TO)                                                                       \
   gemm_simt_kernel<TX, TW, TO><<<grid, 256, 0, stream>>>((const TX*)x, (const TW*)w, bias, bias_dtype, \
-                                                         (TO*)out, M, N, K, ldx, ldo)
+                                                         (TO*)out, M, N, K, ldx, ldo, act)
   if (x_dtype == CO_F32 && w_dtype == CO_F32 && out_dtype == CO_F32) LAUNCH(float, float, float);
   else if (x_dtype == CO_BF16 && w_dtype == CO_BF16 && out_dtype == CO_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16, __nv_bfloat16);
   else if (x_dtype == CO_BF16 && w_dtype == CO_BF16 && out_dtype == CO_F32) LAUNCH(__nv_bfloat16, __nv_bfloat16, float);

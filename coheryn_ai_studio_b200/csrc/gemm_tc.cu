@@ -34,11 +34,11 @@ struct Smem {
 
 // Sixty-four bfloat16 output columns of a warp's 32 rows (lane = row) through shared memory and
 // one TMA store: the accumulator columns come from tensor memory (64 of them, or 128 gate/up
-// columns in the gated case), bias or gate is applied, the 128 bytes of a row go to `stage`
+// columns in the gated case), bias and activation, or the gate, are applied, the 128 bytes of a row go to `stage`
 // (4 KB, 1024-byte aligned) in the 128-byte swizzle of the output tensor map, and lane 0 sends
 // the 32 x 64 box.  Rows and columns beyond the tensor are clipped by the copy.
 // bias_chunk: the bias of the chunk's first accumulator column (or null).
-__device__ __forceinline__ void store_chunk_tma(unsigned tmem_chunk, const float* bias_chunk, int gated,
+__device__ __forceinline__ void store_chunk_tma(unsigned tmem_chunk, const float* bias_chunk, int gated, int act,
                                                 unsigned char* stage, const CUtensorMap* map_out, int out_col,
                                                 int out_row, int lane) {
   uint4 pk[8];
@@ -65,6 +65,7 @@ __device__ __forceinline__ void store_chunk_tma(unsigned tmem_chunk, const float
       for (int j = 0; j < 32; j += 2) {
         float a = __uint_as_float(r[j]), b = __uint_as_float(r[j + 1]);
         if (bias_chunk) { a += bias_chunk[32 * q + j]; b += bias_chunk[32 * q + j + 1]; }
+        if (act) { a = co_gelu(a); b = co_gelu(b); }
         h[q * 16 + (j >> 1)] = __floats2bfloat162_rn(a, b);
       }
     }
@@ -190,7 +191,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
     if (waited && tma_out && !partial) {
       // bfloat16 output through shared memory and TMA stores: every MMA is complete, so the
       // stages are free and serve as the staging area (two 4 KB chunks per warp).
-      const int gated = epilogue;   // 0, or the gate's activation code
+      const int gated = co_gate_word(epilogue), act = co_plain_act(epilogue);   // 0, or the gate's word; 0, or a plain activation
       const int step = gated ? 128 : 64;
       unsigned char* stage = tiles + quarter * 8192;
       int chunk = 0;
@@ -202,7 +203,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           __syncwarp();
         }
         store_chunk_tma(tmem_base + ((unsigned)(quarter * 32) << 16) + (unsigned)c0, bias && !gated ? bias_s + c0 : nullptr,
-                        gated, stage + (chunk & 1) * 4096, &map_out, gated ? (n0 + c0) >> 1 : n0 + c0, m0 + quarter * 32, lane);
+                        gated, act, stage + (chunk & 1) * 4096, &map_out, gated ? (n0 + c0) >> 1 : n0 + c0, m0 + quarter * 32, lane);
       }
       if (lane == 0) tma_store_wait_all();
     } else if (waited) {
@@ -222,7 +223,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           }
           continue;
         }
-        if (epilogue != EPI_PLAIN) {
+        if (co_gate_word(epilogue) != EPI_PLAIN) {
           // columns (2j, 2j+1) = (gate_j, up_j): 16 outputs per 32 columns
           const int oc = (n0 + c0) >> 1;
           float v[16];
@@ -255,6 +256,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
         if (bias) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] += bias_s[c0 + j];
+        }
+        if (co_plain_act(epilogue)) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = co_gelu(v[j]);
         }
         const int nc = n0 + c0;
         if (out_dtype == CO_BF16) {
@@ -294,7 +299,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
 // One 32-column piece of an accumulator row: bias or gate, conversion, store.
 __device__ __forceinline__ void store_piece(const unsigned (&r)[32], int row, int nc, const float* bias_piece,
                                             void* __restrict__ out, int out_dtype, int N, long ldo, int epilogue) {
-  if (epilogue != EPI_PLAIN) {
+  if (co_gate_word(epilogue) != EPI_PLAIN) {
     // columns (2j, 2j+1) = (gate_j, up_j): 16 outputs per 32 columns
     const int oc = nc >> 1, n_out = N >> 1;
     float v[16];
@@ -326,6 +331,10 @@ __device__ __forceinline__ void store_piece(const unsigned (&r)[32], int row, in
   if (bias_piece) {
 #pragma unroll
     for (int j = 0; j < 32; ++j) v[j] += bias_piece[j];
+  }
+  if (co_plain_act(epilogue)) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) v[j] = co_gelu(v[j]);
   }
   if (out_dtype == CO_BF16) {
     __nv_bfloat16* p = (__nv_bfloat16*)out + (size_t)row * ldo + nc;
@@ -369,7 +378,7 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ partial, int spli
       v0 += p[0];
       if (has1) v1 += p[1];
     }
-    if (epilogue != EPI_PLAIN) {
+    if (co_gate_word(epilogue) != EPI_PLAIN) {
       const float r = co_gated(epilogue, v0, v1);
       const size_t o = (size_t)m * ldo + (n >> 1);
       if (out_dtype == CO_BF16) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(r);
@@ -380,6 +389,7 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ partial, int spli
       v0 += co_load_any(bias, bias_dtype, n);
       if (has1) v1 += co_load_any(bias, bias_dtype, n + 1);
     }
+    if (co_plain_act(epilogue)) { v0 = co_gelu(v0); v1 = co_gelu(v1); }
     const size_t o = (size_t)m * ldo + n;
     if (out_dtype == CO_BF16) {
       ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(v0);
@@ -704,7 +714,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
       }
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       if (tma_out) {
-        const int gated = epilogue;   // 0, or the gate's activation code
+        const int gated = co_gate_word(epilogue), act = co_plain_act(epilogue);
         const int step = gated ? 128 : 64;
 #pragma unroll 1
         for (int c0 = 0; c0 < BN; c0 += step, ++chunk) {
@@ -714,7 +724,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
             __syncwarp();
           }
           store_chunk_tma(tmem_base + ((unsigned)(quarter * 32) << 16) + (unsigned)(acc * BN + c0),
-                          bias && !gated ? bias_t + c0 : nullptr, gated,
+                          bias && !gated ? bias_t + c0 : nullptr, gated, act,
                           staging + (quarter * S::SBUF + chunk % S::SBUF) * 4096, &map_out,
                           gated ? (n0 + c0) >> 1 : n0 + c0, m0 + quarter * 32, lane);
         }
@@ -761,8 +771,8 @@ int launch_tc(const CUtensorMap& mx, const CUtensorMap& mw, const void* bias, in
   // bfloat16 output leaves through shared memory and TMA stores where whole chunks of 64 output
   // columns divide the tile.
   CUtensorMap mo = mx;
-  const int tma_out = !(partial && splits > 1) && BN % (epilogue != EPI_PLAIN ? 128 : 64) == 0 &&
-                      make_out_map(&mo, out, out_dtype, M, epilogue != EPI_PLAIN ? N / 2 : N, ldo) ? 1 : 0;
+  const int tma_out = !(partial && splits > 1) && BN % (co_gate_word(epilogue) != EPI_PLAIN ? 128 : 64) == 0 &&
+                      make_out_map(&mo, out, out_dtype, M, co_gate_word(epilogue) != EPI_PLAIN ? N / 2 : N, ldo) ? 1 : 0;
   auto kernel = gemm_tc_kernel<BN, STAGES>;
   constexpr int smem = Smem<BN, STAGES>::TOTAL;
   static bool configured = false;
@@ -868,7 +878,7 @@ int launch_tc_pair(const CUtensorMap& mx, const CUtensorMap& mw, const void* bia
   const long tiles = (long)((N + BN - 1) / BN) * ((M + 2 * BM - 1) / (2 * BM));
   const int pairs = (int)(tiles < slots ? tiles : slots);
   CUtensorMap mo = mx;
-  const int tma_out = make_out_map(&mo, out, out_dtype, M, epilogue != EPI_PLAIN ? N / 2 : N, ldo) ? 1 : 0;
+  const int tma_out = make_out_map(&mo, out, out_dtype, M, co_gate_word(epilogue) != EPI_PLAIN ? N / 2 : N, ldo) ? 1 : 0;
   cudaError_t le = co_launch_cluster(2, kernel, dim3(2 * pairs), dim3(192), (size_t)smem, stream, mx, mw, mo, tma_out, bias, bias_dtype,
                                      out, out_dtype, M, N, K, ldo, epilogue, status);
   if (le != cudaSuccess) CO_FAIL("gemm_tc_pair: launch failed: %s", cudaGetErrorString(le));
@@ -943,7 +953,7 @@ CO_EXPORT int coheryn_gemm_bf16_tc_pair(const void* x, const void* w, const void
 
 // x: [M, K] bfloat16 with row stride ldx; w: [N, K] bfloat16 contiguous; K and ldx multiples
 // of 8, bases 16-byte aligned.  epilogue 0: out[M, N] (+ bias); 1: gated SiLU over
-// interleaved rows of w, out[M, N/2].  status: device word that receives 11/12/13 if a
+// interleaved rows of w, out[M, N/2]; 16: out[M, N] = gelu(product + bias).  status: device word that receives 11/12/13 if a
 // bounded wait of the producer / the MMA issuer / the epilogue ran out (14: the issuer waiting
 // for a free accumulator in the persistent variant).  workspace: see above, may be null.
 CO_EXPORT int coheryn_gemm_bf16_tc(const void* x, const void* w, const void* bias, int bias_dtype, void* out,
@@ -952,7 +962,7 @@ CO_EXPORT int coheryn_gemm_bf16_tc(const void* x, const void* w, const void* bia
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || (K & 7) || (ldx & 7)) CO_FAIL("gemm_bf16_tc: K = %d and the row stride %ld must be multiples of 8", K, ldx);
   if (((uintptr_t)x & 15) || ((uintptr_t)w & 15)) CO_FAIL("gemm_bf16_tc: operands must be 16-byte aligned");
-  if (epilogue != 0 && (N & 1)) CO_FAIL("gemm_bf16_tc: gated epilogue needs an even number of rows");
+  if (co_gate_word(epilogue) != 0 && (N & 1)) CO_FAIL("gemm_bf16_tc: gated epilogue needs an even number of rows");
   if (!co_epilogue_known(epilogue)) CO_FAIL("gemm_bf16_tc: unknown epilogue %d", epilogue);
   if (status && pair_suits(M, N))
     return coheryn_gemm_bf16_tc_pair(x, w, bias, bias_dtype, out, out_dtype, M, N, K, ldx, ldo, epilogue, status, stream);
@@ -990,8 +1000,8 @@ CO_EXPORT int coheryn_gemm_bf16_tc_grouped(const void* x, const void* w, void* o
   if (M <= 0 || N <= 0 || G <= 0 || max_tiles <= 0) return 0;
   if (K <= 0 || (K & 7) || (ldx & 7)) CO_FAIL("gemm_bf16_tc_grouped: K = %d and the row stride %ld must be multiples of 8", K, ldx);
   if (((uintptr_t)x & 15) || ((uintptr_t)w & 15)) CO_FAIL("gemm_bf16_tc_grouped: operands must be 16-byte aligned");
-  if (epilogue != 0 && (N & 1)) CO_FAIL("gemm_bf16_tc_grouped: gated epilogue needs an even number of rows");
-  if (!co_epilogue_known(epilogue)) CO_FAIL("gemm_bf16_tc_grouped: unknown epilogue %d", epilogue);
+  if (co_gate_word(epilogue) != 0 && (N & 1)) CO_FAIL("gemm_bf16_tc_grouped: gated epilogue needs an even number of rows");
+  if (!co_epilogue_known(epilogue) || co_plain_act(epilogue)) CO_FAIL("gemm_bf16_tc_grouped: unknown epilogue %d", epilogue);
   if (!tile_group || !tile_row0 || !offsets || !n_tiles || !status) CO_FAIL("gemm_bf16_tc_grouped: the tile lists are missing");
   int bn = N >= 192 ? 256 : (N >= 96 ? 128 : 64);
   const bool narrow = g_bn == 128 && bn > 128;         // the tuning switch; the W map's box is the tile that runs
@@ -1051,7 +1061,7 @@ CO_EXPORT int coheryn_gemm_bf16_tc_pair(const void* x, const void* w, const void
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || (K & 7) || (ldx & 7)) CO_FAIL("gemm_bf16_tc_pair: K = %d and the row stride %ld must be multiples of 8", K, ldx);
   if (((uintptr_t)x & 15) || ((uintptr_t)w & 15)) CO_FAIL("gemm_bf16_tc_pair: operands must be 16-byte aligned");
-  if (epilogue != 0 && (N & 1)) CO_FAIL("gemm_bf16_tc_pair: gated epilogue needs an even number of rows");
+  if (co_gate_word(epilogue) != 0 && (N & 1)) CO_FAIL("gemm_bf16_tc_pair: gated epilogue needs an even number of rows");
   if (!co_epilogue_known(epilogue)) CO_FAIL("gemm_bf16_tc_pair: unknown epilogue %d", epilogue);
   if (!status) CO_FAIL("gemm_bf16_tc_pair: a status word is required");
   CUtensorMap mx, mw;

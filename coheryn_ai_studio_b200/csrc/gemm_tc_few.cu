@@ -127,7 +127,7 @@ gemm_tc_few_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               if (c0 + j < M) mine[(size_t)(c0 + j) * N] = __uint_as_float(r[j]) + bv;
-        } else if (epilogue != 0) {
+        } else if (co_gate_word(epilogue) != 0) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const float g = __uint_as_float(r[j]);
@@ -144,8 +144,9 @@ gemm_tc_few_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
           for (int j = 0; j < 16; ++j)
             if (c0 + j < M) {
               const size_t o = (size_t)(c0 + j) * ldo + n;
-              if (out_dtype == CO_BF16) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(__uint_as_float(r[j]) + bv);
-              else ((float*)out)[o] = __uint_as_float(r[j]) + bv;
+              const float x = __uint_as_float(r[j]) + bv, y = co_plain_act(epilogue) ? co_gelu(x) : x;
+              if (out_dtype == CO_BF16) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(y);
+              else ((float*)out)[o] = y;
             }
         }
       }
@@ -206,7 +207,7 @@ gemm_tc_few_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
       }
     }
     if (finish) {
-      if (epilogue != 0) {
+      if (co_gate_word(epilogue) != 0) {
         // features (2i, 2i+1) = (gate_i, up_i) sit in neighbouring lanes
         const int n_out = N >> 1;
 #pragma unroll
@@ -227,8 +228,9 @@ gemm_tc_few_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
         for (int j = 0; j < BT; ++j) {
           if (j >= M) break;
           const size_t o = (size_t)j * ldo + n;
-          if (out_dtype == CO_BF16) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(v[j] + bv);
-          else ((float*)out)[o] = v[j] + bv;
+          const float y = co_plain_act(epilogue) ? co_gelu(v[j] + bv) : v[j] + bv;
+          if (out_dtype == CO_BF16) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(y);
+          else ((float*)out)[o] = y;
         }
       }
     }
@@ -299,7 +301,7 @@ CO_EXPORT int coheryn_gemm_tc_few_splits(int N, int K) { return (N <= 0 || K <= 
 
 // x: [M, K] bfloat16 with row stride ldx, M <= 256 (above 64 rows a product whose K is cut needs defer = 1); w: [N, K] bfloat16 contiguous; K and ldx
 // multiples of 8, bases 16-byte aligned.  epilogue 0: out[M, N] (+ bias); 1: gated SiLU over
-// interleaved rows of w, out[M, N/2].  status: device word that receives 11/12/13 if a
+// interleaved rows of w, out[M, N/2]; 16: out[M, N] = gelu(product + bias).  status: device word that receives 11/12/13 if a
 // bounded wait of the producer / the MMA issuer / the epilogue ran out.  workspace: see above.
 // defer = 1 (epilogue 0 only) leaves the addition of the K splits to the consumer: out is then
 // float32 [splits][M][N], contiguous, the bias added to split 0, and no workspace is used.
@@ -311,10 +313,10 @@ CO_EXPORT int coheryn_gemm_bf16_tc_few(const void* x, const void* w, const void*
   if (M > 256) CO_FAIL("gemm_bf16_tc_few: M = %d exceeds 256", M);
   if (K <= 0 || (K & 7) || (ldx & 7)) CO_FAIL("gemm_bf16_tc_few: K = %d and the row stride %ld must be multiples of 8", K, ldx);
   if (((uintptr_t)x & 15) || ((uintptr_t)w & 15)) CO_FAIL("gemm_bf16_tc_few: operands must be 16-byte aligned");
-  if (epilogue != 0 && (N & 1)) CO_FAIL("gemm_bf16_tc_few: gated epilogue needs an even number of rows");
+  if (co_gate_word(epilogue) != 0 && (N & 1)) CO_FAIL("gemm_bf16_tc_few: gated epilogue needs an even number of rows");
   if (!co_epilogue_known(epilogue)) CO_FAIL("gemm_bf16_tc_few: unknown epilogue %d", epilogue);
   const int splits = few_splits(N, K);
-  if (defer && (epilogue != 0 || out_dtype != CO_F32)) CO_FAIL("gemm_bf16_tc_few: deferred splits are float32 and take no gate");
+  if (defer && (epilogue != 0 || out_dtype != CO_F32)) CO_FAIL("gemm_bf16_tc_few: deferred splits are float32 and take no gate and no activation");
   if (splits > 1 && !defer && (!workspace || workspace_floats < coheryn_gemm_tc_few_workspace_floats(M, N, K)))
     CO_FAIL("gemm_bf16_tc_few: the workspace of %ld floats is too small for M=%d N=%d K=%d", workspace_floats, M, N, K);
   const int bt = M <= 16 ? 16 : (M <= 32 ? 32 : (M <= 64 ? 64 : (M <= 128 ? 128 : 256)));

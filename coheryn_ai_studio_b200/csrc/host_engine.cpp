@@ -50,15 +50,17 @@ struct CacheBook {
   int page_size, num_pages, max_requests;
   bool prefix_reuse;
   std::vector<int> windows;                // per group, 0: none
+  std::vector<int> kept_first;             // per group: leading positions that stay although the window has passed them
   std::vector<std::unique_ptr<PagePool>> pools;
   SlotPool slots;
   std::unordered_map<std::string, Held> held;
   long long admissions = 0;
 
-  CacheBook(int ps, int np, int mr, bool reuse, int groups, const int* win)
+  CacheBook(int ps, int np, int mr, bool reuse, int groups, const int* win, const int* kept)
       : page_size(ps), num_pages(np), max_requests(mr), prefix_reuse(reuse), slots(mr) {
     for (int g = 0; g < groups; ++g) {
       windows.push_back(win ? win[g] : 0);
+      kept_first.push_back(kept ? std::max(kept[g], 0) : 0);
       pools.emplace_back(new PagePool(np));
       if (windows.back() > 0) prefix_reuse = false;    // pages behind a window cannot be found again
     }
@@ -146,7 +148,7 @@ struct CacheBook {
   }
 
   // The reserved tokens' keys and values are written: advance the length, hash the pages that
-  // became full, give back the pages a window has passed.
+  // became full, give back the pages a window has passed (but those of the leading positions it keeps).
   void commit(Held& r) {
     r.length = (int)r.tokens.size();
     if (prefix_reuse) {
@@ -162,7 +164,7 @@ struct CacheBook {
     for (size_t g = 0; g < pools.size(); ++g) {
       if (windows[g] <= 0) continue;
       const int upto = std::min(first_needed_block((int)g, r.length), (int)r.tables[g].size());
-      for (int b = 0; b < upto; ++b)
+      for (int b = (kept_first[g] + page_size - 1) / page_size; b < upto; ++b)
         if (r.tables[g][b] >= 0) {
           pools[g]->release(r.tables[g][b]);
           r.tables[g][b] = -1;
@@ -440,9 +442,9 @@ std::string str(const char* s) { return std::string(s ? s : ""); }
 
 // ---------------------------------------------------------------------------- C interface: book
 HOST_EXPORT void* coheryn_book_new(int page_size, int num_pages, int max_requests, int prefix_reuse, int groups,
-                                   const int* windows) {
+                                   const int* windows, const int* kept_first) {
   if (page_size < 1 || num_pages < 0 || max_requests < 0 || groups < 0) return nullptr;
-  return new CacheBook(page_size, num_pages, max_requests, prefix_reuse != 0, groups, windows);
+  return new CacheBook(page_size, num_pages, max_requests, prefix_reuse != 0, groups, windows, kept_first);
 }
 HOST_EXPORT void coheryn_book_delete(void* h) { delete static_cast<CacheBook*>(h); }
 HOST_EXPORT int coheryn_book_prefix_reuse(void* h) { return static_cast<CacheBook*>(h)->prefix_reuse ? 1 : 0; }

@@ -23,7 +23,7 @@
 //     one they weigh, hence <= 0.
 //
 // A row's order of additions is fixed by its place in its request's run, not by what else the step holds.
-#include "common.cuh"
+#include "linear_attention.cuh"
 
 namespace {
 
@@ -52,32 +52,10 @@ struct GlaArgs {
 __device__ __forceinline__ float gla_log_decay(float z, float inv_tau) {
   return (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau;
 }
-__device__ __forceinline__ float gla_gate(int act, float z) {
-  const float s = 1.0f / (1.0f + expf(-z));
-  return act == 1 ? z * s : s;
-}
 __device__ __forceinline__ void gla_store(const GlaArgs& A, size_t t, size_t col, float x) {
   if (A.out_dtype == CO_BF16) ((__nv_bfloat16*)A.out)[t * A.ldo + col] = __float2bfloat16_rn(x);
   else ((float*)A.out)[t * A.ldo + col] = x;
 }
-// Four neighbouring values of a row from column c on; columns >= n are zero.
-__device__ __forceinline__ float4 gla_load4(const float* row, int c, int n, bool vec) {
-  if (vec && c + 3 < n) return *reinterpret_cast<const float4*>(row + c);
-  float4 r;
-  r.x = c < n ? row[c] : 0.f;
-  r.y = c + 1 < n ? row[c + 1] : 0.f;
-  r.z = c + 2 < n ? row[c + 2] : 0.f;
-  r.w = c + 3 < n ? row[c + 3] : 0.f;
-  return r;
-}
-__device__ __forceinline__ void gla_store4(float* row, int c, int n, bool vec, float4 x) {
-  if (vec && c + 3 < n) { *reinterpret_cast<float4*>(row + c) = x; return; }
-  if (c < n) row[c] = x.x;
-  if (c + 1 < n) row[c + 1] = x.y;
-  if (c + 2 < n) row[c + 2] = x.z;
-  if (c + 3 < n) row[c + 3] = x.w;
-}
-
 // ------------------------------------------------------------------------------------------- few tokens per request
 // grid (H, B), 256 threads.  Thread (warp y, lane x) owns rows y, y + 8, .. of S and four neighbouring columns of a tile of
 // 128.  ROWS: rows a thread keeps in registers (0: the state stays in memory, for dk > 256).
@@ -120,7 +98,7 @@ __global__ void __launch_bounds__(256) gla_few_kernel(GlaArgs A, int L, bool vec
 #pragma unroll
       for (int i = 0; i < ROWS; ++i) {
         const int d = warp + 8 * i;
-        s[i] = d < dk && c < dv ? gla_load4(S + (size_t)d * dv, c, dv, vec) : make_float4(0.f, 0.f, 0.f, 0.f);
+        s[i] = d < dk && c < dv ? la_load4(S + (size_t)d * dv, c, dv, vec) : make_float4(0.f, 0.f, 0.f, 0.f);
       }
     }
     for (int t = 0; t < n; ++t) {
@@ -144,9 +122,9 @@ __global__ void __launch_bounds__(256) gla_few_kernel(GlaArgs A, int L, bool vec
         }
       } else if (c < dv) {
         for (int d = warp; d < dk; d += 8) {
-          float4 x = gla_load4(S + (size_t)d * dv, c, dv, vec);
+          float4 x = la_load4(S + (size_t)d * dv, c, dv, vec);
           step(x, d);
-          gla_store4(S + (size_t)d * dv, c, dv, vec, x);
+          la_store4(S + (size_t)d * dv, c, dv, vec, x);
         }
       }
       *reinterpret_cast<float4*>(part + warp * VT + 4 * lane) = o;
@@ -163,7 +141,7 @@ __global__ void __launch_bounds__(256) gla_few_kernel(GlaArgs A, int L, bool vec
 #pragma unroll
       for (int i = 0; i < ROWS; ++i) {
         const int d = warp + 8 * i;
-        if (d < dk && c < dv) gla_store4(S + (size_t)d * dv, c, dv, vec, s[i]);
+        if (d < dk && c < dv) la_store4(S + (size_t)d * dv, c, dv, vec, s[i]);
       }
     }
   }
@@ -173,7 +151,7 @@ __global__ void __launch_bounds__(256) gla_few_kernel(GlaArgs A, int L, bool vec
     ss = co_warp_sum(ss);
     const float sc = 1.0f / sqrtf(ss / (float)dv + A.eps);
     for (int c = lane; c < dv; c += 32) {
-      const float gate = gla_gate(A.gate_act, A.g[(size_t)(t0 + t) * A.ldg + (size_t)h * dv + c]);
+      const float gate = la_gate(A.gate_act, A.g[(size_t)(t0 + t) * A.ldg + (size_t)h * dv + c]);
       gla_store(A, t0 + t, (size_t)h * dv + c, ((os[t * dv + c] * sc) * co_load_any(A.norm_w, A.norm_dtype, c)) * gate);
     }
   }
@@ -244,7 +222,7 @@ __global__ void __launch_bounds__(256) gla_chunk_state_kernel(GlaArgs A, bool ve
 #pragma unroll
   for (int i = 0; i < CH * (VT / 4) / 256; ++i) {
     const int e = threadIdx.x + 256 * i, t = e / (VT / 4), c4 = e % (VT / 4);
-    const float4 x = t < ck.n ? gla_load4(A.v + ((size_t)ck.first + t) * A.ldv + (size_t)h * dv, c0 + 4 * c4, dv, vec)
+    const float4 x = t < ck.n ? la_load4(A.v + ((size_t)ck.first + t) * A.ldv + (size_t)h * dv, c0 + 4 * c4, dv, vec)
                               : make_float4(0.f, 0.f, 0.f, 0.f);
     *reinterpret_cast<float4*>(Vs + t * VT + 4 * c4) = x;
   }
@@ -294,7 +272,7 @@ __global__ void __launch_bounds__(256) gla_chunk_state_kernel(GlaArgs A, bool ve
   for (int i = 0; i < 8; ++i) {
     const int d = d0 + warp * 8 + i;
     if (d < dk && c0 + 4 * lane < dv)
-      gla_store4(dst + (size_t)d * dv, c0 + 4 * lane, dv, vs, make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]));
+      la_store4(dst + (size_t)d * dv, c0 + 4 * lane, dv, vs, make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]));
   }
 }
 
@@ -479,10 +457,10 @@ __global__ void __launch_bounds__(256, 2) gla_chunk_out_kernel(GlaArgs A, bool v
         const int row = warp + 8 * j, c = c0 + 4 * lane;
         next[j] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (i < n_slices) {
-          if (i * SL + row < dk && c < dv) next[j] = gla_load4(S0 + (size_t)(i * SL + row) * dv, c, dv, vec_s);
+          if (i * SL + row < dk && c < dv) next[j] = la_load4(S0 + (size_t)(i * SL + row) * dv, c, dv, vec_s);
         } else {
           const int t = (i - n_slices) * SL + row;
-          if (t < ck.n && c < dv) next[j] = gla_load4(V0 + (size_t)t * A.ldv, c, dv, vec);
+          if (t < ck.n && c < dv) next[j] = la_load4(V0 + (size_t)t * A.ldv, c, dv, vec);
         }
       }
     };
@@ -525,7 +503,7 @@ __global__ void __launch_bounds__(256, 2) gla_chunk_out_kernel(GlaArgs A, bool v
 #pragma unroll
       for (int m = 0; m < 8; ++m)
         if (warp * 8 + m < ck.n && c < dv)
-          gla_store4(A.o_raw + (orow + m) * ((size_t)A.H * dv) + (size_t)h * dv, c, dv, vec_s,
+          la_store4(A.o_raw + (orow + m) * ((size_t)A.H * dv) + (size_t)h * dv, c, dv, vec_s,
                      make_float4(acc[m][0], acc[m][1], acc[m][2], acc[m][3]));
       continue;
     }
@@ -536,7 +514,7 @@ __global__ void __launch_bounds__(256, 2) gla_chunk_out_kernel(GlaArgs A, bool v
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         if (c + e >= dv) break;
-        const float gate = gla_gate(A.gate_act, A.g[(orow + m) * A.ldg + (size_t)h * dv + c + e]);
+        const float gate = la_gate(A.gate_act, A.g[(orow + m) * A.ldg + (size_t)h * dv + c + e]);
         gla_store(A, orow + m, (size_t)h * dv + c + e, ((acc[m][e] * sc) * co_load_any(A.norm_w, A.norm_dtype, c + e)) * gate);
       }
     }
@@ -550,7 +528,7 @@ __global__ void __launch_bounds__(256, 2) gla_chunk_out_kernel(GlaArgs A, bool v
       for (int e = 0; e < 4 && c0 + e < dv; ++e) {
         const int c = c0 + e;
         const float o = A.o_raw[(orow + m) * ((size_t)A.H * dv) + (size_t)h * dv + c];
-        const float gate = gla_gate(A.gate_act, A.g[(orow + m) * A.ldg + (size_t)h * dv + c]);
+        const float gate = la_gate(A.gate_act, A.g[(orow + m) * A.ldg + (size_t)h * dv + c]);
         gla_store(A, orow + m, (size_t)h * dv + c, ((o * sc) * co_load_any(A.norm_w, A.norm_dtype, c)) * gate);
       }
     }

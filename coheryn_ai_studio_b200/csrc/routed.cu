@@ -509,7 +509,7 @@ CO_EXPORT int coheryn_grouped_linear(const void* A, int a_dtype, long lda, long 
   const bool routed = tile_group != nullptr;
   if (routed && (!tile_row0 || !offsets || !n_tiles || max_tiles < 1)) CO_FAIL("grouped_linear: routed groups need their tile lists");
   if (!routed && M <= 0) return 0;
-  if (epilogue && !co_epilogue_known(epilogue)) CO_FAIL("grouped_linear: unknown epilogue %d", epilogue);
+  if (epilogue && (!co_epilogue_known(epilogue) || co_plain_act(epilogue))) CO_FAIL("grouped_linear: unknown epilogue %d", epilogue);
   if (epilogue && (N & 1)) CO_FAIL("grouped_linear: a gated epilogue needs an even number of columns");
   GroupedArgs a{A, lda, a_col, W, w_group, C, ldc, c_col, gather, tile_group, tile_row0, offsets, n_tiles,
                 factor, factor_ld, factor_sigmoid, M, N, K, G, epilogue ? 1 : 0, epilogue};

@@ -57,7 +57,7 @@ def total_launch_count() -> int:
     """Kernel launches made through every library of this package that is loaded."""
     n = launch_count()
     for lib in list(_attn_libs.values()) + list(_maps_libs.values()) + list(_pooled_tc_libs.values()) + [
-            l for l in (_recurrent, _variants, _routed, _linear_recurrence, _pooled, _linear_attention) if l is not None]:
+            l for l in (_recurrent, _variants, _routed, _linear_recurrence, _pooled, _linear_attention, _lightning) if l is not None]:
         n += int(lib.coheryn_launch_count())
     return n
 
@@ -467,8 +467,9 @@ def qkv_rope_parts(x: torch.Tensor, w_qkv: torch.Tensor, b_qkv: Optional[torch.T
     return q
 
 
-def gemm_simt(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor) -> None:
-    """out = x @ w.T (+ bias) with float32 FMA accumulation (no tensor cores)."""
+def gemm_simt(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, act: int = 0) -> None:
+    """out = x @ w.T (+ bias), passed through the plain activation ``act`` (see ``PLAIN_ACTIVATIONS``), with float32 FMA
+    accumulation (no tensor cores)."""
     _dev(x, w, bias, out)
     M, K = x.shape
     N = w.shape[0]
@@ -480,7 +481,7 @@ def gemm_simt(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], ou
     _check(lib, lib.coheryn_gemm_simt(
         _ptr(x), c_int(_code(x)), _ptr(w), c_int(_code(w)), _ptr(bias),
         c_int(_code(bias) if bias is not None else F32), _ptr(out), c_int(_code(out)), c_int(M),
-        c_int(N), c_int(K), c_long(x.stride(0)), c_long(out.stride(0)), _stream()))
+        c_int(N), c_int(K), c_long(x.stride(0)), c_long(out.stride(0)), c_int(act), _stream()))
 
 
 def attention_simple(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
@@ -549,8 +550,9 @@ def apply_penalties(logits, rows, ids, counts, rep, freq, pres) -> None:
 
 
 # ------------------------------------------------------------------------------------
-def gemm_bf16_small(x, w, bias, out, gated: int = 0) -> None:
-    """Tensor-core product for at most 64 rows (decode); see csrc/gemm_bf16_small.cu."""
+def gemm_bf16_small(x, w, bias, out, gated: int = 0, epilogue: int = 0) -> None:
+    """Tensor-core product for at most 64 rows (decode); see csrc/gemm_bf16_small.cu.  ``gated`` (of all these products):
+    the word of a gated epilogue over interleaved rows of w; ``epilogue``: the word of a plain activation."""
     _dev(x, w, bias, out)
     M, K = x.shape
     N = w.shape[0]
@@ -560,7 +562,7 @@ def gemm_bf16_small(x, w, bias, out, gated: int = 0) -> None:
     _check(lib, lib.coheryn_gemm_bf16_small(
         _ptr(x), _ptr(w), _ptr(bias), c_int(_code(bias) if bias is not None else F32), _ptr(out),
         c_int(_code(out)), c_int(M), c_int(N), c_int(K), c_long(x.stride(0)), c_long(out.stride(0)),
-        c_int(int(gated)), _stream()))
+        c_int(int(gated or epilogue)), _stream()))
 
 
 # Up to this many rows the weight-streaming mma.sync kernel runs; beyond it the TMA/tcgen05
@@ -605,7 +607,7 @@ def selftest_bounded_wait(device, tries: int = 300, code: int = 19) -> None:
     _check(lib, lib.coheryn_selftest_bounded_wait(_ptr(tc_status(device)), ctypes.c_uint(tries), c_int(code), _stream()))
 
 
-def gemm_bf16_tc(x, w, bias, out, gated: int = 0) -> None:
+def gemm_bf16_tc(x, w, bias, out, gated: int = 0, epilogue: int = 0) -> None:
     """TMA + tcgen05 product for many rows (prompt portions); see csrc/gemm_tc.cu."""
     _dev(x, w, bias, out)
     M, K = x.shape
@@ -618,7 +620,7 @@ def gemm_bf16_tc(x, w, bias, out, gated: int = 0) -> None:
     _check(lib, lib.coheryn_gemm_bf16_tc(
         _ptr(x), _ptr(w), _ptr(bias), c_int(_code(bias) if bias is not None else F32), _ptr(out),
         c_int(_code(out)), c_int(M), c_int(N), c_int(K), c_long(x.stride(0)), c_long(out.stride(0)),
-        c_int(int(gated)), _ptr(tc_status(x.device)), _ptr(workspace), c_long(floats), _stream()))
+        c_int(int(gated or epilogue)), _ptr(tc_status(x.device)), _ptr(workspace), c_long(floats), _stream()))
 
 
 def set_gemm_pairs(on: bool) -> None:
@@ -632,7 +634,7 @@ def gemm_tc_splits(M: int, N: int, K: int) -> int:
     return max(1, _tc_workspace_floats(M, N, K) // (M * N))
 
 
-def gemm_bf16_tc_pair(x, w, bias, out, gated: int = 0) -> None:
+def gemm_bf16_tc_pair(x, w, bias, out, gated: int = 0, epilogue: int = 0) -> None:
     """The many-rows product by pairs of CTAs sharing 256 x 256 tiles (tcgen05 cta_group::2);
     see gemm_tc_pair_kernel in csrc/gemm_tc.cu."""
     _dev(x, w, bias, out)
@@ -644,7 +646,7 @@ def gemm_bf16_tc_pair(x, w, bias, out, gated: int = 0) -> None:
     _check(lib, lib.coheryn_gemm_bf16_tc_pair(
         _ptr(x), _ptr(w), _ptr(bias), c_int(_code(bias) if bias is not None else F32), _ptr(out),
         c_int(_code(out)), c_int(M), c_int(N), c_int(K), c_long(x.stride(0)), c_long(out.stride(0)),
-        c_int(int(gated)), _ptr(tc_status(x.device)), _stream()))
+        c_int(int(gated or epilogue)), _ptr(tc_status(x.device)), _stream()))
 
 
 _few_workspaces = {}
@@ -680,7 +682,7 @@ def _few_workspace_floats(M: int, N: int, K: int) -> int:
     return int(core().coheryn_gemm_tc_few_workspace_floats(c_int(M), c_int(N), c_int(K)))
 
 
-def gemm_bf16_tc_few(x, w, bias, out, gated: int = 0, defer: bool = False) -> None:
+def gemm_bf16_tc_few(x, w, bias, out, gated: int = 0, defer: bool = False, epilogue: int = 0) -> None:
     """TMA + tcgen05 product for at most 64 rows with the features on the accumulator's
     lanes (decode, short portions); see csrc/gemm_tc_few.cu.  ``defer``: ``out`` is a float32
     stack [splits, M, N] of the K slices' sums, left for the consumer to add."""
@@ -691,7 +693,7 @@ def gemm_bf16_tc_few(x, w, bias, out, gated: int = 0, defer: bool = False) -> No
     assert x.stride(1) == 1 and out.stride(-1) == 1
     lib = core()
     if defer:
-        assert not gated and out.dtype == torch.float32 and out.is_contiguous()
+        assert not gated and not epilogue and out.dtype == torch.float32 and out.is_contiguous()
         assert out.shape == (few_splits(N, K), M, N)
         floats = 0
     else:
@@ -701,7 +703,7 @@ def gemm_bf16_tc_few(x, w, bias, out, gated: int = 0, defer: bool = False) -> No
     _check(lib, lib.coheryn_gemm_bf16_tc_few(
         _ptr(x), _ptr(w), _ptr(bias), c_int(_code(bias) if bias is not None else F32), _ptr(out),
         c_int(_code(out)), c_int(M), c_int(N), c_int(K), c_long(x.stride(0)), c_long(out.stride(-2)),
-        c_int(int(gated)), _ptr(tc_status(x.device)), _ptr(workspace),
+        c_int(int(gated or epilogue)), _ptr(tc_status(x.device)), _ptr(workspace),
         c_long(workspace.numel() if workspace is not None else 0), c_int(1 if defer else 0), _stream()))
 
 
@@ -769,14 +771,16 @@ def _small_ok(x, w) -> bool:
 
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
            out_dtype: Optional[torch.dtype] = None, out: Optional[torch.Tensor] = None,
-           partial_ok: bool = False) -> torch.Tensor:
+           partial_ok: bool = False, activation: Optional[str] = None) -> torch.Tensor:
     """y = x @ w.T (+ bias), float32 accumulation.  float32 operands use FMA on the CUDA
     cores (no reduced-precision tensor mode); bfloat16 operands use the tensor-core
     kernels where the shape allows and the FMA kernel otherwise.  With ``partial_ok`` the
     result may come as a float32 stack [splits, M, N] of partial sums whose addition is left
-    to the consumer (``add_rmsnorm`` takes such a stack as its delta)."""
+    to the consumer (``add_rmsnorm`` takes such a stack as its delta).  ``activation``: y passes this function (a name of
+    ``PLAIN_ACTIVATIONS``) in the product's epilogue, in float32."""
     M, N = x.shape[0], w.shape[0]
-    if (partial_ok and out is None and M and w.shape[1] >= (DEFER_MIN_K_WIDE if M > SMALL_M_SHORT else DEFER_MIN_K)
+    act = plain_activation_code(activation)
+    if (partial_ok and not act and out is None and M and w.shape[1] >= (DEFER_MIN_K_WIDE if M > SMALL_M_SHORT else DEFER_MIN_K)
             and _few_shape_ok(x, w, FEW_DEFER_M)):
         splits = few_splits(N, w.shape[1])
         if splits > 1:
@@ -788,14 +792,29 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     if M == 0:
         return out
     if _few_ok(x, w):
-        gemm_bf16_tc_few(x, w, bias, out)
+        gemm_bf16_tc_few(x, w, bias, out, epilogue=act)
     elif _small_ok(x, w):
-        gemm_bf16_small(x, w, bias, out)
+        gemm_bf16_small(x, w, bias, out, epilogue=act)
     elif _tc_ok(x, w):
-        gemm_bf16_tc(x, w, bias, out)
+        gemm_bf16_tc(x, w, bias, out, epilogue=act)
     else:
-        gemm_simt(x, w, bias, out)
+        gemm_simt(x, w, bias, out, act)
     return out
+
+
+# Activations of a product's own result (one output per column), by the epilogue word that the kernels take: the words
+# from 16 on, beside those of the gates below.
+PLAIN_ACTIVATIONS = {"gelu": 16}
+
+
+def plain_activation_code(activation: Optional[str]) -> int:
+    if activation is None:
+        return 0
+    try:
+        return PLAIN_ACTIVATIONS[activation]
+    except KeyError:
+        raise KernelError(f"the epilogue of the matrix products is not built for activation {activation!r} "
+                          f"(built: {', '.join(sorted(PLAIN_ACTIVATIONS))})") from None
 
 
 def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, step,
@@ -1194,18 +1213,24 @@ def variants():
 
 def unit_norm_rope_kv_write(q, k, v, q_weight, k_weight, eps: float, positions, freq, rot: int, rot_scale: float, slots,
                             k_cache, v_cache, q_units: int, k_units: int, num_kv_heads: int, dk: int, dv: int,
-                            page_size: int, dtype: torch.dtype) -> torch.Tensor:
+                            page_size: int, dtype: torch.dtype, whole_norm: bool = False, v_first: Optional[torch.Tensor] = None,
+                            mix: float = 0.0) -> torch.Tensor:
     """Queries and keys in units of ``dk`` channels (a head has one unit per score map): each unit divided by its root
     mean square and multiplied by a weight [dk] shared by the units (skipped when ``q_weight`` is None), then its first
     ``rot`` channels rotated by the token's position (pairs (i, i + rot/2); ``freq`` float32 [rot/2, 2] holds each pair's
     frequency as a high and a low part, angle = position * frequency; cos and sin are multiplied by ``rot_scale``).  Keys
     ([page, kv head, slot, k_units / kv heads * dk]) and values ([page, kv head, slot, dv]) go to the cache at ``slots``
-    (None: only the queries are made; k and v are not read).  q, k, v: float32 with one row stride.  Returns q
-    [T, q_units * dk] in ``dtype``."""
-    _dev(q, k, v, q_weight, k_weight, positions, freq, slots, k_cache, v_cache)
+    (None: only the queries are made; k and v are not read).  q, k, v: float32 with one row stride.  ``whole_norm``: the
+    root mean square is that of ALL channels of q (and of k), and the weights have one entry per channel ([units * dk]).
+    ``v_first`` (float32 [T, kv heads * dv]): what is cached is (1 - mix) v + mix v_first.  Returns q [T, q_units * dk] in
+    ``dtype``."""
+    _dev(q, k, v, q_weight, k_weight, positions, freq, slots, k_cache, v_cache, v_first)
     _f32(q, "q")
     T = q.shape[0]
     assert q.shape[1] == q_units * dk
+    if v_first is not None:
+        _f32(v_first, "v_first")
+        assert slots is not None and v_first.shape == (T, num_kv_heads * dv)
     if slots is not None:
         _f32(k, "k"); _f32(v, "v"); _i32(slots, "slots")
         assert q.stride(0) == k.stride(0) == v.stride(0)
@@ -1215,7 +1240,8 @@ def unit_norm_rope_kv_write(q, k, v, q_weight, k_weight, eps: float, positions, 
         assert tuple(v_cache.shape[1:]) == (num_kv_heads, page_size, dv)
     normalise = q_weight is not None
     if normalise:
-        assert q_weight.numel() == dk and k_weight.numel() == dk and q_weight.dtype == k_weight.dtype
+        assert q_weight.numel() == (q_units * dk if whole_norm else dk) and k_weight.numel() == (k_units * dk if whole_norm else dk)
+        assert q_weight.dtype == k_weight.dtype and q_weight.is_contiguous() and k_weight.is_contiguous()
     if rot:
         _i32(positions, "positions")
         assert freq.dtype == torch.float32 and freq.is_contiguous() and tuple(freq.shape) == (rot // 2, 2)
@@ -1223,10 +1249,11 @@ def unit_norm_rope_kv_write(q, k, v, q_weight, k_weight, eps: float, positions, 
     lib = variants()
     _check(lib, lib.coheryn_unit_norm_rope_kv_write(
         _ptr(q), _ptr(k), _ptr(v), c_long(q.stride(0)), _ptr(q_weight), _ptr(k_weight),
-        c_int(_code(q_weight) if normalise else F32), c_float(eps), c_int(1 if normalise else 0), _ptr(positions), _ptr(freq),
-        c_int(rot), c_float(rot_scale), _ptr(q_out), c_int(_CODES[dtype]), c_long(q_out.stride(0)), _ptr(slots),
-        _ptr(k_cache), _ptr(v_cache), c_int(T), c_int(q_units), c_int(k_units), c_int(num_kv_heads), c_int(dk), c_int(dv),
-        c_int(page_size), _stream()))
+        c_int(_code(q_weight) if normalise else F32), c_float(eps), c_int((2 if whole_norm else 1) if normalise else 0),
+        _ptr(positions), _ptr(freq), c_int(rot), c_float(rot_scale), _ptr(q_out), c_int(_CODES[dtype]), c_long(q_out.stride(0)),
+        _ptr(slots), _ptr(k_cache), _ptr(v_cache), c_int(T), c_int(q_units), c_int(k_units), c_int(num_kv_heads), c_int(dk),
+        c_int(dv), c_int(page_size), _ptr(v_first), c_long(v_first.stride(0) if v_first is not None else 0), c_float(1.0 - mix),
+        c_float(mix), _stream()))
     return q_out
 
 
@@ -1261,10 +1288,10 @@ def attention_maps(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_
                    num_heads: int, num_kv_heads: int, dk: int, dv: int, maps: int, page_size: int, window: Optional[int],
                    chunk: Optional[int], sink: bool, scale: float, lam: float, head_norm: bool, eps: float,
                    out_scale: float, force_simple: bool = False, sink_scores: Optional[torch.Tensor] = None,
-                   values_in_keys: bool = False, head_gates: Optional[torch.Tensor] = None) -> None:
+                   values_in_keys: bool = False, head_gates: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
     """Attention of every token of the step over its request's cache pages of ``group`` with ``maps`` score maps per
     head (output a_0 - lam * a_1 for two), a mask by chunks (``chunk``: position i sees j <= i with i // chunk ==
-    j // chunk), by a window or causal, an optional sink term in the softmax's denominator, the head's output divided
+    j // chunk), by a window (beside which the first ``keep_first`` positions stay in sight) or causal, an optional sink term in the softmax's denominator, the head's output divided
     by its root mean square over dv (``head_norm``) and multiplied by ``out_scale``.  q [T, heads * maps * dk],
     out [T, heads * dv]; float32 arithmetic on either storage type.  ``sink_scores`` (float32 [heads]): the sink's score
     per head instead of 0.  ``values_in_keys``: the values are the first dv channels of the key rows (``v_cache`` is not
@@ -1299,13 +1326,13 @@ def attention_maps(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_
         B = len(q_lens)
         single = any(n == 1 for n in q_lens)
         floats = int(lib.coheryn_maps_scratch_floats(c_int(B), c_int(num_heads), c_int(step.max_kv_len), c_int(window or 0),
-                                                     c_int(chunk or 0))) if single else 0
+                                                     c_int(chunk or 0), c_int(keep_first))) if single else 0
         scratch = torch.empty(floats, dtype=torch.float32, device=q.device) if floats else None
         _check(lib, lib.coheryn_attention_maps_bf16(
             _ptr(q), c_long(q.stride(0)), _ptr(out), c_long(out.stride(0)), _ptr(k_cache), _ptr(v_cache), _ptr(block_tables),
             c_int(block_tables.shape[1]), _ptr(step.cu_q), _ptr(step.kv_lens), c_int(B), c_int(num_heads), c_int(num_kv_heads),
-            c_int(page_size), c_int(window or 0), c_int(chunk or 0), c_int(1 if sink else 0), c_float(scale), c_float(lam),
-            c_int(1 if head_norm else 0), c_float(eps), c_float(out_scale), c_int(max(q_lens)), c_int(step.max_kv_len),
+            c_int(page_size), c_int(window or 0), c_int(chunk or 0), c_int(keep_first), c_int(1 if sink else 0), c_float(scale),
+            c_float(lam), c_int(1 if head_norm else 0), c_float(eps), c_float(out_scale), c_int(max(q_lens)), c_int(step.max_kv_len),
             c_int(1 if any(n == 1 for n in q_lens) else 0), c_int(1 if any(n > 1 for n in q_lens) else 0), _ptr(scratch),
             c_long(floats), _ptr(sink_scores), _ptr(head_gates), c_long(head_gates.stride(0) if head_gates is not None else 0),
             _stream()))
@@ -1315,8 +1342,8 @@ def attention_maps(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_
         _ptr(q), c_long(q.stride(0)), _ptr(out), c_long(out.stride(0)), _ptr(k_cache), _ptr(v_cache), c_int(_code(q)),
         _ptr(block_tables), c_int(block_tables.shape[1]), _ptr(step.token_req), _ptr(step.positions), c_int(T),
         c_int(num_heads), c_int(num_kv_heads), c_int(dk), c_int(dv), c_int(maps), c_int(page_size), c_int(window or 0),
-        c_int(chunk or 0), c_int(1 if sink else 0), c_float(scale), c_float(lam), c_int(1 if head_norm else 0), c_float(eps),
-        c_float(out_scale), _ptr(sink_scores), c_int(1 if values_in_keys else 0), _stream()))
+        c_int(chunk or 0), c_int(keep_first), c_int(1 if sink else 0), c_float(scale), c_float(lam), c_int(1 if head_norm else 0),
+        c_float(eps), c_float(out_scale), _ptr(sink_scores), c_int(1 if values_in_keys else 0), _stream()))
     if head_gates is not None:
         head_gate(out, head_gates, num_heads)
 
@@ -1877,3 +1904,63 @@ def gated_linear_attention(q, k, v, gate, a1, a2, a2_bias, tau: float, q_scale: 
         _ptr(norm_weight), c_int(_code(norm_weight)), c_float(eps), c_int({"sigmoid": 0, "silu": 1}[gate_activation]), _ptr(out),
         c_int(_code(out)), c_long(out.stride(0)), _ptr(scratch), c_long(floats), c_int(T), c_int(B), c_int(heads), c_int(dk), c_int(dv),
         c_int(longest), c_int(few), _stream()))
+
+
+# ------------------------------------------------------------------------------------
+# Linear attention with a constant decay per head (csrc/lightning_attention.cu, a library of its own that is compiled when
+# a model with such a mixer is first run).
+_lightning = None
+
+
+def lightning():
+    global _lightning
+    if _lightning is None:
+        lib = build.lightning_library()
+        lib.coheryn_last_error.restype = ctypes.c_char_p
+        lib.coheryn_launch_count.restype = ctypes.c_ulonglong
+        lib.coheryn_lightning_scratch.restype = ctypes.c_long
+        if int(lib.coheryn_lightning_chunk()) != LIGHTNING_CHUNK:
+            raise KernelError("the linear attention library was built for another chunk length")
+        _lightning = lib
+    return _lightning
+
+
+LIGHTNING_CHUNK = 64      # tokens per chunk of the kernels for prompt portions
+# A step whose longest run of tokens is at most this takes the tokens one by one with the state in registers.
+LIGHTNING_FEW_TOKENS = int(os.environ.get("COHERYN_LIGHTNING_FEW_TOKENS", "8"))
+
+
+def decay_powers(decay, device) -> torch.Tensor:
+    """float32 [heads, 2, LIGHTNING_CHUNK + 1]: every head's decay to the powers 0 .., and those less 1, made in float64."""
+    a = torch.as_tensor(decay, dtype=torch.float64).reshape(-1, 1)
+    n = torch.arange(LIGHTNING_CHUNK + 1, dtype=torch.float64)
+    less = torch.where(a > 0, torch.expm1(n * torch.log(a.clamp(min=1e-300))), torch.where(n == 0, 0.0, -1.0))
+    return torch.stack([less + 1.0, less], dim=1).to(torch.float32).contiguous().to(device)
+
+
+def lightning_attention(q, k, v, gate, powers: torch.Tensor, silu: bool, state: torch.Tensor, step, heads: int, dk: int, dv: int,
+                        norm_weight: torch.Tensor, eps: float, out: torch.Tensor, gate_activation: str = "sigmoid",
+                        out_scale: float = 1.0) -> None:
+    """S_t = a S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per request and head with a constant a per head (``powers``: see
+    :func:`decay_powers`); ``silu``: q, k and v pass SiLU first; out_t = o_t / rms(o_t) * norm_weight * act(gate_t) *
+    out_scale, the root mean square over all heads together.  ``q``, ``k`` float32 [T, heads * dk], ``v``, ``gate`` float32
+    [T, heads * dv] (column slices are fine); ``state`` float32 [slots, heads * dk * dv] (rows may be strided), read at a
+    request's first token of the step and written behind its last; ``norm_weight`` [heads * dv]; ``out`` [T, heads * dv]."""
+    _dev(q, k, v, gate, powers, state, norm_weight, out, step.cu_q, step.state_slots)
+    T = q.shape[0]
+    for name, t, n in (("q", q, heads * dk), ("k", k, heads * dk), ("v", v, heads * dv), ("gate", gate, heads * dv)):
+        assert t.dtype == torch.float32 and t.stride(1) == 1 and t.shape == (T, n), name
+    assert norm_weight.shape == (heads * dv,) and norm_weight.is_contiguous()
+    assert powers.dtype == torch.float32 and powers.is_contiguous() and tuple(powers.shape) == (heads, 2, LIGHTNING_CHUNK + 1)
+    _f32(state, "state")
+    assert state.shape[1] == heads * dk * dv and state.stride(1) == 1 and out.shape == (T, heads * dv) and out.stride(1) == 1
+    lib = lightning()
+    B, longest, few = step.num_requests, int(step.max_q_len), LIGHTNING_FEW_TOKENS
+    floats = int(lib.coheryn_lightning_scratch(c_int(T), c_int(B), c_int(longest), c_int(few), c_int(heads), c_int(dk), c_int(dv)))
+    scratch = torch.empty(floats, dtype=torch.float32, device=q.device)
+    _check(lib, lib.coheryn_lightning(
+        _ptr(q), c_long(q.stride(0)), _ptr(k), c_long(k.stride(0)), _ptr(v), c_long(v.stride(0)), _ptr(gate), c_long(gate.stride(0)),
+        _ptr(powers), c_int(1 if silu else 0), _ptr(state), c_long(state.stride(0)), _ptr(step.cu_q), _ptr(step.state_slots),
+        _ptr(norm_weight), c_int(_code(norm_weight)), c_float(eps), c_int({"sigmoid": 0, "silu": 1}[gate_activation]),
+        c_float(out_scale), _ptr(out), c_int(_code(out)), c_long(out.stride(0)), _ptr(scratch), c_long(floats), c_int(T), c_int(B),
+        c_int(heads), c_int(dk), c_int(dv), c_int(longest), c_int(few), _stream()))

@@ -232,12 +232,20 @@ class MapsAttention(Mixer):
     multiplied by 1 - ``lambda_init``.  Options, all independent of the number of maps:
 
     * ``qk_norm = "head"``: every query and key map is divided by its root mean square over ``head_dim`` and multiplied
-      by a weight (``q.norm``, ``k.norm``: [head_dim], shared by the heads);
+      by a weight (``q.norm``, ``k.norm``: [head_dim], shared by the heads); ``"projection"``: the WHOLE query projection
+      (all heads at once), and the whole key projection, by its root mean square, with a weight per channel;
+    * ``qkv_bias``: biases on the three projections (tensors ``q.b``, ``k.b``, ``v.b``);
     * ``position``: a rotation of the first ``rotary_dim`` channels of every map of q and k (none: positions do not
-      enter the scores);
+      enter the scores; pairs of neighbouring channels become halves by a permutation of the projections' rows when the
+      weights are bound);
     * mask: ``chunk`` (i sees j <= i with i // chunk == j // chunk, counted from position 0 of the sequence), else
-      ``window`` (i - j < window), else every j <= i;
-    * ``sink``: the softmax's denominator has one more term exp(0), which carries no value;
+      ``window`` (i - j < window; the first ``keep_first`` positions of the sequence stay in sight, and cached, when the
+      window has passed them), else every j <= i;
+    * ``sink``: the softmax's denominator has one more term exp(0), which carries no value; ``learned_sink``: the term is
+      exp(sink_h), a learned score per head (tensor ``sink``);
+    * ``gate``: head h's output is multiplied by sigmoid(g x)_h (tensor ``g`` [heads, width], the projections' input);
+    * ``value_mix``: "first" keeps the layer's values for the later layers of the same step, "later" replaces its own by
+      (1 - lambda) v + lambda v_first before they are cached (tensor ``vmix``, one number; the first layer's is unused);
     * ``head_norm``: the division by the root mean square for a single map too; ``out_factor`` multiplies the output.
 
     A layer may read the keys (as the cache holds them, rotated) and values that an earlier one wrote; it then has no
@@ -249,7 +257,9 @@ class MapsAttention(Mixer):
                  v_head_dim: Optional[int], scale: float, maps: int = 1, lambda_init: Optional[float] = None,
                  chunk: Optional[int] = None, window: Optional[int] = None, sink: bool = False, qk_norm: Optional[str] = None,
                  head_norm: Optional[bool] = None, out_factor: float = 1.0, eps: float = 1e-6, own_kv: bool = True,
-                 float32_output: bool = False, out_scale: float = 1.0, position: Optional[Position] = None):
+                 float32_output: bool = False, out_scale: float = 1.0, position: Optional[Position] = None,
+                 keep_first: int = 0, qkv_bias: bool = False, learned_sink: bool = False, gate: bool = False,
+                 value_mix: Optional[str] = None):
         super().__init__(runtime)
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads do not divide into {num_kv_heads} kv heads")
@@ -257,8 +267,14 @@ class MapsAttention(Mixer):
             raise ValueError("an attention head has one score map or two")
         if maps == 2 and lambda_init is None:
             raise ValueError("two score maps need the constant of their difference (lambda_init)")
-        if qk_norm not in (None, "head"):
-            raise ValueError(f"qk_norm {qk_norm!r} is not built here (None, 'head')")
+        if qk_norm not in (None, "head", "projection"):
+            raise ValueError(f"qk_norm {qk_norm!r} is not built here (None, 'head', 'projection')")
+        if value_mix not in (None, "first", "later"):
+            raise ValueError(f"value_mix {value_mix!r} is not built (None, 'first', 'later')")
+        if keep_first < 0 or (keep_first and (window is None or chunk is not None)):
+            raise ValueError("kept first positions are those that a window would leave behind")
+        if not own_kv and (qkv_bias or value_mix):
+            raise ValueError("biases and mixed values belong to an attention with key and value projections of its own")
         for name, v in (("chunk", chunk), ("window", window)):
             if v is not None and v < 1:
                 raise ValueError(f"an attention {name} must hold at least one position")
@@ -266,20 +282,22 @@ class MapsAttention(Mixer):
         self.dk, self.dv = int(head_dim), int(v_head_dim if v_head_dim is not None else head_dim)
         self.maps, self.scale, self.eps = int(maps), float(scale), float(eps)
         self.lambda_init = float(lambda_init) if lambda_init is not None else 0.0
-        self.chunk, self.window, self.sink, self.qk_norm = chunk, window, bool(sink), qk_norm
+        self.chunk, self.window, self.sink, self.qk_norm = chunk, window, bool(sink) or bool(learned_sink), qk_norm
+        self.keep_first, self.qkv_bias, self.learned_sink, self.gate = int(keep_first), bool(qkv_bias), bool(learned_sink), bool(gate)
+        self.value_mix, self.mix = value_mix, 0.0
         self.head_norm = bool(head_norm) if head_norm is not None else self.maps == 2
         self.out_factor = float(out_factor) * float(out_scale) * ((1.0 - self.lambda_init) if self.maps == 2 else 1.0)
         self.own_kv, self.position = bool(own_kv), position
-        need_halves(position, "attention_maps")
         if position is not None and position.rotary_dim > self.dk:
             raise ValueError(f"{position.rotary_dim} rotated channels do not fit a map of {self.dk}")
         self.out_dtype = torch.float32 if float32_output else None
         self.lam = 0.0
-        self.w_qkv = self.w_o = self.q_norm = self.k_norm = None
+        self.w_in = self.b_in = self.w_o = self.q_norm = self.k_norm = self.sink_scores = None
 
     def cache_requirement(self):
         # a page keeps every position: a chunk's keys are needed until the chunk ends, a window's while it passes
-        return PagedKV(self.num_kv_heads, self.maps * self.dk, self.window if self.chunk is None else None, self.dv)
+        return PagedKV(self.num_kv_heads, self.maps * self.dk, self.window if self.chunk is None else None, self.dv,
+                       keep_first=self.keep_first)
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
         W, H, G, dk, dv, M = self.hidden_size, self.num_heads, self.num_kv_heads, self.dk, self.dv, self.maps
@@ -288,16 +306,49 @@ class MapsAttention(Mixer):
             specs["k"] = TensorSpec((G * M * dk, W))
             specs["v"] = TensorSpec((G * dv, W))
         if self.qk_norm is not None:
-            specs["q.norm"] = TensorSpec((dk,), role="vector", init="norm")
-            specs["k.norm"] = TensorSpec((dk,), role="vector", init="norm")
+            whole = self.qk_norm == "projection"
+            specs["q.norm"] = TensorSpec((H * M * dk if whole else dk,), role="vector", init="norm")
+            specs["k.norm"] = TensorSpec((G * M * dk if whole else dk,), role="vector", init="norm")
+        if self.qkv_bias:
+            specs.update({"q.b": TensorSpec((H * M * dk,), role="vector", init="bias"),
+                          "k.b": TensorSpec((G * M * dk,), role="vector", init="bias"),
+                          "v.b": TensorSpec((G * dv,), role="vector", init="bias")})
+        if self.learned_sink:
+            specs["sink"] = TensorSpec((H,), role="vector", init="bias")
+        if self.gate:
+            specs["g"] = TensorSpec((H, W))
+        if self.value_mix is not None:
+            specs["vmix"] = TensorSpec((), role="vector", init="bias")
         if M == 2:
             for name in ("lq1", "lk1", "lq2", "lk2"):
                 specs[name] = TensorSpec((dk,), role="vector", init="bias")
         return specs
 
+    def _turned_order(self, tensors):
+        """The rows of the query and key projections (with their biases and norm weights) in the order the kernels turn:
+        the rotated channels of every map as halves."""
+        pos, dk = self.position, self.dk
+        if pos is None or pos.pairs == "halves":
+            return tensors
+        tensors = dict(tensors)
+        order = torch.tensor(pos.halves_order() + list(range(pos.rotary_dim, dk)), device=tensors["q"].device)
+        for name in ("q", "k", "q.b", "k.b", "q.norm", "k.norm"):
+            if name in tensors:
+                t = tensors[name]
+                tensors[name] = t.view(t.shape[0] // dk, dk, *t.shape[1:])[:, order].reshape(t.shape)
+        return tensors
+
     def bind(self, tensors):
-        mats = [tensors["q"]] + ([tensors["k"], tensors["v"]] if self.own_kv else [])
-        self.w_qkv = torch.cat(mats, dim=0).contiguous() if len(mats) > 1 else mats[0]
+        tensors = self._turned_order(tensors)
+        # one product for everything that reads the input: queries, keys, values, gate logits
+        mats = [tensors["q"]] + ([tensors["k"], tensors["v"]] if self.own_kv else []) + ([tensors["g"]] if self.gate else [])
+        self.w_in = torch.cat(mats, dim=0).contiguous() if len(mats) > 1 else mats[0]
+        if self.qkv_bias:
+            b = [tensors[n].to(torch.float32) for n in ("q.b", "k.b", "v.b")]
+            self.b_in = torch.cat(b + ([b[0].new_zeros(self.num_heads)] if self.gate else [])).contiguous()
+        self.sink_scores = tensors["sink"].to(torch.float32).contiguous() if self.learned_sink else None
+        if self.value_mix == "later":
+            self.mix = float(tensors["vmix"].double().item())
         self.w_o = tensors["o"]
         if self.qk_norm is not None:
             qn, kn = tensors["q.norm"], tensors["k.norm"]
@@ -311,31 +362,61 @@ class MapsAttention(Mixer):
     def output_weights(self):
         return [self.w_o]
 
-    def _queries(self, x: torch.Tensor, step: StepContext, cache: LayerCache) -> torch.Tensor:
+    def _queries(self, x: torch.Tensor, step: StepContext, cache: LayerCache):
         """The projections of ``x``; queries (and, with projections of its own, keys) normalised and rotated; keys and
-        values of every row written to the cache.  Returns q [T, heads * maps * dk] in the compute dtype."""
+        values of every row written to the cache.  Returns (q [T, heads * maps * dk] in the compute dtype, gate logits
+        float32 [T, heads] or None)."""
         Attention._check(cache)
         if cache.writes != self.own_kv:
             raise ValueError("an attention with key and value projections writes its cache; one without reads another's")
         H, G, dk, dv, M = self.num_heads, self.num_kv_heads, self.dk, self.dv, self.maps
-        nq, nk = H * M * dk, G * M * dk
-        proj = ops.linear(x, self.w_qkv, out_dtype=torch.float32)
+        nq, nk, nv = H * M * dk, G * M * dk, G * dv
+        proj = ops.linear(x, self.w_in, self.b_in, out_dtype=torch.float32)
+        k = v = v_first = None
+        if self.own_kv:
+            k, v = proj[:, nq:nq + nk], proj[:, nq + nk:nq + nk + nv]
+        if self.value_mix == "first":
+            step.shared["v_first"] = v
+        elif self.value_mix == "later":
+            v_first = step.shared.get("v_first")
+            if v_first is None or v_first.shape != v.shape:
+                raise ValueError("an attention that mixes values needs an earlier layer of the step that made as many")
         pos = self.position
         rot = pos.rotary_dim if pos is not None else 0
-        return ops.unit_norm_rope_kv_write(
-            proj[:, :nq], proj[:, nq:nq + nk] if self.own_kv else None, proj[:, nq + nk:] if self.own_kv else None,
-            self.q_norm, self.k_norm, self.eps, step.positions, pos.frequency_pairs() if pos is not None else None, rot,
-            pos.amplitude if pos is not None else 1.0, step.slots[cache.group] if self.own_kv else None, cache.k, cache.v,
-            H * M, G * M, G, dk, dv, cache.page_size, self.runtime.dtype)
+        q = ops.unit_norm_rope_kv_write(
+            proj[:, :nq], k, v, self.q_norm, self.k_norm, self.eps, step.positions,
+            pos.frequency_pairs() if pos is not None else None, rot, pos.amplitude if pos is not None else 1.0,
+            step.slots[cache.group] if self.own_kv else None, cache.k, cache.v, H * M, G * M, G, dk, dv, cache.page_size,
+            self.runtime.dtype, whole_norm=self.qk_norm == "projection", v_first=v_first, mix=self.mix)
+        return q, proj[:, proj.shape[1] - H:] if self.gate else None
 
-    def _attend(self, q: torch.Tensor, out: torch.Tensor, step: StepContext, cache: LayerCache) -> None:
+    def _attend(self, q: torch.Tensor, gates: Optional[torch.Tensor], out: torch.Tensor, step: StepContext, cache: LayerCache) -> None:
         ops.attention_maps(q, out, cache.k, cache.v, step, cache.group, self.num_heads, self.num_kv_heads, self.dk, self.dv,
                            self.maps, cache.page_size, self.window, self.chunk, self.sink, self.scale, self.lam, self.head_norm,
-                           self.eps, self.out_factor)
+                           self.eps, self.out_factor, sink_scores=self.sink_scores, head_gates=gates, keep_first=self.keep_first)
 
     def forward_open(self, x: torch.Tensor, step: StepContext, cache: LayerCache, outs) -> None:
         """The heads' outputs in front of the output product into ``outs[0]`` ([T, heads * dv], rows may be strided)."""
-        self._attend(self._queries(x, step, cache), outs[0], step, cache)
+        q, gates = self._queries(x, step, cache)
+        self._attend(q, gates, outs[0], step, cache)
+
+    supports_open_tail = True
+
+    def forward_open_tail(self, x: torch.Tensor, step: StepContext, cache: LayerCache, outs) -> None:
+        """As ``forward_open`` for the wanted rows only (each as a one-token request of ``step.tail``), once the keys and
+        values of every row are in the cache.  An attention that reads another's cache makes the wanted rows' queries only."""
+        rows, tail = step.tail_rows, step.tail
+        if self.own_kv:
+            q, gates = self._queries(x, step, cache)
+            if not tail.num_tokens:
+                return
+            q = ops.gather_rows(q, rows)
+            gates = ops.gather_rows(gates, rows) if gates is not None else None
+        else:
+            if not tail.num_tokens:
+                return
+            q, gates = self._queries(ops.gather_rows(x, rows), tail, cache)
+        self._attend(q, gates, outs[0], tail, cache)
 
     def forward_into(self, x: torch.Tensor, step: StepContext, cache: LayerCache, out: torch.Tensor) -> None:
         o = torch.empty((x.shape[0], self.num_heads * self.dv), dtype=self.runtime.dtype, device=x.device)
@@ -350,20 +431,11 @@ class MapsAttention(Mixer):
     supports_tail = True
 
     def forward_tail(self, x: torch.Tensor, step: StepContext, cache: LayerCache) -> Optional[torch.Tensor]:
-        """Keys and values of every row go to the cache; only the wanted rows attend (each as a one-token request of
-        ``step.tail``).  An attention that reads another's cache makes the wanted rows' queries only."""
-        rows, tail = step.tail_rows, step.tail
-        if self.own_kv:
-            q = self._queries(x, step, cache)
-            if not tail.num_tokens:
-                return None
-            q = ops.gather_rows(q, rows)
-        else:
-            if not tail.num_tokens:
-                return None
-            q = self._queries(ops.gather_rows(x, rows), tail, cache)
-        o = torch.empty((q.shape[0], self.num_heads * self.dv), dtype=self.runtime.dtype, device=x.device)
-        self._attend(q, o, tail, cache)
+        """Keys and values of every row go to the cache; only the wanted rows attend."""
+        o = torch.empty((step.tail.num_tokens, self.num_heads * self.dv), dtype=self.runtime.dtype, device=x.device)
+        self.forward_open_tail(x, step, cache, [o])
+        if not step.tail.num_tokens:
+            return None
         return ops.linear(o, self.w_o, out_dtype=self.out_dtype, partial_ok=self.partial_output)
 
 
@@ -387,6 +459,7 @@ class LatentAttention(Mixer):
     softmax's denominator with a learned score per head, tensor ``sink``, that carries no value) and ``gate`` (head h's
     output is multiplied by sigmoid(g x)_h, tensor ``g`` [heads, width], the same input as the projections).  A layer
     without keys of its own reads the rows (latent and rotated key) that an earlier one wrote, with its own uk and uv.
+    A ``window`` keeps the positions with i - j < window.
 
     Whole prompts (``_expands``) are attended in the EXPANDED form instead: the step's cached rows become keys
     [uk_h c | rotated key] and values uv_h c per head, which costs ``dim + rd`` and ``dv`` channels per score instead of
@@ -396,8 +469,11 @@ class LatentAttention(Mixer):
 
     def __init__(self, runtime: Runtime, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, v_head_dim: int,
                  kv_rank: int, scale: float, eps: float, sink: bool = False, gate: bool = False, own_kv: bool = True,
-                 float32_output: bool = True, position: Optional[Position] = None):
+                 float32_output: bool = True, position: Optional[Position] = None, window: Optional[int] = None):
         super().__init__(runtime)
+        if window is not None and window < 1:
+            raise ValueError("an attention window must hold at least one position")
+        self.window = window
         self.hidden_size, self.num_heads = int(hidden_size), int(num_heads)
         self.dim, self.rd, self.dv, self.rank = int(head_dim), int(rot_dim), int(v_head_dim), int(kv_rank)
         if min(self.num_heads, self.dim, self.dv, self.rank) < 1 or self.rd < 0:
@@ -415,7 +491,7 @@ class LatentAttention(Mixer):
         return self.rank + self.rd
 
     def cache_requirement(self):
-        return PagedKV(1, self.row, None, 0)
+        return PagedKV(1, self.row, self.window, 0)
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
         W, H = self.hidden_size, self.num_heads
@@ -503,7 +579,7 @@ class LatentAttention(Mixer):
         H = self.num_heads
         o_lat = torch.empty((q_wide.shape[0], H * self.rank), dtype=self.runtime.dtype, device=q_wide.device)
         ops.attention_maps(q_wide, o_lat, cache.k, None, step, cache.group, H, 1, self.row, self.rank, 1, cache.page_size,
-                           None, None, self.sink, self.scale, 0.0, False, self.eps, 1.0, sink_scores=self.sink_scores,
+                           self.window, None, self.sink, self.scale, 0.0, False, self.eps, 1.0, sink_scores=self.sink_scores,
                            values_in_keys=True)
         ops.grouped_linear(o_lat, self.w_uv, out, a_col=self.rank, c_col=self.dv, factor=gates, factor_sigmoid=True)
 
@@ -530,7 +606,7 @@ class LatentAttention(Mixer):
         view = types.SimpleNamespace(block_tables=[dense], token_req=step.token_req, positions=step.positions, cu_q=step.cu_q,
                                      kv_lens=step.kv_lens, q_lens=step.q_lens, max_kv_len=step.max_kv_len)
         ops.attention_maps(q_full, out, keys.view(T, H, 1, dk), values.view(T, H, 1, self.dv), view, 0, H, H, dk, self.dv, 1, 1,
-                           None, None, self.sink, self.scale, 0.0, False, self.eps, 1.0, sink_scores=self.sink_scores,
+                           self.window, None, self.sink, self.scale, 0.0, False, self.eps, 1.0, sink_scores=self.sink_scores,
                            head_gates=gates)
 
     def forward_open(self, x: torch.Tensor, step: StepContext, cache: LayerCache, outs) -> None:
@@ -555,22 +631,30 @@ class LatentAttention(Mixer):
     supports_tail = True
 
     def forward_tail(self, x: torch.Tensor, step: StepContext, cache: LayerCache) -> Optional[torch.Tensor]:
-        """The rows of every token go to the cache; only the wanted rows attend (each as a one-token request of
-        ``step.tail``).  A layer that reads another's cache makes the wanted rows' queries only."""
+        """The rows of every token go to the cache; only the wanted rows attend."""
+        o = torch.empty((step.tail.num_tokens, self.num_heads * self.dv), dtype=self.runtime.dtype, device=x.device)
+        self.forward_open_tail(x, step, cache, [o])
+        if not step.tail.num_tokens:
+            return None
+        return ops.linear(o, self.w_o, out_dtype=self.out_dtype, partial_ok=self.partial_output)
+
+    supports_open_tail = True
+
+    def forward_open_tail(self, x: torch.Tensor, step: StepContext, cache: LayerCache, outs) -> None:
+        """As ``forward_open`` for the wanted rows only (each as a one-token request of ``step.tail``), once the rows of
+        every token are in the cache.  A layer that reads another's cache makes the wanted rows' queries only."""
         rows, tail = step.tail_rows, step.tail
         if self.own_kv:
             q_wide, gates = self._queries(x, step, cache)
             if not tail.num_tokens:
-                return None
+                return
             q_wide = ops.gather_rows(q_wide, rows)
             gates = ops.gather_rows(gates, rows) if gates is not None else None
         else:
             if not tail.num_tokens:
-                return None
+                return
             q_wide, gates = self._queries(ops.gather_rows(x, rows), tail, cache)
-        o = torch.empty((q_wide.shape[0], self.num_heads * self.dv), dtype=self.runtime.dtype, device=x.device)
-        self._attend(q_wide, gates, o, tail, cache)
-        return ops.linear(o, self.w_o, out_dtype=self.out_dtype, partial_ok=self.partial_output)
+        self._attend(q_wide, gates, outs[0], tail, cache)
 
 
 class PooledWindowAttention(Mixer):

@@ -50,6 +50,9 @@ class PagedKV:
                                           # the block whose LAST position is p lives in p's page, at row
                                           # block - floor(page * page_size / stride)
 
+    keep_first: int = 0                   # with a window: the first positions of a sequence, which stay visible (and cached)
+                                          # although the window has passed them
+
     def rows_per_page(self, page_size: int) -> int:
         return -(-page_size // self.stride)
 
@@ -123,6 +126,9 @@ class StepContext:
     # Scratch of parts/native_block.py: what the blocks of this step share once the first of them
     # has described the step to the library.
     native: Optional[object] = None
+    # What a layer of this step leaves for later layers of the same step (for instance the values that later layers mix
+    # into theirs), by a name the parts agree on; emptied when the model starts a step.
+    shared: Dict[str, torch.Tensor] = field(default_factory=dict)
 
 
 @dataclass
@@ -235,6 +241,10 @@ class Mixer(Part):
 
     # True if the part implements forward_tail.
     supports_tail = False
+
+    # True if it implements forward_open_tail(x, step, cache, outs): forward_tail for blocks that take the output product
+    # over (``forward_open``), leaving the wanted rows' activations in ``outs`` (nothing when there are no such rows).
+    supports_open_tail = False
 
     def forward_tail(self, x: torch.Tensor, step: StepContext, cache) -> Optional[torch.Tensor]:
         """Update the cache (or state) for ALL rows of ``x`` as ``forward`` does, but return the

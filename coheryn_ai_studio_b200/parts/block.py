@@ -113,7 +113,7 @@ class ParallelResidual(Arrangement):
     def forward(self, residual, delta, step, cache):
         if not self.mixer.partial_output:
             raise ValueError("parallel_residual needs a model whose norms all take partial sums")
-        h = self.norm.forward(residual, delta)
+        h = self.norm.forward(residual, None if isinstance(delta, StreamCopy) else delta)
         joined = self._joined_output() if ops.JOINED_OUTPUT else False
         if joined:
             w_out, ranges, counts = joined
@@ -133,6 +133,28 @@ class ParallelResidual(Arrangement):
         if self.feed_forward is not None:
             self.feed_forward.forward_into(h, step, out[n_mix:])
         return residual, out
+
+    @property
+    def supports_tail(self):
+        """With one product for all outputs and a mixer whose activations can be made for the wanted rows alone."""
+        return (getattr(self.mixer, "supports_open_tail", False) and self.mixer.partial_output and ops.JOINED_OUTPUT
+                and bool(self._joined_output()))
+
+    def forward_tail(self, residual, delta, step, cache):
+        """The mixer updates its cache for all rows; its outputs, the feed-forward and the output product run for the
+        wanted rows only."""
+        h = self.norm.forward(residual, None if isinstance(delta, StreamCopy) else delta)
+        w_out, ranges, counts = self._joined_output()
+        R = step.tail.num_tokens
+        acts = torch.empty((R, w_out.shape[1]), dtype=w_out.dtype, device=residual.device)
+        views = [acts[:, a:b] for a, b in ranges]
+        self.mixer.forward_open_tail(h, step, cache, views[:counts[0]])
+        if not R:
+            return None, None
+        if self.feed_forward is not None:
+            self.feed_forward.forward_open(ops.gather_rows(h, step.tail_rows), step.tail, None, views[counts[0]:])
+        out = ops.linear(acts, w_out, out_dtype=torch.float32, partial_ok=True)
+        return ops.gather_rows(residual, step.tail_rows), out if out.dim() == 3 else out.unsqueeze(0)
 
 
 class SandwichResidual(Arrangement):

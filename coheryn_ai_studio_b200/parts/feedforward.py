@@ -2,6 +2,8 @@
 silu(g) = g / (1 + exp(-g)), or the tanh form of GELU, in float32
 (crates/coheryn-engine/src/inference.rs:516-540, crates/coheryn-engine/src/cpu.rs:74-78).  ``swish_clamped`` with its
 constant c is the variant g <- min(g, c), u <- clamp(u, -c, c), y = W_down (g sigmoid(1.702 g) (u + 1)).
+
+The feed-forward without a gate, ``mlp``: y = W_down act(W_up x).
 """
 from __future__ import annotations
 
@@ -60,4 +62,43 @@ class GatedMLP(FeedForward):
         ops.linear(ops.gated_linear(x, self.w_gate_up, self.activation, param=self.constant), self.w_down, out=out[0])
 
 
+class MLP(FeedForward):
+    """y = W_down act(W_up x), the activation in the first product's epilogue ("gelu": the exact form)."""
+
+    output_parts = 1
+
+    def __init__(self, runtime: Runtime, hidden_size: int, intermediate_size: int, activation: str,
+                 tensors=("up_proj.weight", "down_proj.weight"), float32_output: bool = False):
+        """``tensors``: the local names of the up and down matrices in the checkpoint.  ``float32_output`` as for
+        :class:`GatedMLP`."""
+        super().__init__(runtime)
+        self.names = tuple(tensors)
+        ops.plain_activation_code(activation)        # refuses an activation the epilogues lack
+        self.activation = activation
+        self.out_dtype = torch.float32 if float32_output else None
+        self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
+        self.w_up = self.w_down = None
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        H, I = self.hidden_size, self.intermediate_size
+        return {self.names[0]: TensorSpec((I, H)), self.names[1]: TensorSpec((H, I))}
+
+    def bind(self, tensors):
+        self.w_up, self.w_down = tensors[self.names[0]], tensors[self.names[1]]
+
+    def output_weights(self):
+        return [self.w_down]
+
+    def forward_open(self, x: torch.Tensor, step: StepContext, cache, outs) -> None:
+        ops.linear(x, self.w_up, out=outs[0], activation=self.activation)
+
+    def forward(self, x: torch.Tensor, step: StepContext) -> torch.Tensor:
+        act = ops.linear(x, self.w_up, activation=self.activation)
+        return ops.linear(act, self.w_down, out_dtype=self.out_dtype, partial_ok=self.partial_output)
+
+    def forward_into(self, x: torch.Tensor, step: StepContext, out: torch.Tensor) -> None:
+        ops.linear(ops.linear(x, self.w_up, activation=self.activation), self.w_down, out=out[0])
+
+
+register_feed_forward("mlp", MLP)
 register_feed_forward("gated_mlp", GatedMLP)

@@ -141,6 +141,7 @@ class DecoderModel:
         ``[len(logit_rows), vocab]`` of the rows asked for."""
         T, H = step.num_tokens, self.spec.hidden_size
         step.native = None      # a step object may be run again (warm-up, then capture): on another stream
+        step.shared = {}
         residual = torch.empty((T, H), dtype=torch.float32, device=self.runtime.device)
         delta = None
         last = len(self.spec.schedule) - 1

@@ -23,6 +23,9 @@ that runs several mixers side by side.
   q = W_q h * d^(-1/2), k = W_k h, v = W_v h;  z = W_a2 (W_a1 h) + b, alpha = sigmoid(z)^(1 / tau);
   S_t = diag(alpha_t) S_(t-1) + k_t v_t^T from S = 0, o_t = S_t^T q_t.  Each head's o is divided by its root mean square,
   multiplied by a weight shared by the heads and by silu(W_g h), then W_o.
+* ``LightningAttention`` (kind ``lightning_attention``): linear attention with a constant decay a per head.  q = silu(W_q h),
+  k = silu(W_k h), v = silu(W_v h);  S_t = a S_(t-1) + k_t v_t^T from S = 0, o_t = S_t^T q_t.  All heads' o together are
+  divided by their root mean square, multiplied by a weight and by sigmoid(W_g h), then W_o.
 * ``SideBySide`` (kind ``side_by_side``): mixers that read the same input; the result is the weighted sum of
   theirs.  Each child multiplies its own output by its weight before its output projection, and the
   children's outputs go to the next norm as separate summands.
@@ -41,7 +44,7 @@ import torch
 from .. import ops
 from ..config.spec import PartSpec
 from ..weights.spec import TensorSpec
-from .base import MIXERS, FixedState, LayerCache, Mixer, NormedSum, Runtime, StepContext, build_part, register_mixer
+from .base import MIXERS, POSITIONS, FixedState, LayerCache, Mixer, NormedSum, Runtime, StepContext, build_part, register_mixer
 
 
 class _StackedInput:
@@ -347,10 +350,66 @@ class GatedLinearAttention(_StateMixer):
         return ops.linear(ops.gather_rows(o, step.tail_rows), self.w_o, out_dtype=self.out_dtype, partial_ok=self.partial_output)
 
 
+class LightningAttention(_StateMixer):
+    def __init__(self, runtime: Runtime, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, decay: Sequence[float],
+                 eps: float, silu: bool = True, gate_activation: str = "sigmoid", out_scale: float = 1.0):
+        """``decay``: the heads' constants, 0 <= a <= 1.  ``silu`` False: the projections enter as they are."""
+        super().__init__(runtime)
+        self.hidden_size, self.num_heads = int(hidden_size), int(num_heads)
+        self.dk, self.dv, self.eps, self.out_scale = int(head_dim), int(v_head_dim), float(eps), float(out_scale)
+        self.decay, self.silu, self.gate_activation = tuple(float(a) for a in decay), bool(silu), gate_activation
+        if min(self.num_heads, self.dk, self.dv) < 1:
+            raise ValueError("a linear attention needs positive head counts and sizes")
+        if len(self.decay) != self.num_heads or not all(0.0 <= a <= 1.0 for a in self.decay):
+            raise ValueError("lightning_attention: one decay per head, from 0 to 1")
+        if gate_activation not in ("sigmoid", "silu"):
+            raise ValueError("lightning_attention: gate_activation is 'sigmoid' or 'silu'")
+        self.stacked = self.norm_w = self.w_o = self.powers = None
+
+    def cache_requirement(self):
+        return FixedState((self.num_heads * self.dk * self.dv,), torch.float32)     # S of every head, [dk, dv] rows first
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        W, H, dk, dv = self.hidden_size, self.num_heads, self.dk, self.dv
+        return {"q": TensorSpec((H * dk, W)), "k": TensorSpec((H * dk, W)), "v": TensorSpec((H * dv, W)), "g": TensorSpec((H * dv, W)),
+                "o": TensorSpec((W, H * dv)), "norm": TensorSpec((H * dv,), role="vector", init="norm")}
+
+    def bind(self, tensors):
+        self.stacked = _StackedInput([(n, tensors[n]) for n in ("q", "k", "v", "g")])     # one product for all that reads h
+        self.norm_w, self.w_o = tensors["norm"], tensors["o"]
+        self.powers = ops.decay_powers(self.decay, self.w_o.device)
+
+    def output_weights(self):
+        return [self.w_o]
+
+    def forward_open(self, x: torch.Tensor, step: StepContext, cache: Optional[LayerCache], outs) -> None:
+        """The normalised, gated heads in front of the output product into ``outs[0]`` [T, heads * dv]."""
+        state = self._state_of(cache)
+        st, proj = self.stacked, self.stacked.project(x)
+        ops.lightning_attention(st.cut(proj, "q"), st.cut(proj, "k"), st.cut(proj, "v"), st.cut(proj, "g"), self.powers, self.silu,
+                                state, step, self.num_heads, self.dk, self.dv, self.norm_w, self.eps, outs[0],
+                                gate_activation=self.gate_activation, out_scale=self.out_scale)
+
+    def forward_into(self, x: torch.Tensor, step: StepContext, cache: Optional[LayerCache], out: torch.Tensor) -> None:
+        o = torch.empty((x.shape[0], self.num_heads * self.dv), dtype=self.runtime.dtype, device=x.device)
+        self.forward_open(x, step, cache, [o])
+        ops.linear(o, self.w_o, out=out[0])
+
+    supports_open_tail = True
+
+    def forward_open_tail(self, x: torch.Tensor, step: StepContext, cache: Optional[LayerCache], outs) -> None:
+        """The state passes every row; the wanted rows' activations are picked out."""
+        o = torch.empty((x.shape[0], self.num_heads * self.dv), dtype=self.runtime.dtype, device=x.device)
+        self.forward_open(x, step, cache, [o])
+        if step.tail.num_tokens:
+            outs[0].copy_(ops.gather_rows(o, step.tail_rows))
+
+
 class SideBySide(Mixer):
-    def __init__(self, runtime: Runtime, hidden_size: int, mixers: Sequence[Tuple[str, PartSpec, float]], position=None,
+    def __init__(self, runtime: Runtime, hidden_size: int, mixers: Sequence[Tuple], position=None,
                  combine: str = "sum", eps: float = 1e-6):
-        """``mixers``: (name under which the child's tensors stand, the child's PartSpec, the weight of its output).
+        """``mixers``: (name under which the child's tensors stand, the child's PartSpec, the weight of its output), or with
+        the PartSpec of a position encoding of the child's own behind them (None: none) where the children's differ.
         ``combine``: "sum" (the weighted sum of the children's outputs) or "normed_mean": every child's output is
         divided by its root mean square over the model width (``eps`` inside the root) and multiplied by a weight
         ``<name>.out`` [width]; the result is the mean of those (the children's weights must be 1)."""
@@ -360,13 +419,14 @@ class SideBySide(Mixer):
             raise ValueError("side_by_side needs at least one mixer")
         if combine not in ("sum", "normed_mean"):
             raise ValueError(f"side_by_side: combine {combine!r} is not built (sum, normed_mean)")
-        if combine == "normed_mean" and any(float(w) != 1.0 for _, _, w in mixers):
+        if combine == "normed_mean" and any(float(m[2]) != 1.0 for m in mixers):
             raise ValueError("side_by_side: normalised outputs take no weights besides their norms'")
         self.combine, self.eps = combine, float(eps)
         self.out_weights = None
         self.children = []
-        for name, spec, weight in mixers:
-            extra = {"position": position} if position is not None else {}
+        for name, spec, weight, *own in mixers:
+            pos = build_part(POSITIONS, "position", own[0], runtime) if own and own[0] is not None else (None if own else position)
+            extra = {"position": pos} if pos is not None else {}
             child = build_part(MIXERS, "mixer", spec, runtime, out_scale=float(weight), **extra)
             if not hasattr(child, "forward_into"):
                 raise ValueError(f"side_by_side: {type(child).__name__} cannot write its output into a stack of summands")
@@ -419,6 +479,19 @@ class SideBySide(Mixer):
             c.forward_open(x, step, sub, outs[at:at + n])
             at += n
 
+    @property
+    def supports_open_tail(self):
+        return self.combine == "sum" and all(c.supports_open_tail for _, c in self.children)
+
+    def forward_open_tail(self, x: torch.Tensor, step: StepContext, cache: Optional[LayerCache], outs) -> None:
+        if cache is None or cache.kind != "several" or len(cache.parts) != len(self.children):
+            raise ValueError("side_by_side needs one cache per child")
+        at = 0
+        for (_, c), sub in zip(self.children, cache.parts):
+            n = len(c.output_weights())
+            c.forward_open_tail(x, step, sub, outs[at:at + n])
+            at += n
+
     def forward(self, x: torch.Tensor, step: StepContext, cache: Optional[LayerCache]) -> torch.Tensor:
         out = torch.empty((self.output_parts, x.shape[0], self.hidden_size), dtype=torch.float32, device=x.device)
         self._children_into(x, step, cache, out)
@@ -435,4 +508,5 @@ register_mixer("matrix_memory", MatrixMemory)
 register_mixer("gated_delta_rule", GatedDeltaRule)
 register_mixer("gated_linear_attention", GatedLinearAttention)
 register_mixer("gated_linear_recurrence", GatedLinearRecurrence)
+register_mixer("lightning_attention", LightningAttention)
 register_mixer("side_by_side", SideBySide)
