@@ -31,7 +31,9 @@ sub-layer), its kernels beside the like kernels of the other models.  ``--worklo
 design (gated linear recurrences, window attention over positions and block means, routed experts with a shared expert, a
 repeated span of layers).  ``--workload zusotar`` does the same for the Zusotar design (latent attention, gated linear
 attention, window attention with a logarithmic bias by distance, routed experts, an average over depth behind every layer)
-beside Guvusun at equal sizes and Qwen2.  ``--workload guvusun`` does the same for the Guvusun
+beside Guvusun at equal sizes and Qwen2.  ``--workload vilazen`` does the same for the Vilazen design (window attention that
+keeps the first positions, attention with a sink beside a linear attention with a constant decay per head, latent attention
+over a window, one norm per layer) beside Zusotar and Qwen2 at equal sizes.  ``--workload guvusun`` does the same for the Guvusun
 design (latent attention with a learned sink and head gates, routed experts, norms after the sum) beside Qwen2 with a dense
 feed-forward of the experts' active size.
 """
@@ -1139,6 +1141,195 @@ def zusotar_workload(args) -> int:
     return 0
 
 
+# Sizes of --workload vilazen: window attention that keeps the first positions, attention with a sink beside a linear
+# attention with a constant decay, and latent attention over a window in the proportion 2 : 1 : 1, every layer with a
+# feed-forward without a gate.  Beside each the closest other design, Zusotar, with as many layers of the same latent
+# attention, gated linear attention and window attention in the same proportion and gated feed-forwards of as many weights
+# (two thirds of the rows); and Qwen2 likewise.
+VILAZEN_SIZES = {
+    "w2048": dict(width=2048, vocab=32000, layers="aplaapla", window=(16, 4, 128, 128, 1024, 16, 64), left=(16, 4, 128, 128, 64),
+                  right=(8, 128, 128), latent=(16, 96, 32, 128, 224, 1024), ff=7680),
+    "w4096": dict(width=4096, vocab=32000, layers="apla", window=(32, 8, 128, 128, 2048, 16, 64), left=(32, 8, 128, 128, 128),
+                  right=(16, 128, 256), latent=(32, 128, 64, 128, 512, 2048), ff=16896),
+}
+
+
+def vilazen_config(z):
+    H, G, dk, dv, size, keep, dims = z["window"]
+    rot = lambda dims, base: {"dims": dims, "base": base}
+    window = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": dk, "vdim": dv, "scale": dk ** -0.5, "v_mix": True,
+                                             "mask": {"size": size, "keep_first": keep}, "rot": rot(dims, 500000.0)}}
+    H, G, dk, dv, dims = z["left"]
+    h, d, v = z["right"]
+    both = {"type": "parallel", "mixer": {
+        "left": {"heads": H, "kv_heads": G, "dim": dk, "vdim": dv, "scale": dk ** -0.5, "rot": rot(dims, 1000000.0)}, "left_scale": 0.5,
+        "right": {"heads": h, "dim": d, "vdim": v, "decay": [1.0 - 2.0 ** (-1.0 - 9.0 * i / h) for i in range(h)]}, "right_scale": 0.5}}
+    H, dim, rd, vd, r, size = z["latent"]
+    latent = {"type": "latent_attention", "mixer": {"heads": H, "dim": dim, "rot_dim": rd, "vdim": vd, "kv_rank": r, "scale": (dim + rd) ** -0.5,
+                                                    "mask": {"size": size}, "rot": rot(rd, 1000000.0)}}
+    kinds = {"a": window, "p": both, "l": latent}
+    return {"architecture": "Vilazen", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+            "layers": [dict(kinds[c], mlp={"kind": "dense", "ff": z["ff"]}) for c in z["layers"]]}
+
+
+def vilazen_workload(args) -> int:
+    """Prefill and decode throughput of Vilazen, of Zusotar and of Qwen2 at equal sizes through the step function, and the
+    design's own kernels alone beside the like kernels of the other models, each with its share of the roofline.  One JSON
+    line."""
+    import torch
+
+    from coheryn_ai_studio_b200 import ops
+    from coheryn_ai_studio_b200.config import Qwen2Config
+    from coheryn_ai_studio_b200.config.vilazen import VilazenConfig
+    from coheryn_ai_studio_b200.config.zusotar import ZusotarConfig
+    from coheryn_ai_studio_b200.engine import random_model_on_device
+
+    tools = model_bench_tools(args)
+    pk, hbm, flops_peak, dev = tools.pk, tools.hbm, tools.flops_peak, tools.dev
+    tokens, batch, context = tools.tokens, tools.batch, tools.context
+    timed, step_like = tools.timed, tools.step_like
+    fma_peak = 148 * 128 * 2 * 1.965e9        # float32 FMA lanes x 2 x the SM clock: what float32 arithmetic is bound by
+
+    def kernels(z):
+        out = {}
+        W, page = z["width"], args.page_size
+        f = lambda *shape: torch.randn(shape, device=dev)
+        b16 = lambda *shape: f(*shape).to(torch.bfloat16)
+        empty = lambda *shape: torch.empty(shape, dtype=torch.bfloat16, device=dev)
+        for name, lengths, starts in (("prefill", [tokens], [0]), ("decode", [1] * batch, [context] * batch)):
+            B, T = len(lengths), sum(lengths)
+            per = -(-max(s + n for s, n in zip(starts, lengths)) // page)
+            tables = torch.arange(B * per, dtype=torch.int32, device=dev).view(B, per)
+            st = step_like(lengths, starts, tables)
+            st.block_tables, st.max_q_len = [tables, tables], max(lengths)
+            st.slots = [(tables[st.token_req.long(), (st.positions // page).long()] * page + st.positions % page).to(torch.int32)]
+            met = lambda size: sum(min(p + 1, size) for s, n in zip(starts, lengths) for p in range(s, s + n))      # keys the rows see
+            read = lambda size: sum(min(s + n, size + n) for s, n in zip(starts, lengths))                          # cached rows read
+
+            def record(label, fn, by=None, flops=None, peak=None, peak_name="of_bf16_peak"):
+                ms = timed(fn)
+                e = out[f"{name}.{label}"] = {"ms": round(ms, 4)}
+                if by is not None:
+                    e["of_hbm"] = round(by / (ms / 1e3) / hbm, 4)
+                if flops is not None:
+                    e["tflops"] = round(flops / ms / 1e9, 1)
+                    e[peak_name] = round(flops / (ms / 1e3) / peak, 4)
+
+            # linear attention with a constant decay per head, and with a decay per channel at the same heads
+            H, dk, dv = z["right"]
+            q, k, v, g = f(T, 2 * H * (dk + dv)).split([H * dk, H * dk, H * dv, H * dv], dim=1)      # one projection, as the mixers have it
+            state = torch.zeros((B, H * dk * dv), dtype=torch.float32, device=dev)
+            o, nw, nw1 = empty(T, H * dv), f(H * dv), f(dv)
+            powers = ops.decay_powers([1.0 - 2.0 ** (-1.0 - 9.0 * i / H) for i in range(H)], dev)
+            by, fl = 8.0 * B * H * dk * dv + T * H * (8.0 * dk + 10.0 * dv), 4.0 * T * H * dk * dv
+            record("lightning_attention", lambda: ops.lightning_attention(
+                q, k, v, g, powers, True, state, st, H, dk, dv, nw, 1e-6, o), by=by, flops=fl, peak=fma_peak, peak_name="of_fma_peak")
+            a1, a2, a2b = f(T, 16), b16(H * dk, 16), f(H * dk)
+            record("zusotar_gated_linear_attention", lambda: ops.gated_linear_attention(
+                q, k, v, g, a1, a2, a2b, 16.0, 1.0, state, st, H, dk, dv, nw1, 1e-6, o), by=by, flops=fl, peak=fma_peak, peak_name="of_fma_peak")
+            # attention over a window that keeps the first positions, with a gate per head; Zusotar's and Qwen2's windows
+            H, G, dk, dv, size, keep, dims = z["window"]
+            io, fl = 2.0 * (dk + dv) * G * read(size + keep) + 2.0 * T * H * (dk + dv), 2.0 * H * (dk + dv) * met(size + keep)
+            kc, vc, qa, oa, gates = b16(B * per + 1, G, page, dk), b16(B * per + 1, G, page, dv), b16(T, H * dk), empty(T, H * dv), f(T, H)
+            record("window_attention_kept_first_head_gates", lambda: ops.attention_maps(
+                qa, oa, kc, vc, st, 0, H, G, dk, dv, 1, page, size, None, False, dk ** -0.5, 0.0, False, 1e-6, 1.0, head_gates=gates,
+                keep_first=keep), by=io, flops=fl, peak=flops_peak)
+            if dk == dv:
+                wide, r1, r2 = f(T, H * dv), f(H).abs(), f(H).abs()
+                record("zusotar_window_attention", lambda: ops.pooled_attention(
+                    qa, oa, kc, vc, None, None, st, 0, None, H, G, dk, dv, page, size, None, dk ** -0.5, None, None, None, wide, None,
+                    log_bias=(r1, r2)), by=io, flops=fl, peak=flops_peak)
+                record("qwen2_attention_same_window", lambda: ops.attention_rows(
+                    qa, oa, kc, vc, tables, st.token_req, st.positions, H, G, dk, page, size, dk ** -0.5, cu_q=st.cu_q, kv_lens=st.kv_lens,
+                    q_lens=st.q_lens, max_kv_len=st.max_kv_len), by=io, flops=fl, peak=flops_peak)
+            proj, first = f(T, (H + G) * dk + G * dv), f(T, G * dv)
+            freq = torch.stack([torch.pow(torch.tensor(5e5), -2.0 * torch.arange(dims // 2) / dims), torch.zeros(dims // 2)], dim=1).to(dev).contiguous()
+            cut = (proj[:, :H * dk], proj[:, H * dk:(H + G) * dk], proj[:, (H + G) * dk:])
+            moved = T * ((H + G) * dk + G * dv) * 6.0
+            wq, wk = f(H * dk), f(G * dk)
+            record("projection_norm_rotation_value_mix_and_cache_write", lambda: ops.unit_norm_rope_kv_write(
+                *cut, wq, wk, 1e-6, st.positions, freq, dims, 1.0, st.slots[0], kc, vc, H, G, G, dk, dv, page, torch.bfloat16, whole_norm=True,
+                v_first=first, mix=0.3), by=moved + T * G * dv * 4.0)
+            w1 = f(dk)
+            record("tutunex_head_norm_rotation_and_cache_write", lambda: ops.unit_norm_rope_kv_write(
+                *cut, w1, w1, 1e-6, st.positions, freq, dims, 1.0, st.slots[0], kc, vc, H, G, G, dk, dv, page, torch.bfloat16), by=moved)
+            # causal attention with a learned sink and a gate per head; Qwen2's
+            H, G, dk, dv, dims = z["left"]
+            every = 1 << 30
+            io, fl = 2.0 * (dk + dv) * G * read(every) + 2.0 * T * H * (dk + dv), 2.0 * H * (dk + dv) * met(every)
+            kc, vc, qa, oa, gates, sinks = b16(B * per + 1, G, page, dk), b16(B * per + 1, G, page, dv), b16(T, H * dk), empty(T, H * dv), f(T, H), f(H)
+            record("causal_attention_sink_head_gates", lambda: ops.attention_maps(
+                qa, oa, kc, vc, st, 0, H, G, dk, dv, 1, page, None, None, True, dk ** -0.5, 0.0, False, 1e-6, 0.5, sink_scores=sinks,
+                head_gates=gates), by=io, flops=fl, peak=flops_peak)
+            if dk == dv:
+                record("qwen2_attention", lambda: ops.attention_rows(
+                    qa, oa, kc, vc, tables, st.token_req, st.positions, H, G, dk, page, None, dk ** -0.5, cu_q=st.cu_q, kv_lens=st.kv_lens,
+                    q_lens=st.q_lens, max_kv_len=st.max_kv_len), by=io, flops=fl, peak=flops_peak)
+                record("zegelix_causal_attention", lambda: ops.pooled_attention(
+                    qa, oa, kc, vc, None, None, st, 0, None, H, G, dk, dv, page, None, None, dk ** -0.5, None, None, sinks, None, None),
+                    by=io, flops=fl, peak=flops_peak)
+            # latent attention over a window (over the latent rows); without one, with a sink (Zusotar)
+            H, dim, rd, vd, rank, size = z["latent"]
+            row = rank + rd
+            kl, ql, ol, sk = b16(B * per + 1, 1, page, row), b16(T, H * row), empty(T, H * rank), f(H)
+            for label, window, sink in (("latent_attention_window", size, None), ("zusotar_latent_attention_sink", None, sk)):
+                n = window or every
+                record(label, lambda: ops.attention_maps(
+                    ql, ol, kl, None, st, 0, H, 1, row, rank, 1, page, window, None, sink is not None, (dim + rd) ** -0.5, 0.0, False, 1e-6, 1.0,
+                    sink_scores=sink, values_in_keys=True), by=2.0 * row * read(n) + 2.0 * T * H * (row + rank), flops=2.0 * H * (row + rank) * met(n),
+                    peak=flops_peak)
+            # the feed-forward's first product with its activation; the gated one of as many weights
+            h, up, gate_up = b16(T, W), b16(z["ff"], W), b16(2 * (z["ff"] // 2), W)
+            act, act2 = empty(T, z["ff"]), empty(T, z["ff"] // 2)
+            by, fl = 2.0 * z["ff"] * W + 2.0 * T * (W + z["ff"]), 2.0 * T * W * z["ff"]
+            record("product_with_gelu", lambda: ops.linear(h, up, out=act, activation="gelu"), by=by, flops=fl, peak=flops_peak)
+            record("product_alone", lambda: ops.linear(h, up, out=act), by=by, flops=fl, peak=flops_peak)
+            record("qwen2_product_with_silu_gate", lambda: ops.gated_linear(h, gate_up, out=act2), by=by, flops=fl, peak=flops_peak)
+            # the embedding with its norm
+            table, x, w2 = b16(z["vocab"], W), f(T, W), f(W)
+            st.token_ids = torch.randint(0, z["vocab"], (T,), dtype=torch.int32, device=dev)
+            status = torch.zeros(1, dtype=torch.int32, device=dev)
+            record("embedding_and_norm", lambda: ops.embed_pair(table, None, st, None, 0, 0, 0, None, w2, 1e-6, x, None, status), by=T * W * 6.0)
+            record("qwen2_embedding", lambda: ops.embed_gather(table, st.token_ids, x, status), by=T * W * 6.0)
+        return out
+
+    sampler = ClockSampler()
+    sampler.start()
+    t0 = time.time()
+    results = {}
+    for name in [n for n in VILAZEN_SIZES if not args.sizes or n in args.sizes.split(",")]:
+        z = VILAZEN_SIZES[name]
+        entry = {}
+
+        def run(label, config):
+            model = random_model_on_device(config, seed=0, dtype="bfloat16", device="cuda:0")
+            entry[label] = tools.run_model(model, z["vocab"])
+            del model
+            torch.cuda.empty_cache()
+        run("vilazen", VilazenConfig.from_dict(vilazen_config(z)))
+        gated = 2 * z["ff"] // 3
+        H, dk, dv = z["right"]
+        near = zusotar_config(dict(
+            width=z["width"], vocab=z["vocab"], layers="".join({"a": "w", "p": "g", "l": "l"}[c] for c in z["layers"]), gla=(H, dk, dv, 16),
+            latent=z["latent"][:5], window=(z["window"][0], z["window"][1], z["window"][2], z["window"][4]), experts=2, top=1, groups=(1, 1),
+            ff=8, shared=8, dense=gated), max(context, tokens) + 1024)
+        run("zusotar_equal_size", ZusotarConfig.from_dict(dict(near, layers=[dict(L, mlp={"kind": "dense", "ff": gated}) for L in near["layers"]])))
+        H, G, d = z["window"][:3]
+        run("qwen2_equal_size", Qwen2Config(
+            vocab_size=z["vocab"], hidden_size=z["width"], intermediate_size=gated, num_hidden_layers=len(z["layers"]),
+            num_attention_heads=H, num_key_value_heads=G, head_dim=d, max_position_embeddings=32768, rms_norm_eps=1e-6, rope_theta=1e6,
+            tie_word_embeddings=False))
+        if not args.no_kernels:
+            entry["kernels"] = kernels(z)
+        results[name] = entry
+    clocks = ClockSampler.summary(sampler.window(t0, time.time()))
+    sampler.stop()
+    print(json.dumps({"workload": "vilazen", "dtype": "bf16", "data": "synthetic", "prefill_tokens": tokens, "decode_batch": batch,
+                      "decode_context": context, "decode_steps": tools.steps, "peaks": pk, "clocks": clocks,
+                      "l2": "flushed before each timed kernel", "gpu_launches": ops.total_launch_count(), "sizes": results}))
+    return 0
+
+
 def timeline(args, make_engine, StepEntry, ops, torch) -> int:
     """Where a decode step's time goes, kernel by kernel, measured inside graph-replayed steps (the
     kernels overlap through programmatic dependent launch, so a kernel's own duration says little):
@@ -1206,10 +1397,10 @@ def main() -> int:
     ap.add_argument("--page-size", type=int, default=16)
     ap.add_argument("--skip-points", action="store_true", help="skip the batch 1 / 64 points")
     ap.add_argument("--no-graphs", action="store_true")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serving-7b", "long-14b", "chat-1.5b", "kapudra", "tutunex", "guvusun", "zegelix", "zusotar"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "serving-7b", "long-14b", "chat-1.5b", "kapudra", "tutunex", "guvusun", "zegelix", "zusotar", "vilazen"],
                     help="decode: the contract's line (default); the others: see the header")
-    ap.add_argument("--sizes", default="", help="--workload kapudra / tutunex / guvusun / zegelix / zusotar: which of its sizes (comma separated; default all)")
-    ap.add_argument("--no-kernels", action="store_true", help="--workload guvusun / zegelix / zusotar: the models only, not the kernels alone")
+    ap.add_argument("--sizes", default="", help="--workload kapudra / tutunex / guvusun / zegelix / zusotar / vilazen: which of its sizes (comma separated; default all)")
+    ap.add_argument("--no-kernels", action="store_true", help="--workload guvusun / zegelix / zusotar / vilazen: the models only, not the kernels alone")
     ap.add_argument("--timeline-raw", action="store_true", help="with --timeline: also every kernel's start and end")
     ap.add_argument("--timeline", action="store_true",
                     help="instead of the benchmark: the kernels of one graph-replayed decode step with their times "
@@ -1236,6 +1427,8 @@ def main() -> int:
         return zegelix_workload(args)
     if args.workload == "zusotar":
         return zusotar_workload(args)
+    if args.workload == "vilazen":
+        return vilazen_workload(args)
     if args.workload != "decode":
         return other_workload(args)
 

@@ -1,6 +1,10 @@
 // Causal (optionally windowed) grouped-query attention over cache pages for prompt portions
 // on the 5th-generation tensor cores, compiled for one head size (CO_HEAD_DIM, a multiple of
-// 64 up to 256).
+// 64 up to 256).  Compiled with CO_VALUE_DIM as well it is the kernel with OPTIONS: values of another
+// head size than keys, both multiples of 16 (columns up to the next multiple of 64 are fetched as
+// zeros), the first positions of the sequence kept in sight beside a window, a sink in the softmax's
+// denominator, a gate per head and a factor on the output, and keys and values that lie densely,
+// position by position of the step's own rows, instead of in cache pages.
 //
 // One CTA owns a tile of query rows of one (request, kv head): TOK = 128 / G whole tokens
 // times the G heads of the group (row r = token * G + head), at most 128 rows = the lanes of
@@ -43,14 +47,27 @@ namespace {
 
 typedef __nv_bfloat16 bf16;
 constexpr int HD = CO_HEAD_DIM;
+#ifdef CO_VALUE_DIM
+constexpr bool OPTIONS = true;
+constexpr int VD = CO_VALUE_DIM;
+constexpr bool SUPPORTED = HD % 16 == 0 && HD <= 256 && VD % 16 == 0 && VD <= 256;
+#else
+constexpr bool OPTIONS = false;
+constexpr int VD = HD;
 constexpr bool SUPPORTED = HD % 64 == 0 && HD <= 256;
+#endif
 constexpr int BN = 128;                          // key positions per tile
-constexpr int KCH = SUPPORTED ? HD / 64 : 1;     // 64-column chunks of the head dim
+constexpr int KCH = SUPPORTED ? (HD + 63) / 64 : 1, VCH = SUPPORTED ? (VD + 63) / 64 : 1;     // 64-column chunks of the head dims
+constexpr int VDP = SUPPORTED ? VCH * 64 : HD;   // value columns as the tiles and the accumulator have them
 constexpr int CHUNK_BYTES = 128 * 128;           // 128 rows of 128 bytes
-constexpr int NST = HD <= 128 ? 3 : 1;           // K/V stages
-constexpr int Q_BYTES = KCH * CHUNK_BYTES, KV_BYTES = KCH * CHUNK_BYTES;
-constexpr int SMEM_BYTES = Q_BYTES + NST * 2 * KV_BYTES + 1024 /* alignment slack */ + 256 /* barriers */ + 1024 /* row_ex */;
-constexpr int COL_S = 0, COL_O = 128, COL_P = 128 + HD;
+constexpr int Q_BYTES = KCH * CHUNK_BYTES, K_BYTES = KCH * CHUNK_BYTES, V_BYTES = VCH * CHUNK_BYTES;
+constexpr int REST_BYTES = 1024 /* alignment slack */ + 256 /* barriers */ + 1024 /* row_ex */;
+constexpr int stages_that_fit(int most) {
+  return most > 1 && Q_BYTES + most * (K_BYTES + V_BYTES) + REST_BYTES > 227 * 1024 ? stages_that_fit(most - 1) : most;
+}
+constexpr int NST = stages_that_fit(3);          // K/V stages
+constexpr int SMEM_BYTES = Q_BYTES + NST * (K_BYTES + V_BYTES) + REST_BYTES;
+constexpr int COL_S = 0, COL_O = 128, COL_P = 128 + VDP;
 constexpr int TMEM_COLS = COL_P + 64 <= 256 ? 256 : 512;
 static_assert(!SUPPORTED || SMEM_BYTES <= 227 * 1024, "the stages fit shared memory");
 
@@ -58,6 +75,30 @@ __device__ __forceinline__ float ex2_approx(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));   // ex2(-inf) = +0
   return y;
+}
+
+// What the kernels with OPTIONS take besides (the plain ones ignore it).
+struct AttnOptions {
+  int keep;                          // with a window: the first positions, which stay in sight
+  int dense;                         // keys and values are [tokens][kv heads][channels] of the step's own rows
+  int sink; const float* sink_scores;   // one more term exp(sink score of the head; null: 0) in the denominator
+  const float* gates; long gates_ld; // [tokens][heads] (null: none): times sigmoid
+  float factor;
+};
+// The first of the run of keys that ends at `pos` (the kept positions stand apart from it unless the two touch).
+__device__ __forceinline__ int run_first(int pos, int window, const AttnOptions& opt) {
+  const int f = window > 0 ? max(0, pos - window + 1) : 0;
+  return OPTIONS && f <= opt.keep ? 0 : f;
+}
+// What a row's accumulator is multiplied by: m, l are its reference maximum (log2 domain) and sum.
+__device__ __forceinline__ float row_factor(float m, float l, int token, int head, const AttnOptions& opt) {
+  if constexpr (!OPTIONS) return 1.0f / l;
+  float f = opt.factor;
+  if (opt.gates) f /= 1.0f + expf(-opt.gates[(size_t)token * opt.gates_ld + head]);
+  if (!opt.sink) return f / l;
+  const float s = opt.sink_scores ? opt.sink_scores[head] * 1.4426950408889634f : 0.f;
+  const float M = fmaxf(m, s), fm = ex2_approx(m - M);
+  return f * fm / (l * fm + ex2_approx(s - M));
 }
 
 __device__ __forceinline__ unsigned cluster_rank() { unsigned r; asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r)); return r; }
@@ -90,21 +131,36 @@ __device__ __forceinline__ void zero_spare_rows(unsigned char* q_tile, int RT) {
         *reinterpret_cast<uint4*>(q_tile + c * CHUNK_BYTES + r * 128 + piece * 16) = make_uint4(0, 0, 0, 0);
   fence_proxy_async();
 }
-constexpr int XLD = HD + 4;                       // row stride (floats) of a CTA's published accumulator
+// The row of the cache tensors where the box of position `pos` starts: through the block table (a page that is not
+// there: a box beyond the tensor, fetched as zeros), or among the step's own rows.
+__device__ __forceinline__ int box_row_of(int pos, const int* table, int max_blocks, int page_size, int nkv, int kvh, int cache_rows,
+                                          int tok0, const AttnOptions& opt) {
+  if (OPTIONS && opt.dense) return tok0 + pos;
+  const int blk = pos / page_size;
+  const int page = blk < max_blocks ? table[blk] : -1;
+  return page >= 0 ? (page * nkv + kvh) * page_size + (pos - blk * page_size) : cache_rows;
+}
+__device__ __forceinline__ void load_box(void* dst, const CUtensorMap* map, int col, int row, int kvh, unsigned long long* full,
+                                         const AttnOptions& opt) {
+  if constexpr (OPTIONS) tma_load_3d(dst, map, col, row, opt.dense ? kvh : 0, full);
+  else tma_load_2d(dst, map, col, row, full);
+}
+constexpr int XLD = VDP + 4;                      // row stride (floats) of a CTA's published accumulator
 constexpr int MAX_CLUSTER = 8;
-static_assert(!SUPPORTED || (size_t)(128 * XLD + 256) * 4 <= (size_t)Q_BYTES + (size_t)NST * 2 * KV_BYTES, "a published accumulator fits the tiles");
+static_assert(!SUPPORTED || (size_t)(128 * XLD + 256) * 4 <= (size_t)Q_BYTES + (size_t)NST * (K_BYTES + V_BYTES), "a published accumulator fits the tiles");
 
 __global__ void __launch_bounds__(320, 1)
 attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, long out_stride,
                const int* __restrict__ block_tables, int max_blocks, const int* __restrict__ cu_q,
                const int* __restrict__ kv_lens, int nh, int nkv, int page_size, int cache_rows, int window,
-               float scale_log2, int skip_small, int rows_per_box, int* __restrict__ status, int n_req, int n_units) {
+               float scale_log2, int skip_rows, int rows_per_box, int* __restrict__ status, int n_req, int n_units,
+               AttnOptions opt) {
   extern __shared__ unsigned char smem_raw[];
   unsigned char* tiles = (unsigned char*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   unsigned char* q_s = tiles;                                   // [KCH][128 rows][128 B]
   unsigned char* kv_s = tiles + Q_BYTES;                        // [NST][K, V][KCH][128 rows][128 B]
-  unsigned long long* bars = (unsigned long long*)(kv_s + NST * 2 * KV_BYTES);
+  unsigned long long* bars = (unsigned long long*)(kv_s + NST * (K_BYTES + V_BYTES));
   unsigned long long* q_full = bars;                // 1
   unsigned long long* k_full = bars + 1;            // [NST]
   unsigned long long* v_full = k_full + NST;        // [NST]
@@ -145,15 +201,17 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
   const int G = nh / nkv, TOK = 128 / G, RT = TOK * G;
   const int tok0 = cu_q[b], q_len = cu_q[b + 1] - tok0, kv_len = kv_lens[b];
   const int rows = q_len * G;
-  const bool active = rt * RT < rows && !(skip_small && rows <= 16);
+  const bool active = rt * RT < rows && rows > skip_rows;
   const int base_pos = kv_len - q_len;
   const int row_first = rt * RT, row_last = min(rows, row_first + RT) - 1;
   const int pos_lo = base_pos + row_first / G, pos_hi = base_pos + row_last / G;
-  const int key_first = window > 0 ? max(0, pos_lo - window + 1) : 0;
-  const int all_tiles = active ? pos_hi / BN - key_first / BN + 1 : 0;        // of the row tile
+  const int key_first = run_first(pos_lo, window, opt);
+  const int n_kept = OPTIONS ? min(key_first / BN, (opt.keep + BN - 1) / BN) : 0;     // tiles of kept positions, then the run's
+  const int all_tiles = active ? n_kept + pos_hi / BN - key_first / BN + 1 : 0;       // of the row tile
   const int my_first = all_tiles * crank / csize;                             // rank r: tiles [N r / C, N (r + 1) / C)
   const int n_tiles = all_tiles * (crank + 1) / csize - my_first;             // of this CTA (0 only below the last rank)
-  const int tile_first = key_first / BN + my_first;                           // this CTA's first key tile
+  const int tile_first = key_first / BN + my_first;                           // this CTA's first key tile, without kept ones
+  auto tile_at = [&](int j) { return !OPTIONS ? tile_first + j : my_first + j < n_kept ? my_first + j : tile_first - n_kept + j; };
   const bool merger = crank == csize - 1;
   float* xfer = reinterpret_cast<float*>(q_s);                                // [128][XLD] accumulator, then m[128], l[128]: over the tiles
   // softmax threads' state, finished after the cluster has met
@@ -176,30 +234,25 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
           ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
           if (!ok) break;
         }
-        unsigned char* k_dst = kv_s + (size_t)s * 2 * KV_BYTES;
-        unsigned char* v_dst = k_dst + KV_BYTES;
+        unsigned char* k_dst = kv_s + (size_t)s * (K_BYTES + V_BYTES);
+        unsigned char* v_dst = k_dst + K_BYTES;
         if (lane == 0) {
-          mbar_expect_tx(&k_full[s], (unsigned)KV_BYTES);
-          mbar_expect_tx(&v_full[s], (unsigned)KV_BYTES);
+          mbar_expect_tx(&k_full[s], (unsigned)K_BYTES);
+          mbar_expect_tx(&v_full[s], (unsigned)V_BYTES);
         }
         __syncwarp();
         for (int i = lane; i < boxes; i += 32) {
-          const int pos = (tile_first + j) * BN + i * rows_per_box;
-          const int blk = pos / page_size;
-          const int page = blk < max_blocks ? table[blk] : -1;
-          // a page that is not there: a box beyond the tensor, fetched as zeros
-          const int row = page >= 0 ? (page * nkv + kvh) * page_size + (pos - blk * page_size) : cache_rows;
-          for (int c = 0; c < KCH; ++c)
-            tma_load_2d(k_dst + c * CHUNK_BYTES + i * rows_per_box * 128, &map_k, c * 64, row, &k_full[s]);
-          for (int c = 0; c < KCH; ++c)
-            tma_load_2d(v_dst + c * CHUNK_BYTES + i * rows_per_box * 128, &map_v, c * 64, row, &v_full[s]);
+          const int pos = tile_at(j) * BN + i * rows_per_box;
+          const int row = box_row_of(pos, table, max_blocks, page_size, nkv, kvh, cache_rows, tok0, opt);
+          for (int c = 0; c < KCH; ++c) load_box(k_dst + c * CHUNK_BYTES + i * rows_per_box * 128, &map_k, c * 64, row, kvh, &k_full[s], opt);
+          for (int c = 0; c < VCH; ++c) load_box(v_dst + c * CHUNK_BYTES + i * rows_per_box * 128, &map_v, c * 64, row, kvh, &v_full[s], opt);
         }
       }
     }
   } else if (warp == 1) {
     if (lane == 0 && n_tiles > 0) {
       constexpr unsigned idesc_qk = umma_idesc(128, BN);
-      constexpr unsigned idesc_pv = umma_idesc_b_mn(128, HD);
+      constexpr unsigned idesc_pv = umma_idesc_b_mn(128, VDP);
       bool ok = mbar_wait(q_full, 0);
       if (!ok) atomicExch(status, 32);
       zero_spare_rows(q_s, RT);
@@ -208,7 +261,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         if (!mbar_wait(&k_full[s], (unsigned)(j / NST) & 1)) { atomicExch(status, 33); return false; }
         if (j > 0 && !mbar_wait(s_free, (unsigned)(j - 1) & 1)) { atomicExch(status, 34); return false; }
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        const unsigned char* k_src = kv_s + (size_t)s * 2 * KV_BYTES;
+        const unsigned char* k_src = kv_s + (size_t)s * (K_BYTES + V_BYTES);
 #pragma unroll
         for (int c = 0; c < KCH; ++c) {
           const unsigned long long dq = umma_desc(q_s + c * CHUNK_BYTES), dk = umma_desc(k_src + c * CHUNK_BYTES);
@@ -228,7 +281,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         if (!mbar_wait(p_full, (unsigned)j & 1)) { atomicExch(status, 35); break; }
         if (!mbar_wait(&v_full[s], (unsigned)(j / NST) & 1)) { atomicExch(status, 36); break; }
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        const unsigned char* v_src = kv_s + (size_t)s * 2 * KV_BYTES + KV_BYTES;
+        const unsigned char* v_src = kv_s + (size_t)s * (K_BYTES + V_BYTES) + K_BYTES;
         // One MMA per 16 positions over the whole head dim: operand B MN-major, its 64-column
         // chunks CHUNK_BYTES apart (the leading offset), groups of eight positions 1024 bytes
         // apart (the stride offset).
@@ -252,7 +305,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
     const bool valid = row < RT && row_first + row < rows;
     const int pos = base_pos + (row_first + row) / G;
     const int hi = valid ? pos : -1;
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int lo = run_first(pos, window, opt);
     for (int j = 0; j < n_tiles; ++j) {
       if (!mbar_wait(s_full, (unsigned)j & 1)) { if (lane == 0) atomicExch(status, 37); ok = false; break; }
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -263,9 +316,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       __syncwarp();
       if (lane == 0) mbar_arrive(s_free);
-      const int key0 = (tile_first + j) * BN + half * 64;
+      const int key0 = tile_at(j) * BN + half * 64;
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-      if (!valid || (key0 >= lo && key0 + 63 <= hi)) {
+      if (!valid || (key0 + 63 <= hi && (key0 >= lo || (OPTIONS && key0 + 64 <= opt.keep)))) {
 #pragma unroll
         for (int i = 0; i < 2; ++i)
 #pragma unroll
@@ -276,7 +329,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
 #pragma unroll
           for (int c = 0; c < 32; ++c) {
             const int key = key0 + i * 32 + c;
-            if (key < lo || key > hi) sr[i][c] = __float_as_uint(-INFINITY);
+            if (key > hi || (key < lo && !(OPTIONS && key < opt.keep))) sr[i][c] = __float_as_uint(-INFINITY);
             mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(sr[i][c]));
           }
       }
@@ -319,7 +372,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         if (moved) {
 #pragma unroll 1
-          for (int c0 = half * (HD / 2); c0 < (half + 1) * (HD / 2); c0 += 32) {
+          for (int c0 = half * (VDP / 2); c0 < (half + 1) * (VDP / 2); c0 += 32) {
             unsigned o[32];
             tmem_ld32(lane_addr + COL_O + c0, o);
 #pragma unroll
@@ -347,7 +400,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
       // any more: the last MMA is complete.
       if (half == 0) { xfer[128 * XLD + row] = m; xfer[128 * XLD + 128 + row] = l; }
 #pragma unroll 1
-      for (int c0 = half * (HD / 2); c0 < (half + 1) * (HD / 2); c0 += 32) {
+      for (int c0 = half * (VDP / 2); c0 < (half + 1) * (VDP / 2); c0 += 32) {
         unsigned o[32];
         tmem_ld32(lane_addr + COL_O + c0, o);
 #pragma unroll
@@ -391,11 +444,11 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
       pm[p] = ex2_approx(pm[p] - M_use);           // now the part's factor (0 for a part without tiles)
       den += pl[p] * pm[p];
     }
-    const float inv = 1.0f / den;
     const int rr = row_first + row;
-    bf16* orow = out + (size_t)(tok0 + rr / G) * out_stride + (size_t)(kvh * G + rr % G) * HD;
+    const float inv = row_factor(M, den, tok0 + (valid ? rr / G : 0), kvh * G + rr % G, opt);
+    bf16* orow = out + (size_t)(tok0 + rr / G) * out_stride + (size_t)(kvh * G + rr % G) * VD;
 #pragma unroll 1
-    for (int c0 = half * (HD / 2); c0 < (half + 1) * (HD / 2); c0 += 32) {
+    for (int c0 = half * (VDP / 2); c0 < (half + 1) * (VDP / 2); c0 += 32) {
       unsigned o[32];
       tmem_ld32(lane_addr + COL_O + c0, o);     // warp-collective: invalid rows read too, and skip the store
       float v[32];
@@ -413,6 +466,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
       if (valid) {
 #pragma unroll
         for (int c = 0; c < 32; c += 4) {
+          if (VD < VDP && c0 + c >= VD) break;
           __nv_bfloat162 a = __floats2bfloat162_rn(v[c] * inv, v[c + 1] * inv);
           __nv_bfloat162 d = __floats2bfloat162_rn(v[c + 2] * inv, v[c + 3] * inv);
           uint2 raw;
@@ -450,10 +504,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
 // Key tiles are 128 positions (an MMA instruction takes about 70 cycles however narrow it is).
 // Two K stages and one V stage, released separately; K runs one tile ahead of V.  Tile A sees
 // fewer keys than tile B by at most one key tile and stops early.  Head sizes up to 128.
-constexpr bool TWO_OK = SUPPORTED && HD <= 128;
+constexpr bool TWO_OK = SUPPORTED && HD <= 128 && VD <= 128;
 constexpr int NKS2 = 2;                           // K stages (V has one)
 constexpr int P2_BYTES = 2 * CHUNK_BYTES;         // 128 rows x 128 bfloat16, as two 64-column chunks
-constexpr int SMEM2_BYTES = 2 * Q_BYTES + (NKS2 + 1) * KV_BYTES + 2 * P2_BYTES + 1024 /* alignment slack */ + 256 /* barriers */;
+constexpr int SMEM2_BYTES = 2 * Q_BYTES + NKS2 * K_BYTES + V_BYTES + 2 * P2_BYTES + 1024 /* alignment slack */ + 256 /* barriers */;
 static_assert(!TWO_OK || SMEM2_BYTES <= 227 * 1024, "two query tiles, the stages and the probabilities fit shared memory");
 
 __global__ void __launch_bounds__(320, 1)
@@ -461,13 +515,14 @@ attn_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
                 const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, long out_stride,
                 const int* __restrict__ block_tables, int max_blocks, const int* __restrict__ cu_q,
                 const int* __restrict__ kv_lens, int nh, int nkv, int page_size, int cache_rows, int window,
-                float scale_log2, int skip_small, int rows_per_box, int* __restrict__ status, int n_req, int n_units) {
+                float scale_log2, int skip_rows, int rows_per_box, int* __restrict__ status, int n_req, int n_units,
+               AttnOptions opt) {
   extern __shared__ unsigned char smem_raw[];
   unsigned char* tiles = (unsigned char*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   unsigned char* q_s = tiles;                                   // [tile][KCH][128 rows][128 B]
   unsigned char* k_s = q_s + 2 * Q_BYTES;                       // [NKS2][KCH][128 rows][128 B]
-  unsigned char* v_s = k_s + NKS2 * KV_BYTES;                   // [KCH][128 rows][128 B]
-  unsigned char* p_s = v_s + KV_BYTES;                          // [tile][2][128 rows][128 B]
+  unsigned char* v_s = k_s + NKS2 * K_BYTES;                    // [VCH][128 rows][128 B]
+  unsigned char* p_s = v_s + V_BYTES;                           // [tile][2][128 rows][128 B]
   unsigned long long* bars = (unsigned long long*)(p_s + 2 * P2_BYTES);
   unsigned long long* q_full = bars;                // 1
   unsigned long long* k_full = bars + 1;            // [NKS2]
@@ -506,17 +561,19 @@ attn_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
   const int G = nh / nkv, TOK = 128 / G, RT = TOK * G;
   const int tok0 = cu_q[b], q_len = cu_q[b + 1] - tok0, kv_len = kv_lens[b];
   const int rows = q_len * G;
-  const bool active_a = 2 * pair * RT < rows && !(skip_small && rows <= 16);
+  const bool active_a = 2 * pair * RT < rows && rows > skip_rows;
   const bool active_b = active_a && (2 * pair + 1) * RT < rows;
   const int base_pos = kv_len - q_len;
   const int first_a = 2 * pair * RT, first_b = first_a + RT;
   const int last_a = min(rows, first_a + RT) - 1, last_b = min(rows, first_b + RT) - 1;
   const int pos_lo = base_pos + first_a / G;                                  // the pair's first position
   const int pos_hi_a = base_pos + last_a / G, pos_hi_b = base_pos + last_b / G;
-  const int key_first = window > 0 ? max(0, pos_lo - window + 1) : 0;
+  const int key_first = run_first(pos_lo, window, opt);
+  const int n_kept = OPTIONS ? min(key_first / BN, (opt.keep + BN - 1) / BN) : 0;     // tiles of kept positions, then the run's
   const int tile_first = key_first / BN;
-  const int n_a = active_a ? pos_hi_a / BN - tile_first + 1 : 0;              // key tiles of tile A, of tile B
-  const int n_b = active_b ? pos_hi_b / BN - tile_first + 1 : 0;
+  const int n_a = active_a ? n_kept + pos_hi_a / BN - tile_first + 1 : 0;     // key tiles of tile A, of tile B
+  const int n_b = active_b ? n_kept + pos_hi_b / BN - tile_first + 1 : 0;
+  auto tile_at = [&](int j) { return !OPTIONS ? tile_first + j : j < n_kept ? j : tile_first - n_kept + j; };
   const int n_tiles = n_b > n_a ? n_b : n_a;
 
   if (warp == 0) {
@@ -533,16 +590,13 @@ attn_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
       // there: a box beyond the tensor, fetched as zeros.
       auto box_row = [&](int j) {
         if (lane >= boxes || j >= n_tiles) return 0;
-        const int pos = (tile_first + j) * BN + lane * rows_per_box;
-        const int blk = pos / page_size;
-        const int page = blk < max_blocks ? table[blk] : -1;
-        return page >= 0 ? (page * nkv + kvh) * page_size + (pos - blk * page_size) : cache_rows;
+        return box_row_of(tile_at(j) * BN + lane * rows_per_box, table, max_blocks, page_size, nkv, kvh, cache_rows, tok0, opt);
       };
-      auto fetch = [&](const CUtensorMap* map, unsigned char* dst, int row, unsigned long long* full) {
-        if (lane == 0) mbar_expect_tx(full, (unsigned)KV_BYTES);
+      auto fetch = [&](const CUtensorMap* map, unsigned char* dst, int row, unsigned long long* full, int chunks) {
+        if (lane == 0) mbar_expect_tx(full, (unsigned)(chunks * CHUNK_BYTES));
         __syncwarp();
         if (lane < boxes)
-          for (int c = 0; c < KCH; ++c) tma_load_2d(dst + c * CHUNK_BYTES + lane * rows_per_box * 128, map, c * 64, row, full);
+          for (int c = 0; c < chunks; ++c) load_box(dst + c * CHUNK_BYTES + lane * rows_per_box * 128, map, c * 64, row, kvh, full, opt);
       };
       auto wait_for = [&](unsigned long long* bar, unsigned parity) {
         int ok = 1;
@@ -552,7 +606,7 @@ attn_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
       // K runs one tile ahead of V: K(0), then K(i + 1) and V(i).  The table entries of a tile are
       // read one step before they are needed.
       int row_v = box_row(0), row_k = box_row(1);
-      fetch(&map_k, k_s, row_v, &k_full[0]);
+      fetch(&map_k, k_s, row_v, &k_full[0], KCH);
       bool ok = true;
       for (int i = 0; i < n_tiles && ok; ++i) {
         const int row_next = box_row(i + 2);
@@ -560,24 +614,24 @@ attn_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
           const int s = (i + 1) % NKS2;
           if (i + 1 >= NKS2) ok = wait_for(&k_empty[s], (unsigned)(((i + 1) / NKS2) - 1) & 1);
           if (!ok) break;
-          fetch(&map_k, k_s + (size_t)s * KV_BYTES, row_k, &k_full[s]);
+          fetch(&map_k, k_s + (size_t)s * K_BYTES, row_k, &k_full[s], KCH);
         }
         if (i >= 1) ok = wait_for(v_empty, (unsigned)(i - 1) & 1);
         if (!ok) break;
-        fetch(&map_v, v_s, row_v, v_full);
+        fetch(&map_v, v_s, row_v, v_full, VCH);
         row_v = row_k; row_k = row_next;
       }
     }
   } else if (warp == 1) {
     if (lane == 0 && n_tiles > 0) {
       constexpr unsigned idesc_qk = umma_idesc(128, BN);
-      constexpr unsigned idesc_pv = umma_idesc_b_mn(128, HD);
+      constexpr unsigned idesc_pv = umma_idesc_b_mn(128, VDP);
       bool ok = mbar_wait(q_full, 0);
       if (!ok) atomicExch(status, 32);
       zero_spare_rows(q_s, RT);
       zero_spare_rows(q_s + Q_BYTES, RT);
       auto issue_qk = [&](int t, int j) {        // S_t = Q_t K(j)^T; K(j) has landed and S_t is free
-        const unsigned char* k_src = k_s + (size_t)(j % NKS2) * KV_BYTES;
+        const unsigned char* k_src = k_s + (size_t)(j % NKS2) * K_BYTES;
 #pragma unroll
         for (int c = 0; c < KCH; ++c) {
           const unsigned long long dq = umma_desc(q_s + t * Q_BYTES + c * CHUNK_BYTES), dk = umma_desc(k_src + c * CHUNK_BYTES);
@@ -640,7 +694,7 @@ attn_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
       const bool valid = row < RT && row_first + row < rows;
       const int pos = base_pos + (row_first + row) / G;
       const int hi = valid ? pos : -1;
-      const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+      const int lo = run_first(pos, window, opt);
       float m = -INFINITY, l = 0.f;
       bool ok = true;
       for (int j = 0; j < my_tiles; ++j) {
@@ -653,9 +707,9 @@ attn_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
         asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         __syncwarp();
         if (lane == 0) mbar_arrive(&s_free[t]);
-        const int key0 = (tile_first + j) * BN;
+        const int key0 = tile_at(j) * BN;
         float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-        if (!valid || (key0 >= lo && key0 + BN - 1 <= hi)) {
+        if (!valid || (key0 + BN - 1 <= hi && (key0 >= lo || (OPTIONS && key0 + BN <= opt.keep)))) {
 #pragma unroll
           for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -666,7 +720,7 @@ attn_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
 #pragma unroll
             for (int c = 0; c < 32; ++c) {
               const int key = key0 + i * 32 + c;
-              if (key < lo || key > hi) sr[i][c] = __float_as_uint(-INFINITY);
+              if (key > hi || (key < lo && !(OPTIONS && key < opt.keep))) sr[i][c] = __float_as_uint(-INFINITY);
               mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(sr[i][c]));
             }
         }
@@ -685,7 +739,7 @@ attn_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
           asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
           if (moved) {
 #pragma unroll 1
-            for (int c0 = 0; c0 < HD; c0 += 32) {
+            for (int c0 = 0; c0 < VDP; c0 += 32) {
               unsigned o[32];
               tmem_ld32(lane_addr + col_o + c0, o);
 #pragma unroll
@@ -728,16 +782,17 @@ attn_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       }
       if (ok) {
-        const float inv = 1.0f / l;
         const int rr = row_first + row;
-        bf16* orow = out + (size_t)(tok0 + rr / G) * out_stride + (size_t)(kvh * G + rr % G) * HD;
+        const float inv = row_factor(m, l, tok0 + (valid ? rr / G : 0), kvh * G + rr % G, opt);
+        bf16* orow = out + (size_t)(tok0 + rr / G) * out_stride + (size_t)(kvh * G + rr % G) * VD;
 #pragma unroll 1
-        for (int c0 = 0; c0 < HD; c0 += 32) {
+        for (int c0 = 0; c0 < VDP; c0 += 32) {
           unsigned o[32];
           tmem_ld32(lane_addr + col_o + c0, o);     // warp-collective: invalid rows read too, and skip the store
           if (valid) {
 #pragma unroll
             for (int c = 0; c < 32; c += 4) {
+              if (VD < VDP && c0 + c >= VD) break;
               __nv_bfloat162 a = __floats2bfloat162_rn(__uint_as_float(o[c]) * inv, __uint_as_float(o[c + 1]) * inv);
               __nv_bfloat162 d = __floats2bfloat162_rn(__uint_as_float(o[c + 2]) * inv, __uint_as_float(o[c + 3]) * inv);
               uint2 raw;
@@ -775,15 +830,16 @@ bool coheryn_attention_tc_takes(int nh, int nkv, int page_size) {
   return page_size >= 8 && (BN % page_size == 0 || page_size % BN == 0);   // a box is whole pages of >= 1024 bytes
 }
 
-int coheryn_attention_tc_launch(const void* q, long q_stride, int total_tokens, void* out, long out_stride,
+// The launch behind both interfaces.  skip_rows: requests with at most this many rows per kv head are left out.
+static int attention_tc_launch(const void* q, long q_stride, int total_tokens, void* out, long out_stride,
                                 const void* k_cache, const void* v_cache, int num_pages, const int* block_tables,
                                 int max_blocks, const int* cu_q, const int* kv_lens, int B, int nh, int nkv,
-                                int page_size, int window, float scale_log2, int max_rows, int max_kv_len, int skip_small,
-                                int* status, cudaStream_t stream) {
-  if (!SUPPORTED) CO_FAIL("attention_tc: head size %d is not a multiple of 64 up to 256", HD);
+                                int page_size, int window, float scale_log2, int max_rows, int max_kv_len, int skip_rows,
+                                int* status, const AttnOptions& opt, cudaStream_t stream) {
+  if (!SUPPORTED) CO_FAIL("attention_tc: head sizes %d and %d are not built", HD, VD);
   const int G = nh / nkv, TOK = 128 / G, RT = TOK * G;
-  const int rows_per_box = page_size < BN ? page_size : BN;
-  const long cache_rows = (long)num_pages * nkv * page_size;
+  const int rows_per_box = opt.dense || page_size >= BN ? BN : page_size;
+  const long cache_rows = opt.dense ? total_tokens : (long)num_pages * nkv * page_size;
   if (cache_rows >= (1L << 31)) CO_FAIL("attention_tc: the cache holds %ld rows per tensor, beyond 2^31", cache_rows);
   CUtensorMap mq, mk, mv;
   {
@@ -793,11 +849,15 @@ int coheryn_attention_tc_launch(const void* q, long q_stride, int total_tokens, 
     if (!make_map_nd(&mq, q, 3, dims, strides, box)) CO_FAIL("attention_tc: the query tensor map was refused");
   }
   {
-    cuuint64_t dims[2] = {(cuuint64_t)HD, (cuuint64_t)cache_rows};
-    cuuint64_t strides[1] = {(cuuint64_t)HD * 2};
-    cuuint32_t box[2] = {64, (cuuint32_t)rows_per_box};
-    if (!make_map_nd(&mk, k_cache, 2, dims, strides, box) || !make_map_nd(&mv, v_cache, 2, dims, strides, box))
-      CO_FAIL("attention_tc: the cache tensor map was refused");
+    // pages: rows of one head after the other; dense: the heads of a token side by side
+    auto map_of = [&](CUtensorMap* map, const void* base, int width) {
+      const int heads = opt.dense ? nkv : 1;
+      cuuint64_t dims[3] = {(cuuint64_t)width, (cuuint64_t)cache_rows, (cuuint64_t)heads};
+      cuuint64_t strides[2] = {(cuuint64_t)width * 2 * heads, opt.dense ? (cuuint64_t)width * 2 : (cuuint64_t)cache_rows * width * 2};
+      cuuint32_t box[3] = {64, (cuuint32_t)rows_per_box, 1};
+      return make_map_nd(map, base, OPTIONS ? 3 : 2, dims, strides, box);
+    };
+    if (!map_of(&mk, k_cache, HD) || !map_of(&mv, v_cache, VD)) CO_FAIL("attention_tc: the cache tensor map was refused");
   }
   static bool configured = false;
   if (!configured) {
@@ -838,7 +898,7 @@ int coheryn_attention_tc_launch(const void* q, long q_stride, int total_tokens, 
     dim3 grid2((unsigned)pair_ctas);
     cudaError_t le2 = co_launch(attn_tc2_kernel, grid2, dim3(320), (size_t)SMEM2_BYTES, stream, mq, mk, mv, (bf16*)out, out_stride,
                                 block_tables, max_blocks, cu_q, kv_lens, nh, nkv, page_size, (int)cache_rows, window, scale_log2,
-                                skip_small, rows_per_box, status, B, pairs);
+                                skip_rows, rows_per_box, status, B, pairs, opt);
     if (le2 != cudaSuccess) CO_FAIL("attention_tc: launch failed: %s", cudaGetErrorString(le2));
     CO_CHECK_LAUNCH("attn_tc2");
     return 0;
@@ -847,8 +907,49 @@ int coheryn_attention_tc_launch(const void* q, long q_stride, int total_tokens, 
   dim3 grid((unsigned)(ctas * cluster));
   cudaError_t le = co_launch_cluster(cluster, attn_tc_kernel, grid, dim3(320), (size_t)SMEM_BYTES, stream, mq, mk, mv, (bf16*)out,
                                      out_stride, block_tables, max_blocks, cu_q, kv_lens, nh, nkv, page_size, (int)cache_rows,
-                                     window, scale_log2, skip_small, rows_per_box, status, B, row_tiles);
+                                     window, scale_log2, skip_rows, rows_per_box, status, B, row_tiles, opt);
   if (le != cudaSuccess) CO_FAIL("attention_tc: launch failed: %s", cudaGetErrorString(le));
   CO_CHECK_LAUNCH("attn_tc");
   return 0;
 }
+
+#ifndef CO_VALUE_DIM
+int coheryn_attention_tc_launch(const void* q, long q_stride, int total_tokens, void* out, long out_stride,
+                                const void* k_cache, const void* v_cache, int num_pages, const int* block_tables,
+                                int max_blocks, const int* cu_q, const int* kv_lens, int B, int nh, int nkv,
+                                int page_size, int window, float scale_log2, int max_rows, int max_kv_len, int skip_small,
+                                int* status, cudaStream_t stream) {
+  return attention_tc_launch(q, q_stride, total_tokens, out, out_stride, k_cache, v_cache, num_pages, block_tables, max_blocks,
+                             cu_q, kv_lens, B, nh, nkv, page_size, window, scale_log2, max_rows, max_kv_len, skip_small ? 16 : 0,
+                             status, AttnOptions{}, stream);
+}
+#else
+CO_EXPORT void coheryn_attention_options_shape(int* dk, int* dv) { *dk = HD; *dv = VD; }
+CO_EXPORT void coheryn_attention_options_set_cluster(int cluster) { coheryn_attention_tc_set_cluster(cluster); }
+CO_EXPORT void coheryn_attention_options_set_two_tiles(int mode) { coheryn_attention_tc_set_two_tiles(mode); }
+
+// The attention of every request that brings more than one token.  q: [total_tokens][nh][HD] bfloat16 rows of stride
+// q_stride; caches: [num_pages][nkv][page_size][HD or VD], or with `dense` [total_tokens][nkv][HD or VD], the step's own
+// rows (whole prompts; num_pages and block_tables are not read).  gates: float32 [total_tokens, nh] with row stride
+// gates_ld.  max_rows and max_kv_len bound the rows per kv head (tokens * heads per kv head) and the lengths.
+CO_EXPORT int coheryn_attention_options(const void* q, long q_stride, int total_tokens, void* out, long out_stride,
+                                        const void* k_cache, const void* v_cache, int num_pages, const int* block_tables,
+                                        int max_blocks, const int* cu_q, const int* kv_lens, int B, int nh, int nkv, int page_size,
+                                        int window, int keep, int dense, int sink, const float* sink_scores, const float* gates,
+                                        long gates_ld, float factor, float scale, int max_rows, int max_kv_len, int* status,
+                                        cudaStream_t stream) {
+  if (B <= 0 || total_tokens <= 0) return 0;
+  if (!dense && !coheryn_attention_tc_takes(nh, nkv, page_size)) CO_FAIL("attention_options: %d heads over %d, pages of %d", nh, nkv, page_size);
+  if (nkv <= 0 || nh % nkv || nh / nkv > 128) CO_FAIL("attention_options: %d heads do not group over %d kv heads", nh, nkv);
+  if (!(scale > 0.f)) CO_FAIL("attention_options: the scale must be positive");
+  if (keep < 0 || (keep > 0 && window <= 0)) CO_FAIL("attention_options: kept first positions stand beside a window (%d kept)", keep);
+  if ((q_stride & 7) || ((uintptr_t)q & 15) || ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15))
+    CO_FAIL("attention_options: rows of q, k and v must start on 16-byte boundaries");
+  if ((out_stride & 3) || ((uintptr_t)out & 7)) CO_FAIL("attention_options: rows of the output must start on 8-byte boundaries");
+  if (!status) CO_FAIL("attention_options: a status word is required");
+  const AttnOptions opt{keep, dense, sink, sink_scores, gates, gates_ld, factor};
+  return attention_tc_launch(q, q_stride, total_tokens, out, out_stride, k_cache, v_cache, num_pages, block_tables, max_blocks, cu_q,
+                             kv_lens, B, nh, nkv, page_size, window, scale * 1.4426950408889634f, max_rows, max_kv_len, nh / nkv, status,
+                             opt, stream);
+}
+#endif

@@ -127,6 +127,134 @@ unit_norm_rope_kv_write_kernel(const float* __restrict__ q, const float* __restr
   }
 }
 
+// The same for sizes in multiples of four channels and rows on 16-byte boundaries: a warp takes a unit, a lane four
+// neighbouring channels (of 128 at a time), every global access is 16 bytes of float32 or 8 of bfloat16.
+template <typename T>
+__device__ __forceinline__ void store4(T* p, float4 v);
+template <>
+__device__ __forceinline__ void store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <>
+__device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<const unsigned*>(&lo);
+  u.y = *reinterpret_cast<const unsigned*>(&hi);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+__device__ __forceinline__ float4 load4_any(const void* p, int dtype, size_t i) {
+  if (dtype == CO_F32) return *reinterpret_cast<const float4*>((const float*)p + i);
+  const uint2 u = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)p + i);
+  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
+}
+template <typename T>
+__global__ void __launch_bounds__(256)
+unit_norm_rope_kv_write_vec_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v, long ld,
+                                   const void* __restrict__ wq, const void* __restrict__ wk, int w_dtype, float eps, int normalise,
+                                   const int* __restrict__ positions, const float* __restrict__ freq, int rot, float rot_scale,
+                                   T* __restrict__ q_out, long ldq, const int* __restrict__ slots, T* __restrict__ k_cache,
+                                   T* __restrict__ v_cache, int q_units, int k_units, int nkv, int dk, int dv, int page_size,
+                                   const float* __restrict__ v_first, long ldf, float keep_v, float mix_v) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float whole_s[2];
+  co_pdl_launch_dependents();
+  co_pdl_wait();
+  const size_t t = blockIdx.x;
+  const int half = rot / 2;
+  const int write = slots != nullptr;
+  const int units = q_units + (write ? k_units : 0);
+  float* cosines = sm;                 // [half]
+  float* sines = sm + half;            // [half]
+  float* xs = sm + 2 * half;           // [units][dk]
+  float* scale_s = xs + (size_t)units * dk;      // [units]
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const float* qr = q + t * ld;
+  const float* kr = k + t * ld;
+#pragma unroll 2
+  for (int u = warp; u < units; u += 8) {
+    const float* src = u < q_units ? qr + (size_t)u * dk : kr + (size_t)(u - q_units) * dk;
+    float ss = 0.f;
+    for (int d = 4 * lane; d < dk; d += 128) {
+      const float4 x = *reinterpret_cast<const float4*>(src + d);
+      *reinterpret_cast<float4*>(xs + u * dk + d) = x;
+      ss = fmaf(x.x, x.x, ss); ss = fmaf(x.y, x.y, ss); ss = fmaf(x.z, x.z, ss); ss = fmaf(x.w, x.w, ss);
+    }
+    if (normalise) {
+      ss = co_warp_sum(ss);
+      if (lane == 0) scale_s[u] = normalise == 2 ? ss : 1.0f / sqrtf(ss / (float)dk + eps);
+    }
+  }
+  if (rot) {
+    const float p = (float)positions[t];
+    for (int i = threadIdx.x; i < half; i += 256) {
+      const float fh = freq[2 * i], fl = freq[2 * i + 1];
+      const float ah = p * fh;
+      const float al = fmaf(p, fh, -ah) + p * fl;
+      float s, c, sl, cl;
+      sincosf(ah, &s, &c);
+      sincosf(al, &sl, &cl);
+      cosines[i] = (c * cl - s * sl) * rot_scale;
+      sines[i] = (s * cl + c * sl) * rot_scale;
+    }
+  }
+  __syncthreads();
+  if (normalise == 2) {
+    if (warp < 2) {      // the sums of a side's units, added in a fixed order
+      const int u0 = warp ? q_units : 0, n = warp ? units - q_units : q_units;
+      float ss = 0.f;
+      for (int u = lane; u < n; u += 32) ss += scale_s[u0 + u];
+      ss = co_warp_sum(ss);
+      if (lane == 0) whole_s[warp] = n > 0 ? 1.0f / sqrtf(ss / ((float)n * (float)dk) + eps) : 0.f;
+    }
+    __syncthreads();
+  }
+  int slot = 0;
+  size_t page = 0, off = 0;
+  if (write) { slot = slots[t]; page = (size_t)(slot / page_size); off = (size_t)(slot % page_size); }
+  const int maps = k_units / (nkv > 0 ? nkv : 1);
+#pragma unroll 2
+  for (int u = warp; u < units; u += 8) {
+    const bool is_q = u < q_units;
+    const int ku = is_q ? u : u - q_units;
+    if (!is_q && slot < 0) continue;
+    const void* w = is_q ? wq : wk;
+    const float scale = normalise == 2 ? whole_s[is_q ? 0 : 1] : normalise ? scale_s[u] : 1.f;
+    const size_t w0 = normalise == 2 ? (size_t)ku * dk : 0;
+    T* dst = is_q ? q_out + t * ldq + (size_t)u * dk
+                  : k_cache + ((page * nkv + ku / maps) * page_size + off) * ((size_t)maps * dk) + (size_t)(ku % maps) * dk;
+    auto val = [&](int d) {
+      float4 x = *reinterpret_cast<const float4*>(xs + u * dk + d);
+      if (normalise) {
+        const float4 g = load4_any(w, w_dtype, w0 + d);
+        x = make_float4((x.x * scale) * g.x, (x.y * scale) * g.y, (x.z * scale) * g.z, (x.w * scale) * g.w);
+      }
+      return x;
+    };
+    for (int d = 4 * lane; d < dk; d += 128) {
+      float4 y = val(d);
+      if (d < rot) {
+        const bool low = d < half;
+        const float4 o = val(low ? d + half : d - half);
+        const float4 c = *reinterpret_cast<const float4*>(cosines + (low ? d : d - half));
+        float4 s = *reinterpret_cast<const float4*>(sines + (low ? d : d - half));
+        if (low) s = make_float4(-s.x, -s.y, -s.z, -s.w);
+        y = make_float4(y.x * c.x + o.x * s.x, y.y * c.y + o.y * s.y, y.z * c.z + o.z * s.z, y.w * c.w + o.w * s.w);
+      }
+      store4<T>(dst + d, y);
+    }
+  }
+  if (!write || slot < 0) return;
+  const float* vr = v + t * ld;
+  for (int e = 4 * threadIdx.x; e < nkv * dv; e += 1024) {
+    const int g = e / dv, d = e - g * dv;
+    float4 x = *reinterpret_cast<const float4*>(vr + e);
+    if (v_first) {
+      const float4 f = *reinterpret_cast<const float4*>(v_first + t * ldf + e);
+      x = make_float4(keep_v * x.x + mix_v * f.x, keep_v * x.y + mix_v * f.y, keep_v * x.z + mix_v * f.z, keep_v * x.w + mix_v * f.w);
+    }
+    store4<T>(v_cache + ((page * nkv + g) * page_size + off) * dv + d, x);
+  }
+}
+
 // ---------------------------------------------------------------------------------
 // One CTA per (token, query head); four warps each run an online softmax per map over the keys
 // n = warp, warp + 4, .. (kept first positions, then those from the first visible one on); their (maximum, sum, accumulator) triples are merged in warp order.
@@ -338,9 +466,12 @@ CO_EXPORT int coheryn_unit_norm_rope_kv_write(const float* q, const float* k, co
   const int units = q_units + (slots ? k_units : 0);
   const size_t smem = ((size_t)rot + units + (size_t)units * dk) * sizeof(float);
   if (smem > 200 * 1024) CO_FAIL("unit_norm_rope_kv_write: %d units of %d channels do not fit in shared memory", units, dk);
+  const auto on16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };      // (null counts as aligned)
+  const bool vec = (dk & 3) == 0 && (dv & 3) == 0 && (rot & 7) == 0 && (ld & 3) == 0 && (ldq & 3) == 0 && (ldf & 3) == 0 && on16(q) && on16(k) &&
+                   on16(v) && on16(wq) && on16(wk) && on16(q_out) && on16(k_cache) && on16(v_cache) && on16(v_first);
 #define GO(TT)                                                                                                        \
   {                                                                                                                   \
-    auto kern = unit_norm_rope_kv_write_kernel<TT>;                                                                   \
+    auto kern = vec ? unit_norm_rope_kv_write_vec_kernel<TT> : unit_norm_rope_kv_write_kernel<TT>;                    \
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);          \
     co_launch(kern, dim3(T), dim3(256), smem, stream, q, k, v, ld, wq, wk, w_dtype, eps, normalise, positions, freq, rot, \
               rot_scale, (TT*)q_out, ldq, slots, (TT*)k_cache, (TT*)v_cache, q_units, k_units, nkv, dk, dv, page_size, v_first, \

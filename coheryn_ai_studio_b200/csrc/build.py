@@ -241,6 +241,14 @@ def attention_library(head_dim: int) -> ctypes.CDLL:
                         {"CO_HEAD_DIM": head_dim})
 
 
+def attention_options_library(dk: int, dv: int) -> ctypes.CDLL:
+    """The tcgen05 attention for prompt portions with options (other value sizes, kept first positions, sink, head gates,
+    dense keys), compiled for one (key channels, value channels) when a model needs it."""
+    if dk % 16 or dv % 16 or not 16 <= dk <= 256 or not 16 <= dv <= 256:
+        raise BuildError(f"the attention with options takes head sizes 16..256 in steps of 16, not ({dk}, {dv})")
+    return load_library(f"attn_options_{dk}_{dv}", ["attention_tc.cu", "runtime.cu"], {"CO_HEAD_DIM": dk, "CO_VALUE_DIM": dv})
+
+
 def recurrent_library() -> ctypes.CDLL:
     """The kernels of mixers with a state of fixed size per request (short convolution, gated delta rule,
     matrix memory), compiled when a model with such a mixer is first run."""
@@ -321,6 +329,7 @@ def build_all(head_dims: Sequence[int] = (16, 32, 64, 128)) -> List[str]:
              build_library("pooled_tc_128_128", ["attention_pooled_tc.cu", "runtime.cu"], {"CO_PW_DK": 128, "CO_PW_DV": 128})]
     paths.append(build_library("maps_96_64_1_vk", ["attention_maps_tc.cu", "runtime.cu"],
                                {"CO_MAPS_DK": 96, "CO_MAPS_DV": 64, "CO_MAPS_N": 1, "CO_MAPS_V_IN_K": 1}))
+    paths.append(build_library("attn_options_96_64", ["attention_tc.cu", "runtime.cu"], {"CO_HEAD_DIM": 96, "CO_VALUE_DIM": 64}))
     for dk, dv, maps in ((64, 128, 2), (64, 64, 1)):
         paths.append(build_library(f"maps_{dk}_{dv}_{maps}", ["attention_maps_tc.cu", "runtime.cu"],
                                    {"CO_MAPS_DK": dk, "CO_MAPS_DV": dv, "CO_MAPS_N": maps}))

@@ -24,7 +24,7 @@ namespace {
 constexpr int CH = 64;            // tokens per chunk
 constexpr int TP = CH + 4;        // pitch of a [channel][token] tile that is read four tokens at a time
 constexpr int SL = 32;            // channels (or tokens) per slice of the output kernel
-constexpr int FC = 32;            // value channels per CTA of the kernel for few tokens
+constexpr int FC = 32;            // value channels per CTA of the kernel for few tokens, times its column groups
 
 struct LightningArgs {
   const float* q; long ldq; const float* k; long ldk; const float* v; long ldv;
@@ -46,31 +46,35 @@ __device__ __forceinline__ void li_axpy(float4& o, float a, const float4& x) {
 }
 
 // ------------------------------------------------------------------------------------------- few tokens per request
-// grid (H, ceil(dv / FC), B), 256 threads.  Eight neighbouring lanes own four columns each; lane group g of the 32 owns the
-// rows g, g + 32, .. of S.  ROWS: rows a thread keeps in registers (0: the state stays in memory, for dk > 256).
-// smem: q, k [L][dk], v [L][FC], the warps' partial outputs [L][8][FC]; L = tokens of the longest run.
-template <int ROWS>
-__global__ void __launch_bounds__(256) lightning_few_kernel(LightningArgs A, int L, bool vec) {
+// grid (H, ceil(dv / (FC NC)), B), 256 threads.  Eight neighbouring lanes own four columns each of every column group; lane
+// group g of the 32 owns the rows g, g + 32, .. of S.  ROWS: rows a thread keeps in registers (0: the state stays in memory,
+// for dk > 256).  NC: column groups of a CTA (two where many heads and requests fill the GPU by themselves).
+// smem: q, k [L][dk], v [L][CW], the warps' partial outputs [L][8][CW]; L = tokens of the longest run.
+template <int ROWS, int NC>
+__global__ void __launch_bounds__(256, NC == 2 ? 3 : 1) lightning_few_kernel(LightningArgs A, int L, bool vec) {
+  constexpr int CW = FC * NC;
   extern __shared__ __align__(16) float sm[];
   co_pdl_launch_dependents();
-  const int h = blockIdx.x, c0 = blockIdx.y * FC, b = blockIdx.z, dk = A.dk, dv = A.dv;
+  const int h = blockIdx.x, c0 = blockIdx.y * CW, b = blockIdx.z, dk = A.dk, dv = A.dv;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int g = threadIdx.x >> 3, c = c0 + 4 * (lane & 7);
-  float* part = sm;                     // [L][8][FC]
-  float* vs = part + L * 8 * FC;        // [L][FC]
-  float* qs = vs + L * FC;
+  float* part = sm;                     // [L][8][CW]
+  float* vs = part + L * 8 * CW;        // [L][CW]
+  float* qs = vs + L * CW;
   float* ks = qs + L * dk;
   const float am1 = A.powers[(size_t)h * 2 * (CH + 1) + CH + 1 + 1];
   co_pdl_wait();
   const int t0 = A.cu_q[b], n = A.cu_q[b + 1] - t0;
   if (n <= 0) return;
   float* S = A.state + (size_t)A.state_slots[b] * A.state_stride + (size_t)h * dk * dv;
-  float4 s[ROWS > 0 ? ROWS : 1];
+  float4 s[ROWS > 0 ? ROWS : 1][NC];
   if (ROWS > 0) {                       // in flight while the projections are read
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
       const int d = g + 32 * i;
-      s[i] = d < dk && c < dv ? la_load4(S + (size_t)d * dv, c, dv, vec) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int j = 0; j < NC; ++j)
+        s[i][j] = d < dk && c + FC * j < dv ? la_load4(S + (size_t)d * dv, c + FC * j, dv, vec) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
   }
   for (int e = threadIdx.x; e < n * dk; e += 256) {
@@ -79,52 +83,57 @@ __global__ void __launch_bounds__(256) lightning_few_kernel(LightningArgs A, int
     qs[e] = li_act(A.silu, A.q[row * A.ldq + ch]);
     ks[e] = li_act(A.silu, A.k[row * A.ldk + ch]);
   }
-  for (int e = threadIdx.x; e < n * FC; e += 256) {
-    const int t = e / FC, x = e - t * FC;
+  for (int e = threadIdx.x; e < n * CW; e += 256) {
+    const int t = e / CW, x = e - t * CW;
     vs[e] = c0 + x < dv ? li_act(A.silu, A.v[(size_t)(t0 + t) * A.ldv + (size_t)h * dv + c0 + x]) : 0.f;
   }
   __syncthreads();
   for (int t = 0; t < n; ++t) {
-    const float4 vv = *reinterpret_cast<const float4*>(vs + t * FC + 4 * (lane & 7));
-    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-    auto step = [&](float4& x, int d) {
-      const float kd = ks[t * dk + d], qd = qs[t * dk + d];
-      x.x += fmaf(kd, vv.x, am1 * x.x); x.y += fmaf(kd, vv.y, am1 * x.y);
-      x.z += fmaf(kd, vv.z, am1 * x.z); x.w += fmaf(kd, vv.w, am1 * x.w);
-      li_axpy(o, qd, x);
-    };
-    if (ROWS > 0) {
 #pragma unroll
-      for (int i = 0; i < ROWS; ++i)
-        if (g + 32 * i < dk) step(s[i], g + 32 * i);
-    } else if (c < dv) {
-      for (int d = g; d < dk; d += 32) {
-        float4 x = la_load4(S + (size_t)d * dv, c, dv, vec);
-        step(x, d);
-        la_store4(S + (size_t)d * dv, c, dv, vec, x);
+    for (int j = 0; j < NC; ++j) {
+      const float4 vv = *reinterpret_cast<const float4*>(vs + t * CW + FC * j + 4 * (lane & 7));
+      float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+      auto step = [&](float4& x, int d) {
+        const float kd = ks[t * dk + d], qd = qs[t * dk + d];
+        x.x += fmaf(kd, vv.x, am1 * x.x); x.y += fmaf(kd, vv.y, am1 * x.y);
+        x.z += fmaf(kd, vv.z, am1 * x.z); x.w += fmaf(kd, vv.w, am1 * x.w);
+        li_axpy(o, qd, x);
+      };
+      if (ROWS > 0) {
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i)
+          if (g + 32 * i < dk) step(s[i][j], g + 32 * i);
+      } else if (c + FC * j < dv) {
+        for (int d = g; d < dk; d += 32) {
+          float4 x = la_load4(S + (size_t)d * dv, c + FC * j, dv, vec);
+          step(x, d);
+          la_store4(S + (size_t)d * dv, c + FC * j, dv, vec, x);
+        }
       }
-    }
 #pragma unroll
-    for (int off = 8; off < 32; off <<= 1) {       // the warp's four lane groups
-      o.x += __shfl_xor_sync(0xffffffffu, o.x, off); o.y += __shfl_xor_sync(0xffffffffu, o.y, off);
-      o.z += __shfl_xor_sync(0xffffffffu, o.z, off); o.w += __shfl_xor_sync(0xffffffffu, o.w, off);
+      for (int off = 8; off < 32; off <<= 1) {       // the warp's four lane groups
+        o.x += __shfl_xor_sync(0xffffffffu, o.x, off); o.y += __shfl_xor_sync(0xffffffffu, o.y, off);
+        o.z += __shfl_xor_sync(0xffffffffu, o.z, off); o.w += __shfl_xor_sync(0xffffffffu, o.w, off);
+      }
+      if (lane < 8) *reinterpret_cast<float4*>(part + (t * 8 + warp) * CW + FC * j + 4 * lane) = o;
     }
-    if (lane < 8) *reinterpret_cast<float4*>(part + (t * 8 + warp) * FC + 4 * lane) = o;
   }
   if (ROWS > 0) {
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
       const int d = g + 32 * i;
-      if (d < dk && c < dv) la_store4(S + (size_t)d * dv, c, dv, vec, s[i]);
+#pragma unroll
+      for (int j = 0; j < NC; ++j)
+        if (d < dk && c + FC * j < dv) la_store4(S + (size_t)d * dv, c + FC * j, dv, vec, s[i][j]);
     }
   }
   __syncthreads();
-  for (int e = threadIdx.x; e < n * FC; e += 256) {
-    const int t = e / FC, x = e - t * FC;
+  for (int e = threadIdx.x; e < n * CW; e += 256) {
+    const int t = e / CW, x = e - t * CW;
     if (c0 + x >= dv) continue;
     float o = 0.f;
 #pragma unroll
-    for (int w = 0; w < 8; ++w) o += part[(t * 8 + w) * FC + x];
+    for (int w = 0; w < 8; ++w) o += part[(t * 8 + w) * CW + x];
     A.o_raw[(size_t)(t0 + t) * ((size_t)A.H * dv) + (size_t)h * dv + c0 + x] = o;
   }
 }
@@ -407,6 +416,53 @@ __global__ void __launch_bounds__(256, 2) lightning_chunk_out_kernel(LightningAr
   }
 }
 
+// The same with a token's row in registers: n a multiple of 4 and at most 512 * 4 * VPT, every row on a 16-byte boundary.
+// Row, gate and weight are requested together, ahead of the sum over the row.
+template <typename TO, int VPT>
+__global__ void __launch_bounds__(512) lightning_norm_vec_kernel(const float* __restrict__ o, const void* __restrict__ w, int w_dtype,
+                                                                 const float* __restrict__ gate, long ldg, int gate_act, float eps,
+                                                                 float factor, TO* __restrict__ out, long ldo, int n) {
+  __shared__ float scratch[33];
+  co_pdl_launch_dependents();
+  const size_t t = blockIdx.x;
+  float4 x[VPT], g[VPT], wv[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {      // no earlier kernel writes the weight
+    const int j = 4 * (threadIdx.x + i * blockDim.x);
+    if (j < n) wv[i] = make_float4(co_load_any(w, w_dtype, j), co_load_any(w, w_dtype, j + 1), co_load_any(w, w_dtype, j + 2), co_load_any(w, w_dtype, j + 3));
+  }
+  co_pdl_wait();
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int j = 4 * (threadIdx.x + i * blockDim.x);
+    x[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (j < n) {
+      x[i] = *reinterpret_cast<const float4*>(o + t * n + j);
+      g[i] = *reinterpret_cast<const float4*>(gate + t * ldg + j);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) { ss = fmaf(x[i].x, x[i].x, ss); ss = fmaf(x[i].y, x[i].y, ss); ss = fmaf(x[i].z, x[i].z, ss); ss = fmaf(x[i].w, x[i].w, ss); }
+  const float inv = 1.0f / sqrtf(co_block_sum(ss, scratch) / (float)n + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int j = 4 * (threadIdx.x + i * blockDim.x);
+    if (j >= n) continue;
+    const float y[4] = {(x[i].x * inv) * wv[i].x * la_gate(gate_act, g[i].x) * factor, (x[i].y * inv) * wv[i].y * la_gate(gate_act, g[i].y) * factor,
+                        (x[i].z * inv) * wv[i].z * la_gate(gate_act, g[i].z) * factor, (x[i].w * inv) * wv[i].w * la_gate(gate_act, g[i].w) * factor};
+    if constexpr (sizeof(TO) == 2) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(y[0], y[1]), hi = __floats2bfloat162_rn(y[2], y[3]);
+      uint2 u;
+      u.x = *reinterpret_cast<const unsigned*>(&lo);
+      u.y = *reinterpret_cast<const unsigned*>(&hi);
+      *reinterpret_cast<uint2*>(out + t * ldo + j) = u;
+    } else {
+      *reinterpret_cast<float4*>(out + t * ldo + j) = make_float4(y[0], y[1], y[2], y[3]);
+    }
+  }
+}
+
 // grid (T), 256 threads: all heads of a token normalised together, times the weight, the gate and a factor.
 template <typename TO>
 __global__ void __launch_bounds__(256) lightning_norm_kernel(const float* __restrict__ o, const void* __restrict__ w, int w_dtype,
@@ -428,7 +484,7 @@ __global__ void __launch_bounds__(256) lightning_norm_kernel(const float* __rest
     out[t * ldo + j] = co_from_float<TO>((row_s[j] * inv) * co_load_any(w, w_dtype, j) * la_gate(gate_act, gate[t * ldg + j]) * factor);
 }
 
-size_t few_smem(int L, int dk) { return ((size_t)L * 9 * FC + (size_t)2 * L * dk) * sizeof(float); }
+size_t few_smem(int L, int dk, int columns) { return ((size_t)L * 9 * columns + (size_t)2 * L * dk) * sizeof(float); }
 size_t state_smem(int vt) { return ((size_t)CH * 64 + (size_t)CH * vt) * sizeof(float); }
 size_t out_smem(int dk, int vt) {
   const size_t slices = (dk + SL - 1) / SL, tiles = (size_t)2 * SL * vt, keys = (size_t)2 * SL * TP;
@@ -463,14 +519,17 @@ CO_EXPORT int coheryn_lightning(const float* q, long ldq, const float* k, long l
   const bool vec_state = (dv & 3) == 0 && (state_stride & 3) == 0 && aligned(state);
   if (max_q_len <= few) {
     A.o_raw = scratch;
-    const size_t smem = few_smem(max_q_len, dk);
+    // twice the columns per CTA once three rounds of the narrow ones would be needed
+    const bool wide = dk <= 128 && dv > FC && (long)H * ((dv + FC - 1) / FC) * B > 3 * 148 * 2;
+    const size_t smem = few_smem(max_q_len, dk, wide ? 2 * FC : FC);
     if (smem > SMEM_LIMIT) CO_FAIL("lightning: %d tokens of %d key channels do not fit a CTA", max_q_len, dk);
-#define GO(ROWS)                                                                                                              \
+#define GO(ROWS, NC)                                                                                                          \
   do {                                                                                                                        \
-    if (smem > 48 * 1024) cudaFuncSetAttribute(lightning_few_kernel<ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-    co_launch(lightning_few_kernel<ROWS>, dim3(H, (dv + FC - 1) / FC, B), dim3(256), smem, stream, A, max_q_len, vec_state);  \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(lightning_few_kernel<ROWS, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    co_launch(lightning_few_kernel<ROWS, NC>, dim3(H, (dv + FC * NC - 1) / (FC * NC), B), dim3(256), smem, stream, A, max_q_len, vec_state); \
   } while (0)
-    if (dk <= 32) GO(1); else if (dk <= 64) GO(2); else if (dk <= 128) GO(4); else if (dk <= 256) GO(8); else GO(0);
+    if (wide) { if (dk <= 32) GO(1, 2); else if (dk <= 64) GO(2, 2); else GO(4, 2); }
+    else if (dk <= 32) GO(1, 1); else if (dk <= 64) GO(2, 1); else if (dk <= 128) GO(4, 1); else if (dk <= 256) GO(8, 1); else GO(0, 1);
 #undef GO
     CO_CHECK_LAUNCH("lightning_few");
   } else {
@@ -501,6 +560,17 @@ CO_EXPORT int coheryn_lightning(const float* q, long ldq, const float* k, long l
     CO_CHECK_LAUNCH("lightning_chunk_out");
   }
   const int n = H * dv;
+  if ((n & 3) == 0 && n <= 512 * 4 * 4 && (ldg & 3) == 0 && (ldo & 3) == 0 && aligned(gate) && aligned(out) && aligned(A.o_raw)) {
+    const int threads = n / 4 >= 512 ? 512 : (n / 4 + 31) / 32 * 32;
+#define GO(TO, VPT)                                                                                                           \
+  co_launch(lightning_norm_vec_kernel<TO, VPT>, dim3(T), dim3(threads), 0, stream, (const float*)A.o_raw, norm_w, norm_dtype, gate, ldg, \
+            gate_act, eps, factor, (TO*)out, ldo, n)
+    if (out_dtype == CO_F32) { if (n <= 2048) GO(float, 1); else GO(float, 4); }
+    else { if (n <= 2048) GO(__nv_bfloat16, 1); else GO(__nv_bfloat16, 4); }
+#undef GO
+    CO_CHECK_LAUNCH("lightning_norm_vec");
+    return 0;
+  }
   const size_t smem = (size_t)n * sizeof(float);
   if (smem > SMEM_LIMIT) CO_FAIL("lightning: %d value channels of all heads do not fit a CTA", n);
 #define GO(TO)                                                                                                                \

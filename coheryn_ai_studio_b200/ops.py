@@ -56,7 +56,7 @@ def launch_count() -> int:
 def total_launch_count() -> int:
     """Kernel launches made through every library of this package that is loaded."""
     n = launch_count()
-    for lib in list(_attn_libs.values()) + list(_maps_libs.values()) + list(_pooled_tc_libs.values()) + [
+    for lib in list(_attn_libs.values()) + list(_maps_libs.values()) + list(_options_libs.values()) + list(_pooled_tc_libs.values()) + [
             l for l in (_recurrent, _variants, _routed, _linear_recurrence, _pooled, _linear_attention, _lightning) if l is not None]:
         n += int(lib.coheryn_launch_count())
     return n
@@ -1284,18 +1284,53 @@ def maps_attention_lib(dk: int, dv: int, maps: int, values_in_keys: bool = False
     return lib
 
 
+_options_libs = {}
+# Whether prompt portions of ordinary (one-map) attention take the tcgen05 kernel with options, and from how many tokens of
+# the longest portion on (its row tiles hold 128 rows, a key/value head's query heads side by side).
+ATTN_OPTIONS = os.environ.get("COHERYN_ATTN_OPTIONS", "1") != "0"
+ATTN_OPTIONS_MIN_TOKENS = int(os.environ.get("COHERYN_ATTN_OPTIONS_MIN_TOKENS", "16"))
+
+
+def set_attention_options(on: bool) -> None:
+    global ATTN_OPTIONS
+    ATTN_OPTIONS = bool(on)
+
+
+def attention_options_lib(dk: int, dv: int):
+    lib = _options_libs.get((dk, dv))
+    if lib is None:
+        lib = build.attention_options_library(dk, dv)
+        lib.coheryn_last_error.restype = ctypes.c_char_p
+        lib.coheryn_launch_count.restype = ctypes.c_ulonglong
+        got = [ctypes.c_int(), ctypes.c_int()]
+        lib.coheryn_attention_options_shape(*[ctypes.byref(g) for g in got])
+        if tuple(g.value for g in got) != (dk, dv):
+            raise KernelError(f"the attention library was built for {tuple(g.value for g in got)}, not {(dk, dv)}")
+        _options_libs[(dk, dv)] = lib
+    return lib
+
+
+def _attention_options_ok(q, out, step, heads: int, kv_heads: int, dk: int, dv: int, page_size: int, scale: float, dense: bool) -> bool:
+    return (ATTN_OPTIONS and q.dtype == torch.bfloat16 and dk % 16 == 0 and dv % 16 == 0 and 16 <= dk <= 256 and 16 <= dv <= 256
+            and scale > 0 and heads // kv_heads <= 128 and max(step.q_lens) >= ATTN_OPTIONS_MIN_TOKENS
+            and (dense or (page_size >= 8 and (128 % page_size == 0 or page_size % 128 == 0)))
+            and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.stride(0) % 4 == 0 and out.data_ptr() % 8 == 0)
+
+
 def attention_maps(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, step, group: int,
                    num_heads: int, num_kv_heads: int, dk: int, dv: int, maps: int, page_size: int, window: Optional[int],
                    chunk: Optional[int], sink: bool, scale: float, lam: float, head_norm: bool, eps: float,
                    out_scale: float, force_simple: bool = False, sink_scores: Optional[torch.Tensor] = None,
-                   values_in_keys: bool = False, head_gates: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
+                   values_in_keys: bool = False, head_gates: Optional[torch.Tensor] = None, keep_first: int = 0,
+                   step_rows: bool = False) -> None:
     """Attention of every token of the step over its request's cache pages of ``group`` with ``maps`` score maps per
     head (output a_0 - lam * a_1 for two), a mask by chunks (``chunk``: position i sees j <= i with i // chunk ==
     j // chunk), by a window (beside which the first ``keep_first`` positions stay in sight) or causal, an optional sink term in the softmax's denominator, the head's output divided
     by its root mean square over dv (``head_norm``) and multiplied by ``out_scale``.  q [T, heads * maps * dk],
     out [T, heads * dv]; float32 arithmetic on either storage type.  ``sink_scores`` (float32 [heads]): the sink's score
     per head instead of 0.  ``values_in_keys``: the values are the first dv channels of the key rows (``v_cache`` is not
-    read).  ``head_gates`` (float32 [T, heads]): head h's output of token t is multiplied by sigmoid(head_gates[t, h])."""
+    read).  ``head_gates`` (float32 [T, heads]): head h's output of token t is multiplied by sigmoid(head_gates[t, h]).
+    ``step_rows``: the caches are the step's own rows [T, kv heads, 1, channels] ("pages" of one position; whole prompts)."""
     block_tables = step.block_tables[group]
     if head_gates is not None:
         _dev(head_gates)
@@ -1322,9 +1357,23 @@ def attention_maps(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_
     if fast:
         # rows that are whole runs of consecutive positions per request, ending at the request's last position
         _i32(step.cu_q, "cu_q"); _i32(step.kv_lens, "kv_lens")
-        lib = maps_attention_lib(dk, dv, maps, values_in_keys)
         B = len(q_lens)
-        single = any(n == 1 for n in q_lens)
+        single, longer = any(n == 1 for n in q_lens), any(n > 1 for n in q_lens)
+        if (longer and maps == 1 and not values_in_keys and not chunk and not head_norm and k_cache.is_contiguous() and v_cache.is_contiguous()
+                and _attention_options_ok(q, out, step, num_heads, num_kv_heads, dk, dv, page_size, scale, step_rows)):
+            # portions on the tcgen05 kernel; single tokens beside them on the decode kernels below
+            olib = attention_options_lib(dk, dv)
+            _check(olib, olib.coheryn_attention_options(
+                _ptr(q), c_long(q.stride(0)), c_int(T), _ptr(out), c_long(out.stride(0)), _ptr(k_cache), _ptr(v_cache),
+                c_int(k_cache.shape[0]), _ptr(block_tables), c_int(block_tables.shape[1]), _ptr(step.cu_q), _ptr(step.kv_lens), c_int(B),
+                c_int(num_heads), c_int(num_kv_heads), c_int(page_size), c_int(window or 0), c_int(keep_first), c_int(1 if step_rows else 0),
+                c_int(1 if sink else 0), _ptr(sink_scores), _ptr(head_gates), c_long(head_gates.stride(0) if head_gates is not None else 0),
+                c_float(out_scale), c_float(scale), c_int(max(q_lens) * (num_heads // num_kv_heads)), c_int(step.max_kv_len),
+                _ptr(tc_status(q.device)), _stream()))
+            longer = False
+            if not single:
+                return
+        lib = maps_attention_lib(dk, dv, maps, values_in_keys)
         floats = int(lib.coheryn_maps_scratch_floats(c_int(B), c_int(num_heads), c_int(step.max_kv_len), c_int(window or 0),
                                                      c_int(chunk or 0), c_int(keep_first))) if single else 0
         scratch = torch.empty(floats, dtype=torch.float32, device=q.device) if floats else None
@@ -1333,7 +1382,7 @@ def attention_maps(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_
             c_int(block_tables.shape[1]), _ptr(step.cu_q), _ptr(step.kv_lens), c_int(B), c_int(num_heads), c_int(num_kv_heads),
             c_int(page_size), c_int(window or 0), c_int(chunk or 0), c_int(keep_first), c_int(1 if sink else 0), c_float(scale),
             c_float(lam), c_int(1 if head_norm else 0), c_float(eps), c_float(out_scale), c_int(max(q_lens)), c_int(step.max_kv_len),
-            c_int(1 if any(n == 1 for n in q_lens) else 0), c_int(1 if any(n > 1 for n in q_lens) else 0), _ptr(scratch),
+            c_int(1 if single else 0), c_int(1 if longer else 0), _ptr(scratch),
             c_long(floats), _ptr(sink_scores), _ptr(head_gates), c_long(head_gates.stride(0) if head_gates is not None else 0),
             _stream()))
         return

@@ -607,7 +607,7 @@ class LatentAttention(Mixer):
                                      kv_lens=step.kv_lens, q_lens=step.q_lens, max_kv_len=step.max_kv_len)
         ops.attention_maps(q_full, out, keys.view(T, H, 1, dk), values.view(T, H, 1, self.dv), view, 0, H, H, dk, self.dv, 1, 1,
                            self.window, None, self.sink, self.scale, 0.0, False, self.eps, 1.0, sink_scores=self.sink_scores,
-                           head_gates=gates)
+                           head_gates=gates, step_rows=True)
 
     def forward_open(self, x: torch.Tensor, step: StepContext, cache: LayerCache, outs) -> None:
         """The gated heads' outputs in front of the output product into ``outs[0]`` ([T, heads * dv])."""

@@ -92,7 +92,7 @@ def test_neighbouring_pairs_become_halves_when_the_weights_are_bound():
     """Rotating the permuted projections in halves gives the same products of queries and keys as rotating the stored ones in
     neighbouring pairs; channels behind the rotated ones keep their place."""
     from coheryn_ai_studio_b200.config.spec import PartSpec
-    from coheryn_ai_studio_b200.parts.attention import Attention, LatentAttention, MapsAttention, PooledWindowAttention
+    from coheryn_ai_studio_b200.parts.attention import Attention, LatentAttention, PooledWindowAttention
     from coheryn_ai_studio_b200.parts.base import POSITIONS, build_part
     rng = np.random.default_rng(1)
     width, H, dim, rd, dv, rank, dims = 20, 3, 4, 10, 5, 7, 6
@@ -117,7 +117,7 @@ def test_neighbouring_pairs_become_halves_when_the_weights_are_bound():
                      plain.rotate_neighbours(d0[:, rank:].numpy(), range(9), dims, 30.0))
     assert np.allclose(got.numpy(), want, atol=1e-9) and torch.allclose(q[..., :dim], q0[..., :dim])
     assert torch.allclose(d[:, :rank], d0[:, :rank]) and torch.allclose(d[:, rank + dims:], d0[:, rank + dims:])
-    for build in (lambda: MapsAttention(CPU, 8, 1, 1, 8, 8, 1.0, position=pos), lambda: PooledWindowAttention(CPU, 8, 1, 1, 8, 8, 1.0, position=pos),
+    for build in (lambda: PooledWindowAttention(CPU, 8, 1, 1, 8, 8, 1.0, position=pos),
                   lambda: Attention(CPU, 8, 1, 1, 8, False, False, None, 1.0, position=pos)):
         with pytest.raises(ValueError):
             build()
