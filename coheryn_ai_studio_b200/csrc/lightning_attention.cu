@@ -416,53 +416,6 @@ __global__ void __launch_bounds__(256, 2) lightning_chunk_out_kernel(LightningAr
   }
 }
 
-// The same with a token's row in registers: n a multiple of 4 and at most 512 * 4 * VPT, every row on a 16-byte boundary.
-// Row, gate and weight are requested together, ahead of the sum over the row.
-template <typename TO, int VPT>
-__global__ void __launch_bounds__(512) lightning_norm_vec_kernel(const float* __restrict__ o, const void* __restrict__ w, int w_dtype,
-                                                                 const float* __restrict__ gate, long ldg, int gate_act, float eps,
-                                                                 float factor, TO* __restrict__ out, long ldo, int n) {
-  __shared__ float scratch[33];
-  co_pdl_launch_dependents();
-  const size_t t = blockIdx.x;
-  float4 x[VPT], g[VPT], wv[VPT];
-#pragma unroll
-  for (int i = 0; i < VPT; ++i) {      // no earlier kernel writes the weight
-    const int j = 4 * (threadIdx.x + i * blockDim.x);
-    if (j < n) wv[i] = make_float4(co_load_any(w, w_dtype, j), co_load_any(w, w_dtype, j + 1), co_load_any(w, w_dtype, j + 2), co_load_any(w, w_dtype, j + 3));
-  }
-  co_pdl_wait();
-  float ss = 0.f;
-#pragma unroll
-  for (int i = 0; i < VPT; ++i) {
-    const int j = 4 * (threadIdx.x + i * blockDim.x);
-    x[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (j < n) {
-      x[i] = *reinterpret_cast<const float4*>(o + t * n + j);
-      g[i] = *reinterpret_cast<const float4*>(gate + t * ldg + j);
-    }
-  }
-#pragma unroll
-  for (int i = 0; i < VPT; ++i) { ss = fmaf(x[i].x, x[i].x, ss); ss = fmaf(x[i].y, x[i].y, ss); ss = fmaf(x[i].z, x[i].z, ss); ss = fmaf(x[i].w, x[i].w, ss); }
-  const float inv = 1.0f / sqrtf(co_block_sum(ss, scratch) / (float)n + eps);
-#pragma unroll
-  for (int i = 0; i < VPT; ++i) {
-    const int j = 4 * (threadIdx.x + i * blockDim.x);
-    if (j >= n) continue;
-    const float y[4] = {(x[i].x * inv) * wv[i].x * la_gate(gate_act, g[i].x) * factor, (x[i].y * inv) * wv[i].y * la_gate(gate_act, g[i].y) * factor,
-                        (x[i].z * inv) * wv[i].z * la_gate(gate_act, g[i].z) * factor, (x[i].w * inv) * wv[i].w * la_gate(gate_act, g[i].w) * factor};
-    if constexpr (sizeof(TO) == 2) {
-      const __nv_bfloat162 lo = __floats2bfloat162_rn(y[0], y[1]), hi = __floats2bfloat162_rn(y[2], y[3]);
-      uint2 u;
-      u.x = *reinterpret_cast<const unsigned*>(&lo);
-      u.y = *reinterpret_cast<const unsigned*>(&hi);
-      *reinterpret_cast<uint2*>(out + t * ldo + j) = u;
-    } else {
-      *reinterpret_cast<float4*>(out + t * ldo + j) = make_float4(y[0], y[1], y[2], y[3]);
-    }
-  }
-}
-
 // grid (T), 256 threads: all heads of a token normalised together, times the weight, the gate and a factor.
 template <typename TO>
 __global__ void __launch_bounds__(256) lightning_norm_kernel(const float* __restrict__ o, const void* __restrict__ w, int w_dtype,
@@ -560,17 +513,6 @@ CO_EXPORT int coheryn_lightning(const float* q, long ldq, const float* k, long l
     CO_CHECK_LAUNCH("lightning_chunk_out");
   }
   const int n = H * dv;
-  if ((n & 3) == 0 && n <= 512 * 4 * 4 && (ldg & 3) == 0 && (ldo & 3) == 0 && aligned(gate) && aligned(out) && aligned(A.o_raw)) {
-    const int threads = n / 4 >= 512 ? 512 : (n / 4 + 31) / 32 * 32;
-#define GO(TO, VPT)                                                                                                           \
-  co_launch(lightning_norm_vec_kernel<TO, VPT>, dim3(T), dim3(threads), 0, stream, (const float*)A.o_raw, norm_w, norm_dtype, gate, ldg, \
-            gate_act, eps, factor, (TO*)out, ldo, n)
-    if (out_dtype == CO_F32) { if (n <= 2048) GO(float, 1); else GO(float, 4); }
-    else { if (n <= 2048) GO(__nv_bfloat16, 1); else GO(__nv_bfloat16, 4); }
-#undef GO
-    CO_CHECK_LAUNCH("lightning_norm_vec");
-    return 0;
-  }
   const size_t smem = (size_t)n * sizeof(float);
   if (smem > SMEM_LIMIT) CO_FAIL("lightning: %d value channels of all heads do not fit a CTA", n);
 #define GO(TO)                                                                                                                \
